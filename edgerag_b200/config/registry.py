@@ -78,6 +78,9 @@ def _register_builtin() -> None:
     from ..models.pudadra import PudadraConfig, pudadra_plan
 
     register_architecture(["Pudadra", "pudadra"], PudadraConfig.from_dict, pudadra_plan)
+    from ..models.sabolorn import SabolornConfig, sabolorn_plan
+
+    register_architecture(["Sabolorn", "sabolorn"], SabolornConfig.from_dict, sabolorn_plan)
 
 
 _register_builtin()

@@ -10,6 +10,8 @@
 // (window <= 0: all keys 0 .. p) and, with a window, also the keys 0 .. keep_first - 1 whatever their
 // distance.  A negative `window` stands for a mask of chunks: the query sees the keys from the start of its own run of
 // -window positions (runs counted from position 0 of the sequence) up to itself.  Query head h reads kv head h / (nq / nkv).
+// With `penalty` (float [2][nq]: r1 of every query head, then r2) the scaled score of a key d positions back is lowered by
+// r1 * ln(1 + r2 * d).
 //
 // Both kernels give every thread its own keys and its own online-softmax state (running max,
 // denominator, float accumulator of D values), so the inner loop has no cross-thread traffic;
@@ -46,7 +48,7 @@ struct LaneState {
   }
   // Visit one key: k and v point at the D elements of the key and the value row.
   template <typename T>
-  __device__ __forceinline__ void visit(const float* q_smem, const T* k, const T* v, float scale) {
+  __device__ __forceinline__ void visit(const float* q_smem, const T* k, const T* v, float scale, float lower) {
     constexpr int N = Vec<T>::N;
     float s = 0.f;
 #pragma unroll
@@ -56,7 +58,7 @@ struct LaneState {
 #pragma unroll
       for (int i = 0; i < N; ++i) s = fmaf(q_smem[d0 + i], kk[i], s);
     }
-    s *= scale;
+    s = fmaf(s, scale, -lower);
     float p;
     if (s > m) {
       const float alpha = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -106,6 +108,15 @@ __device__ __forceinline__ void warp_merge(LaneState<D>& st, float* stage, float
   __syncwarp();
 }
 
+// What a head's distance penalty takes off the score of a key `dist` positions back (no penalty: 0).
+struct Penalty {
+  float r1 = 0.f, r2 = 0.f;
+  __device__ __forceinline__ Penalty(const float* table, int head, int n_heads) {
+    if (table) { r1 = table[head]; r2 = table[n_heads + head]; }
+  }
+  __device__ __forceinline__ float at(int dist) const { return r1 != 0.f ? r1 * log1pf(r2 * (float)dist) : 0.f; }
+};
+
 constexpr int kRowWarps = 4;  // warps (query rows) per block in the row kernel
 
 // ---------------------------------------------------------------------------------------------
@@ -118,7 +129,7 @@ attention_rows_kernel(const T* __restrict__ q, int q_row_stride, const T* __rest
                       const T* __restrict__ v_pages, const int* __restrict__ block_tables, int max_pages,
                       const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                       T* __restrict__ out, int out_row_stride, int n_tokens, int nq, int nkv,
-                      int page_size, int window, int keep_first, float scale) {
+                      int page_size, int window, int keep_first, float scale, const float* __restrict__ penalty) {
   chain_wait();
   extern __shared__ float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -138,16 +149,17 @@ attention_rows_kernel(const T* __restrict__ q, int q_row_stride, const T* __rest
 
   LaneState<D> st;
   st.init();
+  const Penalty pen(penalty, h, nq);
   const int kept = min(keep_first, k_lo);     // the first keys that the window would hide
   for (int k = lane; k < kept; k += 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale);
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
   }
   for (int k = k_lo + lane; k <= pos; k += 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale);
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
   }
   float m_w, l_w, o[(D + 31) / 32];
   warp_merge<D>(st, stage, m_w, l_w, o);
@@ -176,7 +188,7 @@ attention_decode_split_kernel(const T* __restrict__ q, int q_row_stride, const T
                               int max_pages, const int* __restrict__ token_of_seq,
                               const int* __restrict__ positions, float* __restrict__ part_acc,
                               float* __restrict__ part_ml, int max_splits, int nq, int nkv, int page_size,
-                              int window, int keep_first, int split_keys, float scale) {
+                              int window, int keep_first, int split_keys, float scale, const float* __restrict__ penalty) {
   chain_wait();
   extern __shared__ float smem[];
   float* q_s = smem;                                   // D
@@ -202,15 +214,16 @@ attention_decode_split_kernel(const T* __restrict__ q, int q_row_stride, const T
   const int* bt = block_tables + (size_t)seq * max_pages;
   LaneState<D> st;
   st.init();
+  const Penalty pen(penalty, h, nq);
   for (int k = (int)threadIdx.x; k < kept; k += kDecodeWarps * 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale);
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
   }
   for (int k = begin + (int)threadIdx.x; k < end; k += kDecodeWarps * 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale);
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
   }
   float m_w, l_w, o[(D + 31) / 32];
   warp_merge<D>(st, stage + warp * 32 * (D + 1), m_w, l_w, o);
@@ -284,7 +297,7 @@ template <typename T, int D>
 int launch_rows(const void* q, int q_row_stride, const void* k_pages, const void* v_pages,
                 const int* block_tables, int max_pages, const int* seq_of_token, const int* positions,
                 void* out, int out_row_stride, int n_tokens, int nq, int nkv, int page_size, int window,
-                int keep_first, float scale, cudaStream_t s) {
+                int keep_first, float scale, const float* penalty, cudaStream_t s) {
   const size_t smem = (size_t)(kRowWarps * D + kRowWarps * 32 * (D + 1)) * sizeof(float);
   auto kern = attention_rows_kernel<T, D>;
   if (smem > 48 * 1024) {
@@ -294,7 +307,7 @@ int launch_rows(const void* q, int q_row_stride, const void* k_pages, const void
   dim3 grid((n_tokens + kRowWarps - 1) / kRowWarps, nq);
   launch_chained(kern, dim3(grid), dim3(kRowWarps * 32), smem, s, (const T*)q, q_row_stride, (const T*)k_pages, (const T*)v_pages,
       block_tables, max_pages, seq_of_token, positions, (T*)out, out_row_stride, n_tokens, nq, nkv,
-      page_size, window, keep_first, scale);
+      page_size, window, keep_first, scale, penalty);
   return check_launch("attention_rows");
 }
 
@@ -302,7 +315,7 @@ template <typename T, int D>
 int launch_decode(const void* q, int q_row_stride, const void* k_pages, const void* v_pages,
                   const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                   void* out, int out_row_stride, float* part_acc, float* part_ml, int max_splits, int n_seqs,
-                  int nq, int nkv, int page_size, int window, int keep_first, int split_keys, float scale, cudaStream_t s) {
+                  int nq, int nkv, int page_size, int window, int keep_first, int split_keys, float scale, const float* penalty, cudaStream_t s) {
   const size_t smem =
       (size_t)(D + kDecodeWarps * 32 * (D + 1) + kDecodeWarps * (D + 2)) * sizeof(float);
   auto kern = attention_decode_split_kernel<T, D>;
@@ -313,7 +326,7 @@ int launch_decode(const void* q, int q_row_stride, const void* k_pages, const vo
   dim3 grid(max_splits, nq, n_seqs);
   launch_chained(kern, dim3(grid), dim3(kDecodeWarps * 32), smem, s, (const T*)q, q_row_stride, (const T*)k_pages,
       (const T*)v_pages, block_tables, max_pages, token_of_seq, positions, part_acc, part_ml, max_splits,
-      nq, nkv, page_size, window, keep_first, split_keys, scale);
+      nq, nkv, page_size, window, keep_first, split_keys, scale, penalty);
   int rc = check_launch("attention_decode_split");
   if (rc) return rc;
   launch_chained(attention_decode_combine_kernel<T>, dim3(dim3(nq, n_seqs)), dim3(64), 0, s, part_acc, part_ml, token_of_seq,
@@ -353,13 +366,13 @@ ERB_EXPORT int erb_attention_rows(const void* q, int q_row_stride, const void* k
                                   const int* block_tables, int max_pages, const int* seq_of_token,
                                   const int* positions, void* out, int out_row_stride, int n_tokens, int nq,
                                   int nkv, int head_dim, int page_size, int window, int keep_first, float scale,
-                                  void* stream) {
+                                  const float* penalty, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   int rc = check_common("attention_rows", nq, nkv, head_dim, page_size, max_pages);
   if (rc) return rc;
   cudaStream_t s = (cudaStream_t)stream;
   ERB_DISPATCH_D(launch_rows, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, seq_of_token,
-                 positions, out, out_row_stride, n_tokens, nq, nkv, page_size, window, window > 0 ? keep_first : 0, scale, s)
+                 positions, out, out_row_stride, n_tokens, nq, nkv, page_size, window, window > 0 ? keep_first : 0, scale, penalty, s)
   return fail(ERB_ERR_UNSUPPORTED, "attention_rows: head_dim %d", head_dim);
 }
 
@@ -371,7 +384,7 @@ ERB_EXPORT int erb_attention_decode(const void* q, int q_row_stride, const void*
                                     const int* token_of_seq, const int* positions, void* out,
                                     int out_row_stride, float* part_acc, float* part_ml, int max_splits,
                                     int n_seqs, int nq, int nkv, int head_dim, int page_size, int window,
-                                    int keep_first, int split_keys, float scale, void* stream) {
+                                    int keep_first, int split_keys, float scale, const float* penalty, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
   int rc = check_common("attention_decode", nq, nkv, head_dim, page_size, max_pages);
   if (rc) return rc;
@@ -381,7 +394,7 @@ ERB_EXPORT int erb_attention_decode(const void* q, int q_row_stride, const void*
   cudaStream_t s = (cudaStream_t)stream;
   ERB_DISPATCH_D(launch_decode, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                  positions, out, out_row_stride, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size,
-                 window, window > 0 ? keep_first : 0, split_keys, scale, s)
+                 window, window > 0 ? keep_first : 0, split_keys, scale, penalty, s)
   return fail(ERB_ERR_UNSUPPORTED, "attention_decode: head_dim %d", head_dim);
 }
 
@@ -444,5 +457,5 @@ ERB_EXPORT int erb_attention_decode_static(const void* q, int q_row_stride, cons
   float* part_ml = base + (size_t)n_seqs * nq * max_splits * head_dim;
   return erb_attention_decode(q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                               positions, out, out_row_stride, part_acc, part_ml, max_splits, n_seqs, nq, nkv,
-                              head_dim, page_size, window, 0, split_keys, scale, stream);
+                              head_dim, page_size, window, 0, split_keys, scale, nullptr, stream);
 }

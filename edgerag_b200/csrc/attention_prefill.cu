@@ -32,6 +32,9 @@
 // `key_splits` ranges, one block per range (blockIdx.z): a block leaves its rows' unnormalised O, reference
 // maximum and sum in scratch, and a second kernel merges the ranges of each row.
 //
+// With `penalty` (float [2][nq]: r1 of every query head, then r2) the scaled score of a key d positions back is lowered by
+// r1 * ln(1 + r2 * d); the kernel is compiled with and without it.
+//
 // Every wait is bounded: a thread that gives up raises a block-wide flag, every other wait of the
 // block then ends too, the block records a code in *status, lets its copies land, frees its TMEM
 // and returns.
@@ -75,13 +78,15 @@ constexpr float kSumLimit = 1048576.f;   // a tile's sum of P from which on the 
 constexpr uint32_t kIdescS = mma_idesc(BM, BN, false);
 constexpr uint32_t kIdescO = mma_idesc(BM, HD, true);
 
+template <bool PEN>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                          const __nv_bfloat16* __restrict__ q, int q_row_stride,
                          const int* __restrict__ block_tables, int max_pages, const int* __restrict__ seq_starts,
                          const int* __restrict__ positions, __nv_bfloat16* __restrict__ out, int out_row_stride,
                          int n_seqs, int nq, int nkv, int page_size, float scale_log2, int* __restrict__ status,
-                         int key_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep_first) {
+                         int key_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep_first,
+                         const float* __restrict__ penalty) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;             // the swizzle repeats every 1024 bytes
@@ -311,12 +316,17 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     };
     float m_ref = -INFINITY, l_run = 0.f;                // l_run: this thread's half of the row's sum
     const int win_lo = first_visible_key(my_pos, window);               // first key of this row's window or chunk
+    const float pen_r1 = PEN ? penalty[h] : 0.f, pen_r2 = PEN ? penalty[nq + h] : 0.f;
     auto hidden = [&](int key) { return key > my_pos || (key < win_lo && key >= keep_first); };
     for (int j = j0; j < n_end[t]; ++j) {
       wait(kBarSFull + t, (j - j0) & 1);
       if (!ok) break;
       fence_after_sync();
       const int tile_key0 = tile_of(j) * BN, key0 = tile_key0 + half * 64;
+      // 1 + r2 * (distance to this thread's first key of the tile); the keys after it are r2 less each (a key behind the
+      // row's own is masked: its logarithm, which may be no number, is never used)
+      const float pen_at0 = PEN ? fmaf(pen_r2, (float)(my_pos - key0), 1.f) : 0.f;
+      auto lower = [&](int i) { return pen_r1 * __log2f(fmaf(-pen_r2, (float)i, pen_at0)); };   // of key key0 + i, log2 domain
       // some row of the query tile has hidden keys here: keys after its own, or keys before its window that are not kept
       const bool diagonal = tile_key0 + BN - 1 > pos0 + t * BM || (window != 0 && tile_key0 < first_visible_key(pos0 + t * BM + BM - 1, window));
       // The exponentials are taken against the reference maximum of the tiles before, without looking
@@ -336,13 +346,16 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
             tmem_ld32(t_s + 32 * c, s);
             tmem_ld_wait();
 #pragma unroll
-            for (int i = 0; i < 32; ++i) m_half = fmaxf(m_half, (diagonal && hidden(key0 + 32 * c + i)) ? -INFINITY : s[i]);
+            for (int i = 0; i < 32; ++i) {
+              if (PEN) s[i] = fmaf(s[i], scale_log2, -lower(32 * c + i));
+              m_half = fmaxf(m_half, (diagonal && hidden(key0 + 32 * c + i)) ? -INFINITY : s[i]);
+            }
           }
           *mine = m_half;
           named_barrier(pair_barrier, 64);
           // (scale > 0: the maximum of the scaled scores.  A range of keys may begin with a tile of which a row
           // sees nothing: its reference then stays at a finite floor, so that exp2(-inf - reference) is 0, not NaN.)
-          const float m_tile = fmaxf(fmaxf(m_half, *partners) * scale_log2, -1e30f);
+          const float m_tile = fmaxf(fmaxf(m_half, *partners) * (PEN ? 1.f : scale_log2), -1e30f);
           float alpha = 1.f;
           if (m_tile > m_ref) {
             alpha = fast_exp2(m_ref - m_tile);                          // 0 on the first tile
@@ -373,6 +386,10 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           tmem_ld_wait();
           if (c + 1 < 4) tmem_ld16(t_s + 16 * (c + 1), s[(c + 1) & 1]);
           float* sc = s[c & 1];
+          if (PEN) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) sc[i] = fmaf(sc[i], scale_log2, -lower(16 * c + i));
+          }
           if (diagonal) {
 #pragma unroll
             for (int i = 0; i < 16; ++i)
@@ -380,8 +397,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           }
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            const float p0 = fast_exp2(fmaf(sc[2 * i], scale_log2, -m_ref));
-            const float p1 = fast_exp2(fmaf(sc[2 * i + 1], scale_log2, -m_ref));
+            const float p0 = fast_exp2(PEN ? sc[2 * i] - m_ref : fmaf(sc[2 * i], scale_log2, -m_ref));
+            const float p1 = fast_exp2(PEN ? sc[2 * i + 1] - m_ref : fmaf(sc[2 * i + 1], scale_log2, -m_ref));
             l4[i & 3] += p0 + p1;
             __nv_bfloat162 b = __floats2bfloat162_rn(p0, p1);
             packed[8 * c + i] = *reinterpret_cast<uint32_t*>(&b);
@@ -517,7 +534,8 @@ ERB_EXPORT int erb_attention_prefill_tc(const void* q, int q_row_stride, const v
                                         const int* seq_starts, const int* positions, void* out, int out_row_stride,
                                         int n_seqs, int n_blocks, int nq, int nkv, int head_dim, int page_size,
                                         float scale, int* status, int key_splits, int first_row, int n_rows,
-                                        float* part_o, float* part_ml, int window, int keep_first, void* stream) {
+                                        float* part_o, float* part_ml, int window, int keep_first, const float* penalty,
+                                        void* stream) {
   if (n_seqs <= 0 || n_blocks <= 0) return ERB_OK;
   if (key_splits < 1 || key_splits > 64 || (key_splits > 1 && (!part_o || !part_ml || first_row < 0 || n_rows <= 0 || ((uintptr_t)part_o & 15))))
     return fail(ERB_ERR_ARG, "attention_prefill_tc: bad split arguments");
@@ -537,18 +555,18 @@ ERB_EXPORT int erb_attention_prefill_tc(const void* q, int q_row_stride, const v
   if ((rc = pool_map(&mk, k_pages, pool_rows, (unsigned)page_size, "attention_prefill_tc")) ||
       (rc = pool_map(&mv, v_pages, pool_rows, (unsigned)page_size, "attention_prefill_tc")))
     return rc;
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)kSmemBytes);
+  auto kern = penalty ? attention_prefill_kernel<true> : attention_prefill_kernel<false>;
+  static bool configured[2] = {false, false};
+  if (!configured[penalty != nullptr]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemBytes);
     if (e != cudaSuccess) return fail(ERB_ERR_CUDA, "attention_prefill_tc: %s", cudaGetErrorString(e));
-    configured = true;
+    configured[penalty != nullptr] = true;
   }
   const float scale_log2 = scale * 1.4426950408889634f;
-  launch_chained(attention_prefill_kernel, dim3(nq, n_blocks, key_splits), dim3(kThreads), kSmemBytes, (cudaStream_t)stream, mk, mv,
+  launch_chained(kern, dim3(nq, n_blocks, key_splits), dim3(kThreads), kSmemBytes, (cudaStream_t)stream, mk, mv,
                  (const __nv_bfloat16*)q, q_row_stride, block_tables, max_pages, seq_starts, positions,
                  (__nv_bfloat16*)out, out_row_stride, n_seqs, nq, nkv, page_size, scale_log2, status, key_splits, part_o, part_ml,
-                 window, window > 0 && keep_first > 0 ? keep_first : 0);
+                 window, window > 0 && keep_first > 0 ? keep_first : 0, penalty);
   if ((rc = check_launch("attention_prefill_tc")) || key_splits == 1) return rc;
   launch_chained(attention_prefill_merge_kernel, dim3((n_rows * nq + 3) / 4), dim3(128), 0, (cudaStream_t)stream, part_o, part_ml,
                  (__nv_bfloat16*)out, out_row_stride, first_row, n_rows, nq, key_splits);

@@ -25,6 +25,9 @@ ERB_DEFINE_LAST_ERROR(erb_last_error)
 // shuffles and every lane keeps the running max, denominator and 8 accumulators of its slice.
 // Partial results go to the same scratch layout as the general kernel; a combine kernel merges the
 // splits in order.  bfloat16, head size 32, 64 or 128.
+//
+// Both kernels take an optional penalty on the distance (`penalty`, float [2][nq]: r1 of every query head, then r2):
+// the scaled score of a key d positions back is lowered by r1 * ln(1 + r2 * d).
 // =============================================================================================
 namespace {
 
@@ -33,6 +36,15 @@ constexpr int kDecWarps = kDecThreads / 32;
 constexpr int kStages = 3;
 constexpr int kMaxGroup = 8;          // query heads per kv head handled in one pass
 constexpr int kKeysPerGroup = 4;      // keys a lane group handles per stage (independent chains)
+
+// A head's distance penalty in the log2 domain (no table: no penalty).
+struct Penalty2 {
+  float r1 = 0.f, r2 = 0.f;
+  __device__ __forceinline__ void load(const float* table, int head, int n_heads) {
+    if (table) { r1 = table[head]; r2 = table[n_heads + head]; }
+  }
+  __device__ __forceinline__ float at(int dist) const { return r1 * __log2f(fmaf(r2, (float)dist, 1.f)); }
+};
 
 __device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
@@ -125,7 +137,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
                              float* __restrict__ part_acc, float* __restrict__ part_ml, int max_splits, int nq,
                              int nkv, int page_size, int split_keys, float scale_log2, int hg,
                              __nv_bfloat16* __restrict__ out, int out_row_stride, int* __restrict__ status,
-                             int* __restrict__ counters, int window, int keep_first) {
+                             int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty) {
   // Everything up to chain_wait() below reads only what earlier steps or the host wrote (the batch's
   // metadata, keys and values of earlier tokens), so it runs while the kernel before this one (the
   // one that rotates q and writes this step's keys and values) is still at work.
@@ -247,6 +259,9 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
 #pragma unroll
     for (int i = 0; i < 8; ++i) qr[g][i] = tmp[i] * scale_log2;
   }
+  Penalty2 pen[R];
+#pragma unroll
+  for (int g = 0; g < R; ++g) pen[g].load(penalty, (serves ? kvh : kvh0) * R + g, nq);
   float m_run[R], l_run[R], acc[R][8];
 #pragma unroll
   for (int g = 0; g < R; ++g) {
@@ -308,6 +323,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
         float m_new = m_run[g];
 #pragma unroll
         for (int u = 0; u < kKeysPerGroup; ++u) {
+          if (penalty) sc[g][u] -= pen[g].at(pos - (key0 + u));
           if (hidden[u]) sc[g][u] = -INFINITY;     // keys past the end of the split or before the window
           m_new = fmaxf(m_new, sc[g][u]);
         }
@@ -463,7 +479,7 @@ int launch_decode_bulk(const void* q, int q_row_stride, const void* k_pages, con
                        const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                        float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int page_size,
                        int split_keys, float scale_log2, void* out, int out_row_stride, int* status, int* counters, int head_group,
-                       int window, int keep_first, cudaStream_t s) {
+                       int window, int keep_first, const float* penalty, cudaStream_t s) {
   const int hg = decode_head_group(nkv, D, page_size, split_keys, head_group);
   if (hg <= 0) return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: %d heads per block with pages of %d and splits of %d", head_group, page_size, split_keys);
   constexpr int STAGE_BYTES = kDecWarps * (32 / (D / 8)) * kKeysPerGroup * D * 2;
@@ -481,7 +497,7 @@ int launch_decode_bulk(const void* q, int q_row_stride, const void* k_pages, con
   launch_chained(kern, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kDecThreads), smem, s, (const __nv_bfloat16*)q, q_row_stride,
       (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_tables, max_pages, token_of_seq, positions,
       part_acc, part_ml, max_splits, nq, nkv, page_size, split_keys, scale_log2, hg, (__nv_bfloat16*)out, out_row_stride, status, counters,
-      window, keep_first);
+      window, keep_first, penalty);
   return check_launch("attention_decode_bulk");
 }
 
@@ -490,12 +506,12 @@ int dispatch_group(int r, const void* q, int q_row_stride, const void* k_pages, 
                    const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                    float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int page_size,
                    int split_keys, float scale_log2, void* out, int out_row_stride, int* status, int* counters, int head_group,
-                   int window, int keep_first, cudaStream_t s) {
+                   int window, int keep_first, const float* penalty, cudaStream_t s) {
 #define ERB_R(RR)                                                                                              \
   case RR: return launch_decode_bulk<D, RR>(q, q_row_stride, k_pages, v_pages, block_tables, max_pages,        \
                                             token_of_seq, positions, part_acc, part_ml, max_splits, n_seqs, nq, \
                                             nkv, page_size, split_keys, scale_log2, out, out_row_stride,       \
-                                            status, counters, head_group, window, keep_first, s);
+                                            status, counters, head_group, window, keep_first, penalty, s);
   switch (r) { ERB_R(1) ERB_R(2) ERB_R(3) ERB_R(4) ERB_R(5) ERB_R(6) ERB_R(7) ERB_R(8) }
 #undef ERB_R
   return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: %d query heads per kv head (at most %d)", r, kMaxGroup);
@@ -560,7 +576,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             float* __restrict__ part_acc, float* __restrict__ part_ml, int max_splits, int nq,
                             int nkv, int page_size, int split_keys, float scale_log2, int hg,
                             __nv_bfloat16* __restrict__ out, int out_row_stride, int* __restrict__ status,
-                            int* __restrict__ counters, int window, int keep_first) {
+                            int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty) {
   constexpr int D = 64;
   const int R = nq / nkv;
   extern __shared__ uint8_t smem_raw[];
@@ -679,6 +695,8 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       qa[ks][1] = real ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * j + 8) : 0u;
     }
   }
+  Penalty2 pen;
+  if (serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
   float o[8][4];
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb)
@@ -734,7 +752,9 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           const int key = key0 + 8 * b + 2 * j + i;
           // (keys past the split's end, and keys of the window's first page that lie before the window and are not kept)
           const bool seen = key < n_here && !(key_abs0 + key < k_lo && key_abs0 + key >= keep_first);
-          sc[b][i] = seen ? sc[b][i] * scale_log2 : -INFINITY;
+          sc[b][i] *= scale_log2;
+          if (penalty) sc[b][i] -= pen.at(pos - (key_abs0 + key));
+          if (!seen) sc[b][i] = -INFINITY;
           m_new = fmaxf(m_new, sc[b][i]);
         }
       m_new = fmaxf(m_new, __shfl_xor_sync(0xffffffffu, m_new, 1));
@@ -824,7 +844,7 @@ ERB_EXPORT int erb_attention_decode_gqa(const void* q, int q_row_stride, const v
                                         const int* token_of_seq, const int* positions, void* out, int out_row_stride,
                                         float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv,
                                         int head_dim, int page_size, int split_keys, float scale, int* status,
-                                        int* counters, int window, int keep_first, void* stream) {
+                                        int* counters, int window, int keep_first, const float* penalty, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
   keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   if (!erb_attention_decode_gqa_supported(nq, nkv, head_dim, page_size, split_keys))
@@ -862,7 +882,7 @@ ERB_EXPORT int erb_attention_decode_gqa(const void* q, int q_row_stride, const v
   launch_chained(attention_decode_gqa_kernel, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kGqaThreads), smem, s,
                  mk, mv, mkl, mvl, (const __nv_bfloat16*)q, q_row_stride, block_tables, max_pages, token_of_seq, positions,
                  part_acc, part_ml, max_splits, nq, nkv, page_size, split_keys, scale_log2, hg, (__nv_bfloat16*)out, out_row_stride,
-                 status, counters, window, keep_first);
+                 status, counters, window, keep_first, penalty);
   // a single split wrote the result itself; with counters the block that finishes last merges the splits
   if ((rc = check_launch("attention_decode_gqa")) || max_splits == 1 || counters) return rc;
   launch_chained(attention_decode_bulk_combine_kernel, dim3(dim3(nq, n_seqs)), dim3(64), 0, s, part_acc, part_ml, token_of_seq, positions,
@@ -894,7 +914,7 @@ ERB_EXPORT int erb_attention_decode_bulk(const void* q, int q_row_stride, const 
                                          const int* positions, void* out, int out_row_stride, float* part_acc,
                                          float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int head_dim,
                                          int page_size, int split_keys, float scale, int* status, int* counters,
-                                         int head_group, int window, int keep_first, void* stream) {
+                                         int head_group, int window, int keep_first, const float* penalty, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
   if (nq <= 0 || nkv <= 0 || nq % nkv) return fail(ERB_ERR_ARG, "attention_decode_bulk: bad head counts");
   keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
@@ -912,13 +932,13 @@ ERB_EXPORT int erb_attention_decode_bulk(const void* q, int q_row_stride, const 
   switch (head_dim) {
     case 32: rc = dispatch_group<32>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                      positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size, split_keys,
-                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, s); break;
+                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
     case 64: rc = dispatch_group<64>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                      positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size, split_keys,
-                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, s); break;
+                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
     case 128: rc = dispatch_group<128>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                        positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size,
-                                       split_keys, scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, s); break;
+                                       split_keys, scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
     default: return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: head_dim %d (takes 32, 64, 128)", head_dim);
   }
   // a single split wrote the result itself; with counters the block that finishes last merges the splits

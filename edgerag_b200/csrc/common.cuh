@@ -91,6 +91,26 @@ __device__ __forceinline__ void load4(const float* p, float* out) {
   out[0] = raw.x; out[1] = raw.y; out[2] = raw.z; out[3] = raw.w;
 }
 
+// Four neighbouring elements as floats (pointers aligned to four elements).
+template <typename T> struct Pack4;
+template <> struct Pack4<float> {
+  static __device__ __forceinline__ void load(const float* p, float* v) { load4(p, v); }
+  static __device__ __forceinline__ void store(float* p, const float* v) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  }
+};
+template <> struct Pack4<__nv_bfloat16> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* v) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
+    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  }
+};
+
 // silu(g) * u in float.  Where the result is rounded to 16 bits (ERB_ELEM == 1) the exponential and the
 // division are the fast forms (relative error about 2^-21, far below that rounding); the 32-bit path keeps
 // the exact ones.  Every kernel that gates (the gate kernel, the gated epilogues of the products for few

@@ -93,25 +93,6 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ hidden, const T* __restri
 }
 
 // Four elements per thread and step (hidden_size a multiple of 4): 16-byte accesses to the residual.
-template <typename T> struct Pack4;
-template <> struct Pack4<float> {
-  static __device__ __forceinline__ void load(const float* p, float* v) { load4(p, v); }
-  static __device__ __forceinline__ void store(float* p, const float* v) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  }
-};
-template <> struct Pack4<__nv_bfloat16> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* v) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
-    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
-  }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float* v) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
-  }
-};
-
 // The same with 16-byte accesses.  The order in which a row's squares are added is that of VT
 // "virtual threads" (element group g of the row belongs to virtual thread g % VT; warp trees over
 // 32 neighbouring virtual threads, then one tree over the warp sums), whatever the number of real
@@ -764,7 +745,7 @@ ERB_EXPORT int erb_softcap(float* x, int n_rows, int width, int stride, float ca
 }
 
 // ---------------------------------------------------------------------------------------------
-// Residual add between two layer norms (weight and bias; the variance is the mean of the squared
+// Residual add between two layer norms (weight and optional bias; the variance is the mean of the squared
 // deviations from the mean, both taken in float over the whole row):
 //   d = delta[row]                       rows of T, or float partial sums added in order and rounded to T
 //   d = LN(d; post_w, post_b)            when post_w is given: the norm that closes a sublayer, kept in float
@@ -812,7 +793,7 @@ add_layernorm_kernel(float* __restrict__ hidden, const T* __restrict__ delta, co
       }
       const float rs = rsqrtf(block_sum(sq, scratch) * inv_w + post_eps);
       for (int i = threadIdx.x; i < width; i += blockDim.x)
-        row_cache[i] = (row_cache[i] - mean) * rs * post_w[i] + post_b[i];
+        row_cache[i] = (row_cache[i] - mean) * rs * post_w[i] + (post_b ? post_b[i] : 0.f);
     }
   }
   float sum = 0.f;
@@ -839,7 +820,7 @@ add_layernorm_kernel(float* __restrict__ hidden, const T* __restrict__ delta, co
   }
   const float rs = rsqrtf(block_sum(sq, scratch) * inv_w + eps);
   for (int i = threadIdx.x; i < width; i += blockDim.x)
-    Elem<T>::store(y + i, (row_cache[i] - mean) * rs * w[i] + b[i]);
+    Elem<T>::store(y + i, (row_cache[i] - mean) * rs * w[i] + (b ? b[i] : 0.f));
 }
 
 // The same with 16-byte accesses and the row in registers: a thread owns up to V groups of four neighbouring
@@ -911,9 +892,9 @@ add_layernorm_vec4_kernel(float* __restrict__ hidden, const T* __restrict__ delt
 #pragma unroll
       for (int v = 0; v < V; ++v) {
         if (!on[v]) continue;
-        float pw[4], pb[4];
+        float pw[4], pb[4] = {0.f, 0.f, 0.f, 0.f};
         load4(post_w + col[v], pw);
-        load4(post_b + col[v], pb);
+        if (post_b) load4(post_b + col[v], pb);
 #pragma unroll
         for (int i = 0; i < 4; ++i) x[v][i] = (x[v][i] - mean) * rs * pw[i] + pb[i];
       }
@@ -952,9 +933,9 @@ add_layernorm_vec4_kernel(float* __restrict__ hidden, const T* __restrict__ delt
 #pragma unroll
   for (int v = 0; v < V; ++v) {
     if (!on[v]) continue;
-    float ww[4], wb[4], res[4];
+    float ww[4], wb[4] = {0.f, 0.f, 0.f, 0.f}, res[4];
     load4(w + col[v], ww);
-    load4(b + col[v], wb);
+    if (b) load4(b + col[v], wb);
 #pragma unroll
     for (int i = 0; i < 4; ++i) res[i] = (hv[v][i] - mean) * rs * ww[i] + wb[i];
     Pack4<T>::store(y + col[v], res);
@@ -975,8 +956,8 @@ ERB_EXPORT int erb_add_layernorm(void* hidden, const void* delta, int n_parts, l
                                  const float* post_b, float post_eps, const float* w, const float* b, float eps, void* out,
                                  int out_ld, const int* rows, int n_rows, int width, int write_back, void* stream) {
   if (n_rows <= 0) return ERB_OK;
-  if (width <= 0 || (out && out_ld < width) || (w && !b) || (post_w && !post_b) || (post_w && !delta))
-    return fail(ERB_ERR_ARG, "add_layernorm: bad sizes or a weight without its bias");
+  if (width <= 0 || (out && out_ld < width) || (b && !w) || (post_b && !post_w) || (post_w && !delta))
+    return fail(ERB_ERR_ARG, "add_layernorm: bad sizes or a bias without its weight");
   const elem_t* d_rows = n_parts > 0 ? (const elem_t*)nullptr : (const elem_t*)delta;
   const float* d_parts = n_parts > 0 ? (const float*)delta : (const float*)nullptr;
   const uintptr_t all = (uintptr_t)hidden | (uintptr_t)delta | (uintptr_t)post_w | (uintptr_t)post_b | (uintptr_t)w | (uintptr_t)b |
@@ -1687,4 +1668,26 @@ ERB_EXPORT int erb_scale_rows(float* x, int n_rows, int width, int stride, float
   if (y > 64) y = 64;
   launch_chained(scale_rows_kernel, dim3(n_rows, y), dim3(256), 0, (cudaStream_t)stream, x, width, stride, scale);
   return check_launch("scale_rows");
+}
+
+// ---------------------------------------------------------------------------------------------
+// x[t][i] *= sigmoid(gate[t][i]), in float, rounded once: an output gate with an entry per column.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void sigmoid_gate_kernel(T* __restrict__ x, int ld_x, const T* __restrict__ gate, int ld_g, int width) {
+  chain_wait();
+  T* row = x + (size_t)blockIdx.x * ld_x;
+  const T* g = gate + (size_t)blockIdx.x * ld_g;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < width; i += gridDim.y * blockDim.x)
+    Elem<T>::store(row + i, Elem<T>::load(row + i) / (1.f + expf(-Elem<T>::load(g + i))));
+}
+
+ERB_EXPORT int erb_sigmoid_gate(void* x, int ld_x, const void* gate, int ld_g, int n_rows, int width, void* stream) {
+  if (n_rows <= 0 || width <= 0) return ERB_OK;
+  if (ld_x < width || ld_g < width) return fail(ERB_ERR_ARG, "sigmoid_gate: strides must cover a row");
+  int y = (width + 1023) / 1024;
+  if (y > 64) y = 64;
+  launch_chained(sigmoid_gate_kernel<elem_t>, dim3(n_rows, y), dim3(256), 0, (cudaStream_t)stream, (elem_t*)x, ld_x,
+                 (const elem_t*)gate, ld_g, width);
+  return check_launch("sigmoid_gate");
 }

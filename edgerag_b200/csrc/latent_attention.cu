@@ -17,7 +17,8 @@
 //                            one split of them), an optional sink in the denominator, an optional
 //                            sigmoid gate per head on the result.
 //   latent_combine_kernel    merges the splits of a row in split order.
-// Rotation convention: neighbouring pairs (2i, 2i+1), angle = position * inv_freq[i] in float.
+// Rotation convention: neighbouring pairs (2i, 2i+1), angle = position * inv_freq[i] in float; cosine and sine are both
+// multiplied by `rot_mult` (1 for a plain rotation).
 #include "common.cuh"
 
 using namespace erb;
@@ -43,7 +44,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 latent_store_kernel(const T* __restrict__ proj, int ld, int off_kv, int R, int dr, const float* __restrict__ kv_weight,
                     float eps, const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dims,
-                    const int* __restrict__ slots, T* __restrict__ pages, int off_q, int q_rank,
+                    float rot_mult, const int* __restrict__ slots, T* __restrict__ pages, int off_q, int q_rank,
                     const float* __restrict__ q_weight, T* __restrict__ q_latent) {
   chain_wait();
   __shared__ float scratch[32];
@@ -67,6 +68,7 @@ latent_store_kernel(const T* __restrict__ proj, int ld, int off_kv, int R, int d
         if (2 * i < rot_dims) {
           float sn, cs;
           sincosf(pos * inv_freq[i], &sn, &cs);
+          sn *= rot_mult; cs *= rot_mult;
           const float a = u * cs - v * sn, b = v * cs + u * sn;
           u = a; v = b;
         }
@@ -93,7 +95,7 @@ latent_store_kernel(const T* __restrict__ proj, int ld, int off_kv, int R, int d
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_q_rotate_kernel(const T* __restrict__ q, int ld, int H, int dn, int dr, int R, const int* __restrict__ positions,
-                       const float* __restrict__ inv_freq, int rot_dims, float* __restrict__ q_lat) {
+                       const float* __restrict__ inv_freq, int rot_dims, float rot_mult, float* __restrict__ q_lat) {
   chain_wait();
   const int t = blockIdx.x;
   const float pos = (float)positions[t];
@@ -105,6 +107,7 @@ latent_q_rotate_kernel(const T* __restrict__ q, int ld, int H, int dn, int dr, i
     if (2 * i < rot_dims) {
       float sn, cs;
       sincosf(pos * inv_freq[i], &sn, &cs);
+      sn *= rot_mult; cs *= rot_mult;
       const float a = u * cs - v * sn, b = v * cs + u * sn;
       u = a; v = b;
     }
@@ -595,7 +598,7 @@ void launch_attention(dim3 grid, cudaStream_t stream, const float* q_lat, const 
 
 // The token's cache row from its down-projection (when off_kv >= 0) and its query latent (when q_rank > 0).
 ERB_EXPORT int erb_latent_store(const void* proj, int n_tokens, int ld, int off_kv, int R, int dr, const float* kv_weight,
-                                float eps, const int* positions, const float* inv_freq, int rot_dims, const int* slots,
+                                float eps, const int* positions, const float* inv_freq, int rot_dims, float rot_mult, const int* slots,
                                 void* pages, int off_q, int q_rank, const float* q_weight, void* q_latent, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   if (off_kv >= 0 && (R <= 0 || dr < 0 || dr % 2 || rot_dims > dr || rot_dims % 2 || !kv_weight || !slots || !pages ||
@@ -603,18 +606,18 @@ ERB_EXPORT int erb_latent_store(const void* proj, int n_tokens, int ld, int off_
     return fail(ERB_ERR_ARG, "latent_store: bad sizes or missing tensors for the cache row");
   if (q_rank > 0 && (!q_weight || !q_latent)) return fail(ERB_ERR_ARG, "latent_store: the query latent needs a weight and a target");
   launch_chained(latent_store_kernel<elem_t>, dim3(n_tokens), dim3(128), 0, (cudaStream_t)stream, (const elem_t*)proj, ld,
-                 off_kv, R, dr, kv_weight, eps, positions, inv_freq, rot_dims, slots, (elem_t*)pages, off_q, q_rank, q_weight,
+                 off_kv, R, dr, kv_weight, eps, positions, inv_freq, rot_dims, rot_mult, slots, (elem_t*)pages, off_q, q_rank, q_weight,
                  (elem_t*)q_latent);
   return check_launch("latent_store");
 }
 
 ERB_EXPORT int erb_latent_q_rotate(const void* q, int n_tokens, int ld, int H, int dn, int dr, int R, const int* positions,
-                                   const float* inv_freq, int rot_dims, float* q_lat, void* stream) {
+                                   const float* inv_freq, int rot_dims, float rot_mult, float* q_lat, void* stream) {
   if (n_tokens <= 0 || dr == 0) return ERB_OK;
   if (dr % 2 || rot_dims > dr || rot_dims % 2 || (rot_dims > 0 && !inv_freq))
     return fail(ERB_ERR_ARG, "latent_q_rotate: the rotated part must be even and at least as wide as the rotation");
   launch_chained(latent_q_rotate_kernel<elem_t>, dim3(n_tokens), dim3(128), 0, (cudaStream_t)stream, (const elem_t*)q, ld, H, dn,
-                 dr, R, positions, inv_freq, rot_dims, q_lat);
+                 dr, R, positions, inv_freq, rot_dims, rot_mult, q_lat);
   return check_launch("latent_q_rotate");
 }
 

@@ -3,6 +3,8 @@
 //
 //   1. route:   z = W_router x (float), s = sigmoid(z); the `top` experts with the largest z (the lower index wins a tie);
 //               per token the chosen experts and their scores s.  A (token, choice) is a "pair", numbered token * top + choice.
+//               With a correction per expert the choice goes by s + correction; a group of experts counts as much as its
+//               best expert or as the sum of its two best; the chosen scores may be divided by their sum.
 //   2. lists:   one block per expert counts all choices, makes its offset (and its offset in row tiles) and writes the
 //               pair numbers of its expert in rising order behind the offset.
 //   3. gate/up: for every expert the rows of its pairs, each row the token's input times the pair's score (rounded to T
@@ -25,6 +27,9 @@ ERB_DEFINE_LAST_ERROR(erb_last_error)
 #define ERB_MOE_GATED 1
 #define ERB_MOE_SINGLE 2
 #define ERB_ACT_RELU_SQUARED 1
+// what a group of experts counts as
+#define ERB_GROUP_BEST 0
+#define ERB_GROUP_TOP2_SUM 1
 
 namespace {
 
@@ -37,12 +42,14 @@ constexpr int kRouteTokens = 4;
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_router, int n_tokens, int width, int n_experts,
-                 int top, int* __restrict__ choice, float* __restrict__ score, int score_kind, int n_groups, int keep_groups) {
+                 int top, int* __restrict__ choice, float* __restrict__ score, int score_kind, int n_groups, int keep_groups,
+                 const float* __restrict__ correction, int group_kind, int normalise) {
   chain_wait();
   extern __shared__ float z_s[];                 // [kRouteTokens][n_experts padded to 4] logits, the same again for the
-  const int e_pad = (n_experts + 3) & ~3;        // groups' maxima, then [kRouteTokens][width]
+  const int e_pad = (n_experts + 3) & ~3;        // groups' values and for what the choice goes by, then [kRouteTokens][width]
   float* g_s = z_s + kRouteTokens * e_pad;
-  float* x_s = g_s + kRouteTokens * e_pad;
+  float* c_s = g_s + kRouteTokens * e_pad;
+  float* x_s = c_s + kRouteTokens * e_pad;
   const int t0 = blockIdx.x * kRouteTokens, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int n_here = min(kRouteTokens, n_tokens - t0);
 #pragma unroll
@@ -95,15 +102,25 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
     for (int e = lane; e < n_experts; e += 32) sum += expf(z[e] - z_top);
     denom = warp_sum(sum);
   }
-  // groups of neighbouring experts: a group's score is its largest logit (the scores rise with the logits); the experts
+  // What the choice goes by: the logits (the scores rise with them), or sigmoid scores plus correction.
+  float* cv = c_s + warp * e_pad;
+  const bool by_score = correction != nullptr || group_kind == ERB_GROUP_TOP2_SUM;
+  for (int e = lane; e < n_experts; e += 32)
+    cv[e] = by_score ? 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f) : z[e];
+  __syncwarp();
+  // groups of neighbouring experts: a group counts as much as its best expert or as the sum of its two best; the experts
   // of all but the `keep_groups` best groups are ruled out (the lower group wins a tie)
   if (n_groups > 1 && keep_groups < n_groups) {
     float* gm = g_s + warp * e_pad;
     const int per = n_experts / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
-      float mx = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) mx = fmaxf(mx, z[e]);
-      gm[g] = mx;
+      float mx = -INFINITY, second = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = cv[e];
+        second = fmaxf(second, fminf(mx, v));
+        mx = fmaxf(mx, v);
+      }
+      gm[g] = group_kind == ERB_GROUP_TOP2_SUM && per > 1 ? mx + second : mx;
     }
     __syncwarp();
     for (int c = 0; c < keep_groups; ++c) {
@@ -123,14 +140,15 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
       __syncwarp();
     }
     for (int e = lane; e < n_experts; e += 32)
-      if (gm[e / per] == gm[e / per]) z[e] = -INFINITY;       // not NaN: the group was not kept
+      if (gm[e / per] == gm[e / per]) cv[e] = -INFINITY;      // not NaN: the group was not kept
     __syncwarp();
   }
+  float total = 0.f;
   for (int c = 0; c < top; ++c) {
     float best = -INFINITY;
     int arg = 0x7fffffff;
     for (int e = lane; e < n_experts; e += 32) {
-      const float zv = z[e];
+      const float zv = cv[e];
       if (zv > best) { best = zv; arg = e; }     // rising e within a lane: the first maximum stays
     }
 #pragma unroll
@@ -139,13 +157,18 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
       const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
       if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
     }
+    if (arg >= n_experts) arg = c;                // (no expert compares: logits that are no numbers; any choice does)
     if (lane == 0) {
+      const float s = score_kind == ERB_SCORE_SOFTMAX ? expf(z[arg] - z_top) / denom : 1.f / (1.f + expf(-z[arg]));
       choice[(size_t)t * top + c] = arg;
-      score[(size_t)t * top + c] = score_kind == ERB_SCORE_SOFTMAX ? expf(best - z_top) / denom : 1.f / (1.f + expf(-best));
-      z[arg] = -INFINITY;
+      score[(size_t)t * top + c] = s;
+      cv[arg] = -INFINITY;
+      total += s;
     }
     __syncwarp();
   }
+  if (normalise && lane == 0)
+    for (int c = 0; c < top; ++c) score[(size_t)t * top + c] /= total + 1e-20f;
 }
 
 // One block per expert e builds the expert's part of the lists on its own: a histogram of all choices in shared memory
@@ -307,7 +330,8 @@ ERB_EXPORT int erb_moe_tile_rows() { return kTM; }
 
 ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n_tokens, int width, int n_experts, int top,
                              int* choice, float* score, int* counts, int* offsets, int* tiles, int* order, int tile_rows,
-                             int score_kind, int n_groups, int keep_groups, void* stream) {
+                             int score_kind, int n_groups, int keep_groups, const float* correction, int group_kind,
+                             int normalise, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   if (width <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || n_experts > 8192)
     return fail(ERB_ERR_ARG, "moe_route: %d of %d experts", top, n_experts);
@@ -315,16 +339,20 @@ ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n
       keep_groups < 1 || keep_groups > n_groups || top > keep_groups * (n_experts / n_groups))
     return fail(ERB_ERR_ARG, "moe_route: %d groups of which %d are kept cannot give %d of %d experts", n_groups, keep_groups, top,
                 n_experts);
+  if ((group_kind != ERB_GROUP_BEST && group_kind != ERB_GROUP_TOP2_SUM) ||
+      (score_kind != ERB_SCORE_SIGMOID && (correction || group_kind != ERB_GROUP_BEST)))
+    return fail(ERB_ERR_ARG, "moe_route: a correction and groups that count their two best go with sigmoid scores");
   cudaStream_t s = (cudaStream_t)stream;
   const int n_pairs = n_tokens * top;
-  const size_t route_smem = sizeof(float) * kRouteTokens * (2 * (size_t)((n_experts + 3) & ~3) + width);
+  const size_t route_smem = sizeof(float) * kRouteTokens * (3 * (size_t)((n_experts + 3) & ~3) + width);
   if (route_smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(moe_route_kernel<elem_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)route_smem);
     if (err != cudaSuccess) return fail(ERB_ERR_CUDA, "moe_route: %s", cudaGetErrorString(err));
   }
   if (route_smem > 200 * 1024) return fail(ERB_ERR_UNSUPPORTED, "moe_route: rows of %d entries with %d experts", width, n_experts);
   launch_chained(moe_route_kernel<elem_t>, dim3((n_tokens + kRouteTokens - 1) / kRouteTokens), dim3(kRouteThreads), route_smem, s,
-                 (const elem_t*)x, ld, w_router, n_tokens, width, n_experts, top, choice, score, score_kind, n_groups, keep_groups);
+                 (const elem_t*)x, ld, w_router, n_tokens, width, n_experts, top, choice, score, score_kind, n_groups, keep_groups,
+                 correction, group_kind, normalise);
   int rc = check_launch("moe_route");
   if (rc) return rc;
   launch_chained(moe_lists_kernel, dim3(n_experts), dim3(256), sizeof(int) * n_experts, s, (const int*)choice, n_pairs, n_experts,

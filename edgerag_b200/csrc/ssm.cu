@@ -66,6 +66,100 @@ conv_state_update_kernel(const T* __restrict__ proj, int ld, int off, int channe
   }
 }
 
+// Rows [q heads | k heads | v heads] of a fused product made ready for attention by a short causal convolution per channel:
+//   u = row + bias,   y_t = sum_j w[j] u_(t - (taps - 1 - j))   (u before the sequence's start: zero; no taps: y = u)
+// in float, from the portion's own rows and, before its first token, from the request's record of biased inputs (float
+// [slots][taps - 1][channels], oldest first).  q goes to rows of its own, k and v to the token's cache slot (page *
+// page_size + offset; negative: not written).  A thread owns four neighbouring channels of one token.  A sequence with one
+// token in the step gets its record moved on by the same thread (nobody else reads those channels of that record); the
+// records of longer portions are moved on by qkv_conv_state_kernel, after this kernel.
+// weight: float [taps][channels].
+template <typename T>
+__global__ void __launch_bounds__(128)
+qkv_conv_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, const float* __restrict__ weight, int taps,
+                float* __restrict__ conv_state, const int* __restrict__ seq_of_token, const int* __restrict__ seq_starts,
+                const int* __restrict__ state_slots, const int* __restrict__ slots, T* __restrict__ q_out,
+                T* __restrict__ k_pages, T* __restrict__ v_pages, int nq, int nkv, int D, int page_size) {
+  chain_wait();
+  const int t = blockIdx.x, ch = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  const int qw = nq * D, kw = nkv * D, channels = qw + 2 * kw;
+  if (ch >= channels) return;
+  float b[4] = {0.f, 0.f, 0.f, 0.f};
+  if (bias) load4(bias + ch, b);
+  auto input = [&](int row, float* u) {
+    Pack4<T>::load(proj + (size_t)row * ld + ch, u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) u[i] += b[i];
+  };
+  float y[4], u[4];
+  input(t, u);
+  if (taps <= 0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) y[i] = u[i];
+  } else {
+    const int seq = seq_of_token[t], start = seq_starts[seq], n = seq_starts[seq + 1] - start, i0 = t - start;
+    float* rec = conv_state ? conv_state + (size_t)state_slots[seq] * (taps - 1) * channels + ch : nullptr;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) y[i] = 0.f;
+    for (int j = 0; j < taps; ++j) {
+      const int r = i0 - (taps - 1 - j);               // index inside the portion of the input under tap j
+      float x[4], w[4];
+      if (j == taps - 1) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[i] = u[i];
+      } else if (r >= 0) {
+        input(start + r, x);
+      } else {
+        load4(rec + (size_t)(taps - 1 + r) * channels, x);
+      }
+      load4(weight + (size_t)j * channels + ch, w);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] = fmaf(w[i], x[i], y[i]);
+    }
+    if (n == 1 && taps > 1) {
+      for (int k = 0; k + 1 < taps - 1; ++k)
+        *reinterpret_cast<float4*>(rec + (size_t)k * channels) = *reinterpret_cast<const float4*>(rec + (size_t)(k + 1) * channels);
+      *reinterpret_cast<float4*>(rec + (size_t)(taps - 2) * channels) = make_float4(u[0], u[1], u[2], u[3]);
+    }
+  }
+  if (ch < qw) {
+    Pack4<T>::store(q_out + (size_t)t * qw + ch, y);
+    return;
+  }
+  const int slot = slots ? slots[t] : -1;
+  if (slot < 0) return;
+  const bool is_k = ch < qw + kw;
+  const int c = ch - qw - (is_k ? 0 : kw), head = c / D, e = c % D;
+  T* pages = is_k ? k_pages : v_pages;
+  Pack4<T>::store(pages + (((size_t)(slot / page_size) * nkv + head) * page_size + slot % page_size) * D + e, y);
+}
+
+// The records of the sequences with more than one token in the step: the last taps - 1 of (record, then the biased rows).
+template <typename T>
+__global__ void __launch_bounds__(128)
+qkv_conv_state_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, int taps, float* __restrict__ conv_state,
+                      const int* __restrict__ seq_starts, const int* __restrict__ state_slots, int first_seq, int channels) {
+  chain_wait();
+  const int seq = first_seq + blockIdx.x, ch = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  const int start = seq_starts[seq], n = seq_starts[seq + 1] - start, K = taps - 1;
+  if (n <= 1 || ch >= channels) return;
+  float* rec = conv_state + (size_t)state_slots[seq] * K * channels + ch;
+  float b[4] = {0.f, 0.f, 0.f, 0.f};
+  if (bias) load4(bias + ch, b);
+  for (int k = 0; k < K; ++k) {                        // rising k: entry k + n is read before it is written
+    const int src = k + n;
+    float x[4];
+    if (src < K) {
+      load4(rec + (size_t)src * channels, x);
+    } else {
+      Pack4<T>::load(proj + (size_t)(start + src - K) * ld + ch, x);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] += b[i];
+    }
+    *reinterpret_cast<float4*>(rec + (size_t)k * channels) = make_float4(x[0], x[1], x[2], x[3]);
+  }
+}
+
 constexpr int kScanChunk = 16;     // tokens staged in shared memory at a time
 
 // One block per (head, request); thread (l, p): column p of the state, rows l * NL .. l * NL + NL - 1, in
@@ -315,4 +409,26 @@ ERB_EXPORT int erb_gated_group_norm(const void* x, int x_is_float, int x_ld, con
     launch_chained(gated_group_norm_kernel<elem_t, false>, dim3(n_tokens, parts), dim3(256), 0, (cudaStream_t)stream, x, x_ld,
                    (const elem_t*)gate, gate_ld, weight, (elem_t*)out, out_ld, width, parts, eps);
   return check_launch("gated_group_norm");
+}
+
+// taps 0: no convolution; otherwise `weight` float [taps][channels] and, for taps > 1, the records `conv_state`.
+// Sequences before `first_portion` bring one token each.
+ERB_EXPORT int erb_qkv_conv(const void* proj, int ld, const float* bias, const float* weight, int taps, float* conv_state,
+                            const int* seq_of_token, const int* seq_starts, const int* state_slots, const int* slots, void* q_out,
+                            void* k_pages, void* v_pages, int n_tokens, int n_seqs, int first_portion, int nq, int nkv, int D,
+                            int page_size, void* stream) {
+  if (n_tokens <= 0) return ERB_OK;
+  const int channels = (nq + 2 * nkv) * D;
+  if (nq <= 0 || nkv <= 0 || D <= 0 || D % 4 || ld % 4 || ld < channels || taps < 0 || page_size <= 0 || (taps > 0 && !weight) ||
+      (taps > 1 && !conv_state) || (slots && (!k_pages || !v_pages)))
+    return fail(ERB_ERR_ARG, "qkv_conv: bad sizes (heads of %d, rows of %d) or missing tensors", D, ld);
+  const int y = (channels / 4 + 127) / 128;
+  launch_chained(qkv_conv_kernel<elem_t>, dim3(n_tokens, y), dim3(128), 0, (cudaStream_t)stream, (const elem_t*)proj, ld, bias, weight,
+                 taps, conv_state, seq_of_token, seq_starts, state_slots, slots, (elem_t*)q_out, (elem_t*)k_pages, (elem_t*)v_pages,
+                 nq, nkv, D, page_size);
+  int rc = check_launch("qkv_conv");
+  if (rc || taps <= 1 || n_seqs <= first_portion) return rc;
+  launch_chained(qkv_conv_state_kernel<elem_t>, dim3(n_seqs - first_portion, y), dim3(128), 0, (cudaStream_t)stream,
+                 (const elem_t*)proj, ld, bias, taps, conv_state, seq_starts, state_slots, first_portion, channels);
+  return check_launch("qkv_conv_state");
 }

@@ -239,6 +239,8 @@ class ModelRunner:
             n = e.n_tokens
             if n <= 0:
                 raise StepError(f"request {e.request_id!r}: an entry needs at least one token")
+            if e.embeds is not None and getattr(self.model, "needs_token_ids", False):
+                raise StepError(f"request {e.request_id!r}: this model looks at the tokens' ids, rows of embeddings cannot stand in for them")
             if e.embeds is not None and (e.embeds.dim() != 2 or e.embeds.shape[1] != hidden):
                 raise StepError(f"request {e.request_id!r}: embeds must be [n, {hidden}]")
             if e.tokens is not None and not all(0 <= int(t) < vocab for t in e.tokens):

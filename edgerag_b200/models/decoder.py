@@ -27,14 +27,14 @@ class DecoderModel:
         for layer in plan.layers:
             norm1 = build_part("norm", layer.norm1, dtype, device)
             mixer = build_part("mixer", layer.mixer, dtype, device)
-            if (layer.norm2 is None) != (layer.ffn is None):
-                raise ValueError(f"layer {layer.prefix!r}: a second norm and a feed-forward come together or not at all")
-            norm2 = build_part("norm", layer.norm2, dtype, device) if layer.norm2 is not None else None
-            ffn = build_part("ffn", layer.ffn, dtype, device) if layer.ffn is not None else None
             try:
                 block_cls = _REGISTRY["block"][layer.block.kind]
             except KeyError:
                 raise KeyError(f"no block arrangement named {layer.block.kind!r}") from None
+            if not getattr(block_cls, "single_norm", False) and (layer.norm2 is None) != (layer.ffn is None):
+                raise ValueError(f"layer {layer.prefix!r}: a second norm and a feed-forward come together or not at all")
+            norm2 = build_part("norm", layer.norm2, dtype, device) if layer.norm2 is not None else None
+            ffn = build_part("ffn", layer.ffn, dtype, device) if layer.ffn is not None else None
             block = block_cls(norm1=norm1, mixer=mixer, norm2=norm2, ffn=ffn, hidden=plan.hidden_size,
                               dtype=dtype, device=device, **layer.block.params)
             self.blocks.append(block)
@@ -57,6 +57,8 @@ class DecoderModel:
         #: every part may be captured in a CUDA graph (an attention mixer also vouches for its position encoding)
         self.graph_safe = all(part.graph_safe for _, part in self._owners) and all(
             getattr(getattr(b.mixer, "position", None), "graph_safe", True) for b in self.blocks)
+        #: some part looks at the tokens' ids: rows of embeddings cannot stand in for them
+        self.needs_token_ids = any(part.needs_token_ids for _, part in self._owners)
         self.logits_stride = -(-plan.vocab_size // 8) * 8  # rows of the logits buffer start 32-byte aligned
 
     # --- cache needs ------------------------------------------------------------------------------

@@ -55,19 +55,19 @@ _SIGNATURES = {
     "erb_linear_tc_rope": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "erb_attention_rows": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
+                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "erb_attention_decode": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                              c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_float, c_void_p],
+                             c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "erb_attention_prefill_tc": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
-                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
+                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "erb_attention_decode_bulk": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                   c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                                  c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "erb_attention_decode_gqa": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_float, c_void_p, c_void_p, c_int, c_int, c_void_p],
+                                 c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "erb_glu_bounded": [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "erb_add_layernorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float,
                           c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -79,8 +79,8 @@ _SIGNATURES = {
     "erb_linear_batched": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                            c_longlong, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p],
     "erb_latent_store": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int,
-                         c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
-    "erb_latent_q_rotate": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                         c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "erb_latent_q_rotate": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p,
                             c_void_p],
     "erb_latent_attention": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                              c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -107,6 +107,13 @@ _SIGNATURES = {
                              c_float, c_void_p],
     "erb_rms_between": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p,
                         c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+    "erb_sigmoid_gate": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+    "erb_qkv_conv": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                     c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "erb_sum_updates": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_longlong, c_void_p],
+    "erb_side_gate": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+    "erb_depth_mix": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_float, c_void_p, c_longlong, c_int, c_void_p, c_int,
+                      c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "erb_bias_rows": [c_void_p, c_void_p, c_int, c_int, c_void_p],
     "erb_qkv_whole_norm": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
                            c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -115,7 +122,7 @@ _SIGNATURES = {
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "erb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "erb_moe_route": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     "erb_moe_tc_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "erb_moe_tc_gate_up": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                            c_void_p, c_void_p],
@@ -263,9 +270,9 @@ def residual_add(hidden: torch.Tensor, delta: torch.Tensor, dtype: torch.dtype |
 
 
 def add_layernorm(hidden: torch.Tensor, weight: torch.Tensor | None, bias: torch.Tensor | None, out: torch.Tensor | None,
-                  eps: float, delta: torch.Tensor | None = None, post: tuple[torch.Tensor, torch.Tensor, float] | None = None,
+                  eps: float, delta: torch.Tensor | None = None, post: tuple[torch.Tensor, torch.Tensor | None, float] | None = None,
                   rows: torch.Tensor | None = None, write_back: bool = True) -> None:
-    """The residual add between two layer norms (weight and bias, statistics in float): with ``post = (w, b, eps)``
+    """The residual add between two layer norms (weight and an optional bias, statistics in float): with ``post = (w, b, eps)``
     the update is normed first, ``d = LN(delta; w, b)`` kept in float; ``hidden += d`` in place when ``write_back``;
     ``out = LN(hidden (+ d); weight, bias)`` rounded once, or the plain cast of the sum where ``weight`` is None, or
     nothing where ``out`` is None.  ``delta``: rows of the element type or float32 partial sums ``[parts, rows,
@@ -280,14 +287,14 @@ def add_layernorm(hidden: torch.Tensor, weight: torch.Tensor | None, bias: torch
     _need(delta, "delta", torch.float32 if in_parts else elem)
     if delta is not None and delta.shape[-2:] != hidden.shape:
         raise KernelError("add_layernorm: delta and hidden disagree")
-    if (weight is None) != (bias is None) or (weight is not None and (weight.numel() != h or bias.numel() != h)):
-        raise KernelError("add_layernorm: weight and bias come together and have the row's width")
+    if (bias is not None and weight is None) or any(v is not None and v.numel() != h for v in (weight, bias)):
+        raise KernelError("add_layernorm: weight and bias have the row's width, a bias comes with a weight")
     pw = pb = None
     peps = 0.0
     if post is not None:
         pw, pb, peps = post
         _need(pw, "post weight", torch.float32); _need(pb, "post bias", torch.float32)
-        if delta is None or pw.numel() != h or pb.numel() != h:
+        if delta is None or pw.numel() != h or (pb is not None and pb.numel() != h):
             raise KernelError("add_layernorm: a norm of the update needs the update and vectors of the row's width")
     if out is not None:
         n = out.shape[0]
@@ -546,6 +553,86 @@ def scale_rows(x: torch.Tensor, scale: float, dtype: torch.dtype) -> None:
     n, width = x.shape
     _call(_fn("elementwise", _ELEM[dtype], "erb_scale_rows"), x.data_ptr(), n, width, x.stride(0) if n > 1 else width, float(scale),
           _stream())
+
+
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> None:
+    """x[t, i] *= sigmoid(gate[t, i]) in place, in float, rounded once (both may be row-strided views)."""
+    _need(x, "x", contiguous=False); _need(gate, "gate", x.dtype, contiguous=False)
+    n, width = x.shape
+    if gate.shape != x.shape or x.stride(1) != 1 or gate.stride(1) != 1:
+        raise KernelError("sigmoid_gate: shapes or strides disagree")
+    _call(_fn("elementwise", _elem(x), "erb_sigmoid_gate"), x.data_ptr(), x.stride(0) if n > 1 else width, gate.data_ptr(),
+          gate.stride(0) if n > 1 else width, n, width, _stream())
+
+
+# --- the stream between layers -----------------------------------------------------------------
+
+def _update(u: torch.Tensor | None, hidden: torch.Tensor, elem: torch.dtype, who: str) -> tuple[int | None, int, int]:
+    """(pointer, parts, stride between parts) of an update: rows of the element type, or float partial sums ``[parts, rows, width]``."""
+    if u is None:
+        return None, 0, 0
+    parts = u.dim() == 3
+    _need(u, "update", torch.float32 if parts else elem)
+    if u.shape[-2:] != hidden.shape:
+        raise KernelError(f"{who}: an update and the stream disagree")
+    return u.data_ptr(), (u.shape[0] if parts else 0), (u.stride(0) if parts else 0)
+
+
+def sum_updates(hidden: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, dtype: torch.dtype,
+                out: torch.Tensor | None = None) -> None:
+    """hidden += a + b (``b`` may be None) in float; ``out`` (if given) receives the sum rounded to the element type
+    ``dtype``.  ``a`` and ``b``: rows of the element type or float partial sums ``[parts, rows, width]``, added in order."""
+    _need(hidden, "hidden", torch.float32); _need(out, "out", dtype)
+    if out is not None and out.shape != hidden.shape:
+        raise KernelError("sum_updates: out and hidden disagree")
+    pa, na, sa = _update(a, hidden, dtype, "sum_updates")
+    pb, nb, sb = _update(b, hidden, dtype, "sum_updates")
+    _call(_fn("depth", _ELEM[dtype], "erb_sum_updates"), hidden.data_ptr(), pa, na, sa, pb, nb, sb, _ptr(out), hidden.numel(), _stream())
+
+
+def side_gate(g: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, offset: int, dim: int, out: torch.Tensor) -> None:
+    """out[t, i] = gelu_tanh(g[t, i]) * table[ids[t], offset + i] for i < ``dim``, in float, rounded once; the columns of
+    ``out`` from ``dim`` on receive zeros."""
+    _need(g, "g", contiguous=False); _need(table, "table", g.dtype); _need(ids, "ids", torch.int32); _need(out, "out", g.dtype)
+    n, ld_out = out.shape
+    if g.shape[0] != n or g.shape[1] < dim or dim > ld_out or g.stride(1) != 1 or ids.numel() < n or not 0 <= offset <= table.shape[1] - dim:
+        raise KernelError("side_gate: shapes disagree")
+    _call(_fn("depth", _elem(g), "erb_side_gate"), g.data_ptr(), g.stride(0) if n > 1 else g.shape[1], table.data_ptr(), table.shape[1],
+          table.shape[0], ids.data_ptr(), int(offset), int(dim), out.data_ptr(), ld_out, n, _stream())
+
+
+DEPTH_OUT = {"cast": 0, "layernorm": 1, "rmsnorm": 2}
+
+
+def depth_mix(hidden: torch.Tensor, history: torch.Tensor, layer: int, mix: torch.Tensor, dtype: torch.dtype, *,
+              delta: torch.Tensor | None = None, post: tuple[torch.Tensor, float] | None = None, out: torch.Tensor | None = None,
+              out_kind: str = "cast", weight: torch.Tensor | None = None, bias: torch.Tensor | None = None, eps: float = 0.0,
+              rows: torch.Tensor | None = None, write_back: bool = True) -> None:
+    """With ``history`` float ``[layers + 1, rows, width]`` holding the results 0 .. layer (0: the embedding's):
+    ``x = hidden + delta`` (``post = (w, eps)``: the update is brought to unit RMS times ``w`` first); ``history[layer + 1]
+    = x``; ``hidden = sum_j mix[j] history[j]`` over all ``layer + 2`` of them; ``out`` = the row normed as ``out_kind``
+    says (``layernorm`` / ``rmsnorm`` with ``weight``, ``bias`` and ``eps``; ``cast``: rounded).  ``rows`` picks the rows
+    that ``out`` gets; hidden and history are then left alone, as with ``write_back`` False."""
+    _need(hidden, "hidden", torch.float32); _need(history, "history", torch.float32); _need(mix, "mix", torch.float32)
+    _need(out, "out", dtype, contiguous=False); _need(rows, "rows", torch.int32)
+    n, h = hidden.shape
+    if history.dim() != 3 or history.shape[1:] != hidden.shape or not 0 <= layer < history.shape[0] - 1 or mix.numel() != layer + 2:
+        raise KernelError("depth_mix: history, mix and the layer disagree")
+    for name, v in (("weight", weight), ("bias", bias), ("post weight", post[0] if post else None)):
+        _need(v, name, torch.float32)
+        if v is not None and v.numel() != h:
+            raise KernelError("depth_mix: vectors must have the row's width")
+    if out is not None and (out.shape[1] != h or out.stride(1) != 1 or (rows is None and out.shape[0] != n) or
+                            (rows is not None and rows.numel() < out.shape[0])):
+        raise KernelError("depth_mix: out must be [rows, width] with unit inner stride")
+    if rows is not None and out is None:
+        raise KernelError("depth_mix: a selection of rows needs an output")
+    n_rows = n if out is None else out.shape[0]
+    pd, nd, sd = _update(delta, hidden, dtype, "depth_mix")
+    _call(_fn("depth", _ELEM[dtype], "erb_depth_mix"), hidden.data_ptr(), pd, nd, sd, _ptr(post[0]) if post else None,
+          float(post[1]) if post else 0.0, history.data_ptr(), history.stride(0), layer + 1, mix.data_ptr(), DEPTH_OUT[out_kind],
+          _ptr(weight), _ptr(bias), float(eps), _ptr(out), h if out is None else (out.stride(0) if n_rows > 1 else max(h, out.stride(0))),
+          _ptr(rows), n_rows, h, int(write_back and rows is None), _stream())
 
 
 # --- matrix products -------------------------------------------------------------------------
@@ -859,11 +946,11 @@ def linear_batched(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> 
 def latent_store(proj: torch.Tensor, positions: torch.Tensor, eps: float, *, off_kv: int = -1, rank: int = 0, rot_dim: int = 0,
                  kv_weight: torch.Tensor | None = None, inv_freq: torch.Tensor | None = None, rot_dims: int = 0,
                  slots: torch.Tensor | None = None, pages: torch.Tensor | None = None, off_q: int = 0, q_rank: int = 0,
-                 q_weight: torch.Tensor | None = None, q_latent: torch.Tensor | None = None) -> None:
+                 q_weight: torch.Tensor | None = None, q_latent: torch.Tensor | None = None, rot_mult: float = 1.0) -> None:
     """From each token's row of a fused projection: (``off_kv >= 0``) the cache row ``[unit_rms(row[off_kv :
     off_kv + rank]) * kv_weight | pairs of the next rot_dim entries turned by the position]`` written to slot
     ``slots[t]`` of ``pages`` (``[n_pages, 1, page_size, rank + rot_dim]``); (``q_rank > 0``) ``q_latent[t] =
-    unit_rms(row[off_q : off_q + q_rank]) * q_weight``."""
+    unit_rms(row[off_q : off_q + q_rank]) * q_weight``.  ``rot_mult`` multiplies cosines and sines."""
     _need(proj, "proj", contiguous=False); _need(positions, "positions", torch.int32)
     _need(kv_weight, "kv_weight", torch.float32); _need(q_weight, "q_weight", torch.float32)
     _need(inv_freq, "inv_freq", torch.float32); _need(slots, "slots", torch.int32)
@@ -883,20 +970,22 @@ def latent_store(proj: torch.Tensor, positions: torch.Tensor, eps: float, *, off
         raise KernelError("latent_store: the query latent lies outside the row or its target has another shape")
     _call(_fn("latent_attention", _elem(proj), "erb_latent_store"), proj.data_ptr(), n, proj.stride(0) if n > 1 else proj.shape[1],
           int(off_kv), int(rank), int(rot_dim), _ptr(kv_weight), float(eps), positions.data_ptr(), _ptr(inv_freq), int(rot_dims),
-          _ptr(slots), _ptr(pages), int(off_q), int(q_rank), _ptr(q_weight), _ptr(q_latent), _stream())
+          float(rot_mult), _ptr(slots), _ptr(pages), int(off_q), int(q_rank), _ptr(q_weight), _ptr(q_latent), _stream())
 
 
 def latent_q_rotate(q: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor | None, n_heads: int, dim: int,
-                    rot_dim: int, rank: int, rot_dims: int, q_lat: torch.Tensor) -> None:
+                    rot_dim: int, rank: int, rot_dims: int, q_lat: torch.Tensor, rot_mult: float = 1.0) -> None:
     """q rows hold per head ``dim`` plain then ``rot_dim`` rotated entries; the latter go, pairs turned by
-    the position, to ``q_lat[t, head, rank:]`` (float ``[tokens, heads, rank + rot_dim]``)."""
+    the position, to ``q_lat[t, head, rank:]`` (float ``[tokens, heads, rank + rot_dim]``); ``rot_mult`` multiplies
+    cosines and sines."""
     _need(q, "q", contiguous=False); _need(positions, "positions", torch.int32); _need(inv_freq, "inv_freq", torch.float32)
     _need(q_lat, "q_lat", torch.float32)
     n = q.shape[0]
     if q.stride(1) != 1 or q.shape[1] < n_heads * (dim + rot_dim) or q_lat.shape != (n, n_heads, rank + rot_dim):
         raise KernelError("latent_q_rotate: shapes disagree")
     _call(_fn("latent_attention", _elem(q), "erb_latent_q_rotate"), q.data_ptr(), n, q.stride(0) if n > 1 else q.shape[1],
-          n_heads, dim, rot_dim, rank, positions.data_ptr(), _ptr(inv_freq), int(rot_dims), q_lat.data_ptr(), _stream())
+          n_heads, dim, rot_dim, rank, positions.data_ptr(), _ptr(inv_freq), int(rot_dims),
+          float(rot_mult), q_lat.data_ptr(), _stream())
 
 
 def latent_scratch_floats(n_tokens: int, n_heads: int, rank: int, n_splits: int) -> int:
@@ -1151,6 +1240,38 @@ def conv_silu(proj: torch.Tensor, off: int, weight: torch.Tensor, bias: torch.Te
           state_slots.data_ptr(), out.data_ptr(), _stream())
 
 
+def qkv_conv(proj: torch.Tensor, q_out: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int, *, taps: int,
+             bias: torch.Tensor | None, weight: torch.Tensor | None, conv_state: torch.Tensor | None, seq_of_token: torch.Tensor,
+             seq_starts: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, first_portion: int, slots: torch.Tensor | None,
+             k_pages: torch.Tensor | None, v_pages: torch.Tensor | None, page_size: int) -> None:
+    """Rows ``[q heads | k heads | v heads]`` of ``proj`` made ready for attention: ``u = row + bias``, then the causal
+    convolution ``y_t = sum_j weight[j] u_(t - taps + 1 + j)`` per channel (``weight`` float ``[taps, channels]``; ``taps``
+    0: ``y = u``), in float.  Inputs before a portion come from the request's record in ``conv_state`` (float ``[slots,
+    taps - 1, channels]``, biased, oldest first), which is moved on to the step's last ``taps - 1`` inputs.  q goes to
+    ``q_out``, k and v to the tokens' cache slots.  Sequences before ``first_portion`` bring one token each."""
+    _need(proj, "proj", contiguous=False); _need(q_out, "q_out", proj.dtype); _need(bias, "bias", torch.float32)
+    _need(weight, "weight", torch.float32); _need(conv_state, "conv_state", torch.float32); _need(slots, "slots", torch.int32)
+    _need(k_pages, "k_pages", proj.dtype); _need(v_pages, "v_pages", proj.dtype)
+    for name, t in (("seq_of_token", seq_of_token), ("seq_starts", seq_starts), ("state_slots", state_slots)):
+        _need(t, name, torch.int32)
+    n = proj.shape[0]
+    channels = (n_q_heads + 2 * n_kv_heads) * head_dim
+    if proj.stride(1) != 1 or proj.shape[1] < channels or q_out.shape != (n, n_q_heads * head_dim):
+        raise KernelError("qkv_conv: proj or q_out disagree with the heads")
+    if (bias is not None and bias.numel() != channels) or (taps > 0 and (weight is None or weight.shape != (taps, channels))) or \
+            (taps > 1 and (conv_state is None or tuple(conv_state.shape[1:]) != (taps - 1, channels))):
+        raise KernelError("qkv_conv: bias, weight or state have the wrong size")
+    if slots is not None and (k_pages is None or v_pages is None or tuple(k_pages.shape[1:]) != (n_kv_heads, page_size, head_dim)
+                              or v_pages.shape != k_pages.shape or slots.numel() < n):
+        raise KernelError("qkv_conv: pages or slots disagree with the heads")
+    fn = _fn("ssm", _elem(proj), "erb_qkv_conv")
+    fn._erb_own = 2 if taps > 1 and n_seqs > first_portion else 1
+    _call(fn, proj.data_ptr(), proj.stride(0) if n > 1 else proj.shape[1], _ptr(bias), _ptr(weight), int(taps),
+          _ptr(conv_state) if taps > 1 else None, seq_of_token.data_ptr(), seq_starts.data_ptr(), state_slots.data_ptr(), _ptr(slots),
+          q_out.data_ptr(), _ptr(k_pages), _ptr(v_pages), n, int(n_seqs), int(first_portion), n_q_heads, n_kv_heads, head_dim,
+          int(page_size), _stream())
+
+
 def conv_state_update(proj: torch.Tensor, off: int, conv_state: torch.Tensor, n_seqs: int, seq_starts: torch.Tensor,
                       state_slots: torch.Tensor) -> None:
     """Every request's record in ``conv_state`` becomes the last ``taps - 1`` inputs of (record, then the step's rows)."""
@@ -1282,10 +1403,12 @@ def _moe_lists(lists: torch.Tensor, n_tokens: int, n_experts: int, top: int):
 
 
 MOE_SCORES = {"sigmoid": 0, "softmax": 1}
+MOE_GROUP_SCORES = {"best": 0, "top2_sum": 1}
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Tensor, score: torch.Tensor,
-              tile_rows: int = 0, scores: str = "sigmoid", groups: tuple[int, int] | None = None) -> None:
+              tile_rows: int = 0, scores: str = "sigmoid", groups: tuple[int, int] | None = None,
+              correction: torch.Tensor | None = None, group_score: str = "best", normalise: bool = False) -> None:
     """Route every row of ``x`` (element type, row-strided view allowed): logits ``w_router x`` in float (``w_router``
     float ``[experts, width]``), the ``top`` largest chosen (the lower index wins a tie), ``score`` float ``[tokens *
     top]`` their sigmoids; ``lists`` (int32, ``moe_lists_ints`` entries) receives the choices and, per expert, the list
@@ -1293,7 +1416,15 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     that the lists' tile offsets count (0: those of ``moe_gate_up`` and ``moe_down``; ``moe_tc_tile_rows`` for the
     tensor-core products).  ``scores``: ``sigmoid`` of the logit, or ``softmax`` over all experts' logits.  ``groups =
     (count, keep)``: the experts form ``count`` equal groups of neighbours, a group counts as much as its best expert, and
-    only experts of the ``keep`` best groups can be chosen."""
+    only experts of the ``keep`` best groups can be chosen.  With ``correction`` (float ``[experts]``, sigmoid scores) the
+    choice goes by score + correction, while ``score`` stays without it; ``group_score = "top2_sum"``: a group counts as
+    much as the sum of its two best experts (in what the choice goes by); ``normalise``: the chosen scores are divided by
+    their sum (+ 1e-20)."""
+    _need(correction, "correction", torch.float32)
+    if correction is not None and correction.numel() != w_router.shape[0]:
+        raise KernelError("moe_route: one correction per expert")
+    if group_score not in MOE_GROUP_SCORES:
+        raise KernelError(f"moe_route: unknown group score {group_score!r}; known: {sorted(MOE_GROUP_SCORES)}")
     _need(x, "x", contiguous=False); _need(w_router, "w_router", torch.float32); _need(lists, "lists", torch.int32)
     n_groups, keep = groups if groups else (1, 1)
     _need(score, "score", torch.float32)
@@ -1304,7 +1435,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     choice, order, counts, offsets, tiles = _moe_lists(lists, n, n_experts, top)
     _call(_fn("moe", _elem(x), "erb_moe_route"), x.data_ptr(), x.stride(0) if n > 1 else width, w_router.data_ptr(), n, width,
           n_experts, int(top), choice.data_ptr(), score.data_ptr(), counts.data_ptr(), offsets.data_ptr(), tiles.data_ptr(),
-          order.data_ptr(), int(tile_rows), MOE_SCORES[scores], int(n_groups), int(keep), _stream())
+          order.data_ptr(), int(tile_rows), MOE_SCORES[scores], int(n_groups), int(keep), _ptr(correction),
+          MOE_GROUP_SCORES[group_score], int(bool(normalise)), _stream())
 
 
 def moe_tc_supported(dtype: torch.dtype, width: int, ff: int) -> bool:
@@ -1374,10 +1506,10 @@ def moe_tc_down(act: torch.Tensor, w_down: torch.Tensor, lists: torch.Tensor, to
           _stream())
 
 
-def moe_gate_up(x: torch.Tensor, w_gate_up: torch.Tensor, lists: torch.Tensor, score: torch.Tensor, top: int,
+def moe_gate_up(x: torch.Tensor, w_gate_up: torch.Tensor, lists: torch.Tensor, score: torch.Tensor | None, top: int,
                 act: torch.Tensor) -> None:
-    """act[list row] = silu(W_gate r) * (W_up r) with ``r = round(score * x[token])`` for every (token, choice) pair,
-    in the order of the experts' lists.  ``w_gate_up`` ``[experts, 2 * ff, width]`` (gate rows, then up rows)."""
+    """act[list row] = silu(W_gate r) * (W_up r) with ``r = round(score * x[token])`` for every (token, choice) pair
+    (``score`` None: ``r = x[token]``), in the order of the experts' lists.  ``w_gate_up`` ``[experts, 2 * ff, width]`` (gate rows, then up rows)."""
     _need(x, "x", contiguous=False); _need(w_gate_up, "w_gate_up", x.dtype); _need(act, "act", x.dtype)
     n, width = x.shape
     n_experts, two_ff, k = w_gate_up.shape
@@ -1385,7 +1517,7 @@ def moe_gate_up(x: torch.Tensor, w_gate_up: torch.Tensor, lists: torch.Tensor, s
         raise KernelError("moe_gate_up: shapes disagree")
     _, order, _, offsets, tiles = _moe_lists(lists, n, n_experts, top)
     _call(_fn("moe", _elem(x), "erb_moe_product"), x.data_ptr(), x.stride(0) if n > 1 else width, w_gate_up.data_ptr(),
-          offsets.data_ptr(), tiles.data_ptr(), order.data_ptr(), score.data_ptr(), n_experts, int(top), n, two_ff // 2, width,
+          offsets.data_ptr(), tiles.data_ptr(), order.data_ptr(), _ptr(score), n_experts, int(top), n, two_ff // 2, width,
           1, act.data_ptr(), None, _stream())
 
 
@@ -1433,13 +1565,22 @@ def mask_reach(window: int, chunk: int) -> int:
     return int(window) if window else -int(chunk)
 
 
+def _penalty(penalty: torch.Tensor | None, n_q_heads: int) -> int | None:
+    _need(penalty, "penalty", torch.float32)
+    if penalty is not None and tuple(penalty.shape) != (2, n_q_heads):
+        raise KernelError("attention: a penalty is [2, query heads]")
+    return _ptr(penalty)
+
+
 def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_tables: torch.Tensor,
                    seq_of_token: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
-                   scale: float, window: int = 0, keep_first: int = 0, chunk: int = 0) -> None:
+                   scale: float, window: int = 0, keep_first: int = 0, chunk: int = 0,
+                   penalty: torch.Tensor | None = None) -> None:
     """Causal attention of every token over its sequence's pages (general kernel, any portion sizes).
     ``window`` > 0: a query sees the last ``window`` keys (its own included) and the first ``keep_first`` of the sequence.
     ``chunk`` > 0 (instead of a window): a query sees the earlier keys of its own run of ``chunk`` positions, runs
-    counted from position 0 of the sequence.
+    counted from position 0 of the sequence.  ``penalty`` float ``[2, n_q_heads]`` (``r1``, then ``r2`` of every query
+    head): the scaled score of a key ``d`` positions back is lowered by ``r1 * ln(1 + r2 * d)``.
 
     ``q``: ``[tokens, >= n_q_heads * D]`` view with unit inner stride (the q part of a qkv buffer);
     ``out``: ``[tokens, n_q_heads * D]``; pages ``[n_pages, n_kv_heads, page_size, D]``;
@@ -1455,7 +1596,7 @@ def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     _call(_fn("attention", _elem(q), "erb_attention_rows"), q.data_ptr(), q.stride(0), k_pages.data_ptr(),
           v_pages.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], seq_of_token.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), n, n_q_heads, nkv, d, page_size, mask_reach(window, chunk),
-          int(keep_first), float(scale), _stream())
+          int(keep_first), float(scale), _penalty(penalty, n_q_heads), _stream())
 
 
 _sm_counts: dict[int, int] = {}
@@ -1573,10 +1714,11 @@ def decode_scratch_floats(n_seqs: int, n_q_heads: int, head_dim: int, max_splits
 def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_tables: torch.Tensor,
                      token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                      scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
-                     window: int = 0, split_keys: int = DECODE_SPLIT_KEYS, keep_first: int = 0, chunk: int = 0) -> None:
+                     window: int = 0, split_keys: int = DECODE_SPLIT_KEYS, keep_first: int = 0, chunk: int = 0,
+                     penalty: torch.Tensor | None = None) -> None:
     """Attention of one new token per sequence, keys cut into splits of ``split_keys`` (split-KV).
     With a window the first ``keep_first`` keys stay visible; the first split of the window takes them along.
-    ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``.
+    ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``; ``penalty``: as there.
 
     ``token_of_seq`` int32 ``[sequences]`` gives each sequence's row in q/out/positions.  Scratch:
     ``part_acc`` float ``[sequences * heads * max_splits * D]``, ``part_ml`` twice
@@ -1597,7 +1739,7 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
           v_pages.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], token_of_seq.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(),
           max_splits, n_seqs, n_q_heads, nkv, d, page_size, mask_reach(window, chunk), int(keep_first), int(split_keys),
-          float(scale), _stream())
+          float(scale), _penalty(penalty, n_q_heads), _stream())
 
 
 def decode_bulk_supported(dtype: torch.dtype, head_dim: int, window: int, n_q_heads: int, n_kv_heads: int,
@@ -1635,7 +1777,7 @@ def attention_decode_bulk(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
                           token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                           scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
                           status: torch.Tensor, split_keys: int = DECODE_SPLIT_KEYS, head_group: int = 0, window: int = 0,
-                          keep_first: int = 0, chunk: int = 0) -> None:
+                          keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
     """``attention_decode`` for bfloat16 with keys and values streamed by bulk asynchronous copies.
     ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``.
     ``window`` > 0: the last ``window`` keys and the first ``keep_first``; the splits are counted from the one
@@ -1659,7 +1801,8 @@ def attention_decode_bulk(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
           v_pages.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], token_of_seq.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(), max_splits,
           n_seqs, n_q_heads, nkv, d, page_size, int(split_keys), float(scale), status.data_ptr(),
-          split_counters(q.device, n_seqs * nkv).data_ptr(), int(head_group), mask_reach(window, chunk), int(keep_first), _stream())
+          split_counters(q.device, n_seqs * nkv).data_ptr(), int(head_group), mask_reach(window, chunk), int(keep_first),
+          _penalty(penalty, n_q_heads), _stream())
 
 
 @functools.lru_cache(maxsize=4096)
@@ -1677,7 +1820,7 @@ def attention_decode_gqa(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                          scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
                          status: torch.Tensor, split_keys: int = DECODE_SPLIT_KEYS, window: int = 0, keep_first: int = 0,
-                         chunk: int = 0) -> None:
+                         chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
     """``attention_decode`` for several query heads per kv head on tensor cores (``window`` and ``keep_first`` as in
     ``attention_decode_bulk``): the query heads of a
     kv head are the rows of one matrix tile, pages arrive by TMA tensor copies."""
@@ -1697,7 +1840,8 @@ def attention_decode_gqa(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
           v_pages.data_ptr(), n_pages, block_tables.data_ptr(), block_tables.shape[1], token_of_seq.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(), max_splits,
           n_seqs, n_q_heads, nkv, d, page_size, int(split_keys), float(scale), status.data_ptr(),
-          split_counters(q.device, n_seqs * nkv).data_ptr(), mask_reach(window, chunk), int(keep_first), _stream())
+          split_counters(q.device, n_seqs * nkv).data_ptr(), mask_reach(window, chunk), int(keep_first),
+          _penalty(penalty, n_q_heads), _stream())
 
 
 #: query rows of one (sequence, head) that a block of the tensor-core prefill kernel takes
@@ -1738,7 +1882,7 @@ def attention_prefill_tc(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
                          seq_starts: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_blocks: int,
                          n_q_heads: int, scale: float, status: torch.Tensor, key_splits: int = 1, first_row: int = 0,
                          part_o: torch.Tensor | None = None, part_ml: torch.Tensor | None = None, window: int = 0,
-                         keep_first: int = 0, chunk: int = 0) -> None:
+                         keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
     """Causal attention of prompt portions on tcgen05 tensor cores (bfloat16, head_dim 64).  ``window`` > 0: a
     query sees the last ``window`` keys (its own included) and the first ``keep_first`` of its sequence.
     ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``.
@@ -1768,7 +1912,7 @@ def attention_prefill_tc(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
           v_pages.data_ptr(), n_pages, block_tables.data_ptr(), block_tables.shape[1], seq_starts.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), n_seqs, int(n_blocks), n_q_heads, nkv, d, page_size,
           float(scale), status.data_ptr(), int(key_splits), int(first_row), qkv.shape[0] - int(first_row), _ptr(part_o), _ptr(part_ml),
-          mask_reach(window, chunk), int(keep_first), _stream())
+          mask_reach(window, chunk), int(keep_first), _penalty(penalty, n_q_heads), _stream())
     if key_splits > 1:
         launch_counts["own"] += 1          # the merge of the ranges
 

@@ -35,6 +35,7 @@ LIBRARIES: dict[str, tuple[str, tuple[str, ...], bool]] = {
     "diff_attention": ("diff_attention.cu", (), True),
     "ssm": ("ssm.cu", (), True),
     "delta": ("delta.cu", (), True),
+    "depth": ("depth.cu", (), True),
     "moe": ("moe.cu", (), True),
     "moe_tc": ("moe_tc.cu", ("-lcuda",), False),
     "attention_tc": ("attention_tc.cu", ("-lcuda",), False),

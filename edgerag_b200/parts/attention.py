@@ -20,7 +20,13 @@ projections (``all_bias``; the output's rides with the update to whoever adds it
 query projection and whole key projection with a weight per entry (``whole_norm_eps``), values of another size than
 queries and keys (``v_dim``), and a mask of chunks (``chunk``: a query sees the earlier keys of its own run of ``chunk``
 positions, runs counted from the sequence's start; no key is ever out of every later query's sight, so the cache
-keeps all pages).  Heads whose sizes differ or are no multiple of 8 are stored padded with zeros to one size ``D``:
+keeps all pages).  A third (``kernels.qkv_conv``): biases on q, k and v only (``qkv_bias``) and a short causal convolution over time on every
+channel of q, k and v, directly after the projection (``conv`` taps, tensors ``<name>.conv`` of shape ``[channels, taps]``);
+the last ``conv - 1`` biased inputs of every channel live in a state record.  With ``penalty`` (the names of two tensors
+``[heads]``, ``r1`` and ``r2``) the scaled score of a key ``d`` positions back is lowered by ``r1 ln(1 + r2 d)``; every
+attention kernel takes it.
+
+Heads whose sizes differ or are no multiple of 8 are stored padded with zeros to one size ``D``:
 scores and outputs are unchanged, and the norm's mean divides by the true count.
 
 Single new tokens go through the split-KV decode kernels, portions of prompts through the tensor-core
@@ -32,7 +38,7 @@ from __future__ import annotations
 
 import torch
 
-from ..cache.manager import KVGroupSpec
+from ..cache.manager import KVGroupSpec, StateSpec
 from ..ops import kernels
 from .base import LayerCall, Mixer, PartSpec, WeightSpec, build_part, register_part
 
@@ -45,7 +51,8 @@ class Attention(Mixer):
                  dtype: torch.dtype, device: torch.device, window: int = 0, own_kv: bool = True,
                  scale: float | None = None, keep_first: int = 0, qk_bias: bool = False, qk_norm_eps: float | None = None,
                  values_are_keys: bool = False, names: dict[str, str] | None = None, chunk: int = 0, v_dim: int | None = None,
-                 all_bias: bool = False, whole_norm_eps: float | None = None) -> None:
+                 all_bias: bool = False, whole_norm_eps: float | None = None, qkv_bias: bool = False, conv: int = 0,
+                 penalty: tuple[str, str] | None = None) -> None:
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads are not divisible by {n_kv_heads} kv heads")
         self.chunk = int(chunk or 0)
@@ -57,7 +64,13 @@ class Attention(Mixer):
         widest = max(self.qk_dim, self.v_dim)
         padded = -(-widest // 8) * 8 if widest <= 128 else -(-widest // 16) * 16
         #: the second family's kernel handles padded heads, a norm over the projection and the four biases
-        self.whole = self.all_bias or whole_norm_eps is not None or padded != self.qk_dim or self.v_dim != self.qk_dim
+        self.qkv_bias, self.taps = bool(qkv_bias), int(conv or 0)
+        self.conv_form = self.qkv_bias or self.taps > 0
+        self.whole = self.conv_form or self.all_bias or whole_norm_eps is not None or padded != self.qk_dim or self.v_dim != self.qk_dim
+        if self.taps < 0 or (self.conv_form and (self.all_bias or whole_norm_eps is not None or not own_kv or position.kind != "none")):
+            raise ValueError("attention: a convolution or biases on q, k and v exclude a norm, another layer's keys and a position encoding")
+        self.penalty_names, self.penalty = tuple(penalty) if penalty else None, None
+        self.conv_w = self.conv_bias = None
         if self.whole and (qk_bias or qk_norm_eps is not None or values_are_keys):
             raise ValueError("attention: the two families of options exclude each other")
         if self.chunk < 0 or (self.chunk and window):
@@ -85,14 +98,16 @@ class Attention(Mixer):
         self.w_qkv: torch.Tensor | None = None
         self.w_o: torch.Tensor | None = None
 
-    def cache_spec(self) -> KVGroupSpec:
-        return KVGroupSpec(1, self.n_kv, self.head_dim, self.window, keep_first=self.keep_first)
+    def cache_spec(self) -> KVGroupSpec | list:
+        pages = KVGroupSpec(1, self.n_kv, self.head_dim, self.window, keep_first=self.keep_first)
+        return [pages, StateSpec("attn_conv", (self.taps - 1, self.in_width))] if self.taps > 1 else pages
 
     def weight_specs(self) -> list[WeightSpec]:
         nm = self.names
+        pen = [WeightSpec(n, (self.n_q,), "vector32") for n in self.penalty_names or ()]
         if self.whole:
-            return self._whole_specs()
-        specs = [WeightSpec(nm["q"], (self.q_width, self.hidden))]
+            return self._whole_specs() + pen
+        specs = pen + [WeightSpec(nm["q"], (self.q_width, self.hidden))]
         if self.own_kv:
             specs.append(WeightSpec(nm["k"], (self.kv_width, self.hidden)))
             if not self.values_are_keys:
@@ -108,13 +123,15 @@ class Attention(Mixer):
         nm = self.names
         q_true, k_true, v_true = self.n_q * self.qk_dim, self.n_kv * self.qk_dim, self.n_kv * self.v_dim
         specs = [WeightSpec(nm["q"], (q_true, self.hidden))]
-        if self.all_bias:
+        if self.all_bias or self.qkv_bias:
             specs.append(WeightSpec(nm["q_bias"], (q_true,), "vector32"))
+        if self.taps:
+            specs += [WeightSpec(nm[n] + ".conv", (rows, self.taps), "vector32") for n, rows in (("q", q_true), ("k", k_true), ("v", v_true))]
         if self.whole_norm_eps is not None:
             specs.append(WeightSpec(nm["q_norm"], (q_true,), "vector32"))
         if self.own_kv:
             specs += [WeightSpec(nm["k"], (k_true, self.hidden)), WeightSpec(nm["v"], (v_true, self.hidden))]
-            if self.all_bias:
+            if self.all_bias or self.qkv_bias:
                 specs += [WeightSpec(nm["k_bias"], (k_true,), "vector32"), WeightSpec(nm["v_bias"], (v_true,), "vector32")]
             if self.whole_norm_eps is not None:
                 specs.append(WeightSpec(nm["k_norm"], (k_true,), "vector32"))
@@ -147,6 +164,14 @@ class Attention(Mixer):
             if self.own_kv:
                 self.k_bias = self._pad_heads(tensors[nm["k_bias"]], self.n_kv, self.qk_dim, f32)
                 self.v_bias = self._pad_heads(tensors[nm["v_bias"]], self.n_kv, self.v_dim, f32)
+        if self.conv_form:
+            pad = lambda key, suffix="": [self._pad_heads(tensors[nm[n + key] + suffix], heads, true, f32)      # noqa: E731
+                                          for n, heads, true in (("q", self.n_q, self.qk_dim), ("k", self.n_kv, self.qk_dim),
+                                                                 ("v", self.n_kv, self.v_dim))]
+            if self.qkv_bias:
+                self.conv_bias = torch.cat(pad("_bias"), 0).contiguous()
+            if self.taps:
+                self.conv_w = torch.cat(pad("", ".conv"), 0).t().contiguous()          # [taps, channels]
         if self.whole_norm_eps is not None:
             self.q_norm = self._pad_heads(tensors[nm["q_norm"]], self.n_q, self.qk_dim, f32)
             if self.own_kv:
@@ -154,6 +179,8 @@ class Attention(Mixer):
 
     def load_weights(self, tensors: dict[str, torch.Tensor]) -> None:
         nm = self.names
+        if self.penalty_names:
+            self.penalty = torch.stack([tensors[n].to(device=self.device, dtype=torch.float32) for n in self.penalty_names]).contiguous()
         if self.whole:
             return self._load_whole(tensors)
         f32 = lambda t: t.to(device=self.device, dtype=torch.float32).contiguous()   # noqa: E731
@@ -206,7 +233,16 @@ class Attention(Mixer):
         group = ctx.group_of(call.cache_layer)
         write = call.writes_cache and self.own_kv
         pages, slots = ((k_pages, v_pages), ctx.slots[group]) if write else (None, None)
-        self._prepare(x, qkv, ctx, pages, slots)
+        if self.conv_form:      # queries into rows of their own: a row's convolution reads the rows before it
+            kernels.linear(x, self.w_qkv, qkv)
+            q = ctx.buf("attn.q", (n, self.q_width), self.dtype)
+            kernels.qkv_conv(qkv, q, self.n_q, self.n_kv, d, taps=self.taps, bias=self.conv_bias, weight=self.conv_w,
+                             conv_state=ctx.state("attn_conv", call.cache_layer) if self.taps > 1 else None,
+                             seq_of_token=ctx.seq_of_token, seq_starts=ctx.seq_starts, state_slots=ctx.state_slots, n_seqs=ctx.n_seqs,
+                             first_portion=ctx.n_decode, slots=slots, k_pages=k_pages, v_pages=v_pages, page_size=ctx.page_size)
+            qkv = q
+        else:
+            self._prepare(x, qkv, ctx, pages, slots)
         out = ctx.buf("attn.out", (n, self.q_width), self.dtype)
         tables = ctx.block_tables[group]
         nd = ctx.n_decode
@@ -235,16 +271,16 @@ class Attention(Mixer):
             if may_group and kernels.decode_gqa_supported(self.dtype, d, self.window, self.n_q, self.n_kv, ctx.page_size, split, max_splits):
                 kernels.attention_decode_gqa(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                              out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits, ctx.status,
-                                             split_keys=split, window=self.window, keep_first=self.keep_first, chunk=self.chunk)
+                                             split_keys=split, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
             elif kernels.decode_bulk_supported(self.dtype, d, self.window, self.n_q, self.n_kv, max_splits):
                 kernels.attention_decode_bulk(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                               out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits, ctx.status,
                                               split_keys=split, head_group=heads_per_block, window=self.window,
-                                              keep_first=self.keep_first, chunk=self.chunk)
+                                              keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
             else:
                 kernels.attention_decode(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                          out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits,
-                                         window=self.window, split_keys=split, keep_first=self.keep_first, chunk=self.chunk)
+                                         window=self.window, split_keys=split, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
         if n > nd and kernels.prefill_tc_supported(self.dtype, d, self.window, ctx.page_size):
             blocks = kernels.prefill_tc_blocks(ctx.host_q_len[nd:])
             # a portion that is short against its past: its few blocks' keys are cut into ranges
@@ -259,10 +295,10 @@ class Attention(Mixer):
                 part_ml = ctx.buf("attn.range_ml", (need_ml,), torch.float32)
             kernels.attention_prefill_tc(qkv, k_pages, v_pages, tables[nd:], ctx.seq_starts[nd:], ctx.positions, out, blocks,
                                          self.n_q, self.scale, ctx.status, key_splits=ranges, first_row=nd, part_o=part_o,
-                                         part_ml=part_ml, window=self.window, keep_first=self.keep_first, chunk=self.chunk)
+                                         part_ml=part_ml, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
         elif n > nd:
             kernels.attention_rows(qkv[nd:], k_pages, v_pages, tables, ctx.seq_of_token[nd:], ctx.positions[nd:],
-                                   out[nd:], self.n_q, self.scale, window=self.window, keep_first=self.keep_first, chunk=self.chunk)
+                                   out[nd:], self.n_q, self.scale, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
         return self._project_out(out, ctx)
 
     def _project_out(self, out: torch.Tensor, ctx) -> torch.Tensor:

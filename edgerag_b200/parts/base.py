@@ -17,8 +17,9 @@ Interfaces (duck-typed; the base classes document them):
 * ``Mixer.cache_spec()`` and ``Mixer.forward(x, ctx, call) -> Tensor``;
 * ``FeedForward.forward(x, ctx) -> Tensor``;
 * ``Block.forward(hidden, delta, ctx, call) -> delta`` (the update that is still to be added: rows, float32
-  partial sums, a ``NormedUpdate`` when a norm has to act on it before the add, or a ``ScaledUpdate`` when a
-  constant multiplies it);
+  partial sums, a ``NormedUpdate`` when a norm has to act on it before the add, a ``ScaledUpdate`` when a constant
+  multiplies it, a ``SumUpdate`` when it comes in two pieces, or a ``DepthUpdate`` when the stream is to be averaged
+  with earlier layers' results);
 * ``StreamOp.begin(ctx, hidden)`` and ``StreamOp.forward(hidden, delta, ctx, call) -> delta``: a step of the run
   order between layers that rewrites the residual stream itself (``StreamCall`` in the plan's schedule).
 """
@@ -118,6 +119,28 @@ class ScaledUpdate:
 
 
 @dataclass
+class SumUpdate:
+    """An update of the residual stream in two pieces, ``hidden += a + b`` (each rows or float32 partial sums): what a block
+    whose sublayers read the same normed rows hands on as its ``delta``."""
+
+    a: torch.Tensor
+    b: torch.Tensor
+
+
+@dataclass
+class DepthUpdate:
+    """A rewriting of the stream that is still to be done: with ``x = hidden + (the pending update)`` as the newest entry of
+    ``history``, the stream becomes the average of all entries with the weights ``mix``.  A norm that reads the stream next
+    does it in its own kernel where it has one (``kernels.depth_mix``)."""
+
+    history: torch.Tensor                        # float [layers + 1, rows, width]; entries 0 .. layer are filled
+    layer: int
+    mix: torch.Tensor                            # float [layer + 2]
+    tensor: "torch.Tensor | None" = None         # the pending update: rows or float32 partial sums, or None
+    post: "tuple[torch.Tensor, float] | None" = None   # (weight, eps) of the RMS norm that closes it
+
+
+@dataclass
 class ModelPlan:
     hidden_size: int
     vocab_size: int
@@ -142,6 +165,8 @@ class Part:
     #: step context's tensors (never baked in from its host copies), and nothing may allocate or
     #: synchronise.  Parts that do not say so keep their model on the eager path.
     graph_safe = False
+    #: ``forward`` looks at the tokens' ids: steps that bring rows of embeddings instead are refused
+    needs_token_ids = False
 
     def weight_specs(self) -> list[WeightSpec]:
         return []
@@ -159,7 +184,7 @@ class Norm(Part):
         ``[rows, hidden]`` of the model's element type or float32 partial sums ``[parts, rows, hidden]``.  ``settled`` is a
         hint that a norm may ignore: the caller vouches that ``hidden`` was not written by the kernel
         launched just before this call (only ``delta`` was), so it may be read while that kernel runs.
-        ``delta`` may also be a ``NormedUpdate``; a norm without a kernel for that calls ``settle_update``
+        ``delta`` may also be a ``NormedUpdate``, a ``SumUpdate`` or a ``DepthUpdate``; a norm without a kernel for that calls ``settle_update``
         first and goes on without an update."""
         raise NotImplementedError
 
@@ -212,6 +237,9 @@ class FeedForward(Part):
 
 
 class Block(Part):
+    #: the arrangement has one norm for both sublayers: a layer's ``norm2`` is then None whether or not it has a feed-forward
+    single_norm = False
+
     def forward(self, hidden: torch.Tensor, delta: "torch.Tensor | NormedUpdate | None", ctx: Any,
                 call: LayerCall) -> "torch.Tensor | NormedUpdate | None":
         raise NotImplementedError
@@ -240,6 +268,10 @@ def settle_update(hidden: torch.Tensor, delta: "torch.Tensor | NormedUpdate | No
             delta.norm.add_normed(hidden, delta.tensor, bias=delta.bias)
         else:
             delta.norm.add_normed(hidden, delta.tensor)
+    elif isinstance(delta, SumUpdate):
+        kernels.sum_updates(hidden, delta.a, delta.b, dtype)
+    elif isinstance(delta, DepthUpdate):
+        kernels.depth_mix(hidden, delta.history, delta.layer, delta.mix, dtype, delta=delta.tensor, post=delta.post)
     elif isinstance(delta, ScaledUpdate):
         kernels.residual_add(hidden, delta.tensor, dtype, scale=delta.scale)
     else:

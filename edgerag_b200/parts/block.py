@@ -10,6 +10,9 @@ The closing norms belong to the block (their tensors sit beside the layer's othe
 the opening places it is the arrangement whose sublayers read the stream itself and norm only what they add.  An update leaves a
 sublayer as a ``NormedUpdate``, so that the closing norm, the residual add and the norm that opens the next
 sublayer run as one kernel where the norms have one.
+
+``ParallelBlock`` has one norm whose rows both sublayers read: ``x = norm1(h); h += mixer(x) + ffn(x)``.  Its update leaves
+as a ``SumUpdate``, so that whoever adds it reads both sublayers' outputs in one kernel.
 """
 
 from __future__ import annotations
@@ -17,8 +20,8 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels
-from .base import (Block, FeedForward, LayerCall, Mixer, Norm, NormedUpdate, PartSpec, ScaledUpdate, WeightSpec, build_part,
-                   register_part)
+from .base import (Block, FeedForward, LayerCall, Mixer, Norm, NormedUpdate, PartSpec, ScaledUpdate, SumUpdate, WeightSpec,
+                   build_part, register_part)
 
 
 @register_part("block", "prenorm")
@@ -95,3 +98,29 @@ class SandwichBlock(Block):
         self.norm2.forward(hidden, x, mixed)             # hidden += post1(mixed); x = norm2(hidden)
         ctx.stream_written = kernels.launches()
         return NormedUpdate(self.ffn.forward(x, ctx), self.post2)
+
+
+@register_part("block", "parallel")
+class ParallelBlock(Block):
+    graph_safe = True
+    single_norm = True
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm | None, ffn: FeedForward | None, hidden: int,
+                 dtype: torch.dtype, device: torch.device) -> None:
+        """``norm2`` is None (one norm serves both sublayers); ``ffn`` None: a layer that is its mixer only."""
+        if norm2 is not None:
+            raise ValueError("a parallel block has one norm")
+        if getattr(mixer, "has_update_bias", False):
+            raise ValueError("a mixer whose update carries a bias needs a block that closes the update with a norm")
+        self.norm1, self.mixer, self.ffn = norm1, mixer, ffn
+        self.hidden, self.dtype = hidden, dtype
+
+    def forward(self, hidden: torch.Tensor, delta, ctx, call: LayerCall):
+        x = ctx.buf("block.normed", (hidden.shape[0], self.hidden), self.dtype)
+        self.norm1.forward(hidden, x, delta)             # hidden += delta (or is rewritten); x = norm1(hidden)
+        if delta is not None:
+            ctx.stream_written = kernels.launches()
+        mixed = self.mixer.forward(x, ctx, call)
+        if self.ffn is None:
+            return mixed
+        return SumUpdate(mixed, self.ffn.forward(x, ctx))

@@ -13,6 +13,8 @@ attention kernel is multi-query attention over the cache rows, shared by all hea
 have a sink per head (a learnt logit that takes part in the denominator only), the queries may come
 through a normed latent of their own (``q_rank``), and a layer may read the cache rows that another
 layer wrote (``own_kv=False`` with a ``LayerCall`` that names that layer's cache and does not write).
+With ``gate_entries`` the gate has a logit per entry of the concatenated heads (``H * v_dim`` rows of ``g``) and multiplies
+them after ``Uv_h``.  A scaled rotation may multiply its cosines and sines by a constant (``parts.rope.rotary_multiplier``).
 With ``window`` a query sees its last ``window`` cache rows only (itself among them), the pages behind the
 window go back to the pool, and ``gated=False`` leaves the sigmoid gate out.
 
@@ -27,7 +29,7 @@ import torch
 from ..cache.manager import KVGroupSpec
 from ..ops import kernels
 from .base import LayerCall, Mixer, WeightSpec, register_part
-from .rope import rotary_frequencies
+from .rope import rotary_frequencies, rotary_multiplier
 
 
 def _pad8(n: int) -> int:
@@ -41,13 +43,15 @@ class LatentAttention(Mixer):
     def __init__(self, hidden: int, n_heads: int, dim: int, rot_dim: int, v_dim: int, kv_rank: int, scale: float,
                  rot_base: float, rot_dims: int, eps: float, dtype: torch.dtype, device: torch.device, q_rank: int = 0,
                  sink: bool = False, own_kv: bool = True, gated: bool = True, window: int = 0,
-                 rot_scaling: dict | None = None) -> None:
+                 rot_scaling: dict | None = None, gate_entries: bool = False) -> None:
         if rot_dim % 2 or rot_dims % 2 or rot_dims > rot_dim or kv_rank % 2:
             raise ValueError("latent attention: kv_rank, rot_dim and the rotated dimensions must be even, rot_dims <= rot_dim")
         self.hidden, self.n_heads, self.dim, self.rot_dim, self.v_dim = hidden, n_heads, dim, rot_dim, v_dim
         self.kv_rank, self.q_rank, self.rot_dims = kv_rank, int(q_rank or 0), rot_dims
         self.scale, self.eps = float(scale), float(eps)
         self.sink_on, self.own_kv, self.gated = bool(sink), bool(own_kv), bool(gated)
+        self.gate_entries = bool(gate_entries) and self.gated
+        self.gate_width = 0 if not self.gated else n_heads * v_dim if self.gate_entries else n_heads
         self.window = int(window or 0)
         if self.window < 0:
             raise ValueError("latent attention: a window is positive (or 0 for none)")
@@ -57,8 +61,9 @@ class LatentAttention(Mixer):
         first = self.q_rank or self.q_width
         self.off_kv = first
         self.off_g = first + (kv_rank + rot_dim if own_kv else 0)
-        self.in_width = _pad8(self.off_g + (n_heads if gated else 0))
+        self.in_width = _pad8(self.off_g + self.gate_width)
         self.inv_freq = rotary_frequencies(rot_base, rot_dims, rot_scaling).to(device=device, dtype=torch.float32).contiguous()
+        self.rot_mult = rotary_multiplier(rot_scaling)
         self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = None
         self.kv_norm = self.q_norm = self.sink = None
 
@@ -79,7 +84,7 @@ class LatentAttention(Mixer):
         if self.sink_on:
             specs.append(WeightSpec("sink", (H,), "vector32"))
         if self.gated:
-            specs.append(WeightSpec("g", (H, self.hidden)))
+            specs.append(WeightSpec("g", (self.gate_width, self.hidden)))
         return specs + [WeightSpec("o", (self.hidden, H * self.v_dim))]
 
     def load_weights(self, tensors: dict[str, torch.Tensor]) -> None:
@@ -156,21 +161,25 @@ class LatentAttention(Mixer):
             kernels.latent_store(proj, ctx.positions, self.eps, off_kv=self.off_kv if write else -1, rank=r, rot_dim=dr,
                                  kv_weight=self.kv_norm, inv_freq=self.inv_freq, rot_dims=self.rot_dims,
                                  slots=ctx.slots[group] if write else None, pages=pages if write else None, off_q=0,
-                                 q_rank=self.q_rank, q_weight=self.q_norm, q_latent=q_latent)
+                                 q_rank=self.q_rank, q_weight=self.q_norm, q_latent=q_latent,
+                                 rot_mult=self.rot_mult)
         if self.q_rank:
             q = ctx.buf("latent.qfull", (n, self.q_width), self.dtype)
             kernels.linear(q_latent, self.w_uq, q)
         else:
             q = proj[:, : self.q_width]
         q_lat = ctx.buf("latent.q", (n, H, r + dr), torch.float32)
-        kernels.latent_q_rotate(q, ctx.positions, self.inv_freq, H, self.dim, dr, r, self.rot_dims, q_lat)
+        kernels.latent_q_rotate(q, ctx.positions, self.inv_freq, H, self.dim, dr, r, self.rot_dims, q_lat,
+                                rot_mult=self.rot_mult)
         q_heads = q.as_strided((n, H, self.dim), (q.stride(0), self.dim + dr, 1))
         kernels.linear_batched(q_heads, self.w_uk_t, q_lat[:, :, :r])
         o_lat = ctx.buf("latent.o", (n, H, r), self.dtype)
-        gate = proj[:, self.off_g: self.off_g + H] if self.gated else None
+        gate = proj[:, self.off_g: self.off_g + H] if self.gated and not self.gate_entries else None
         self._attend(ctx, q_lat, pages, ctx.block_tables[group], o_lat, gate)
         heads = ctx.buf("latent.heads", (n, H, self.v_dim), self.dtype)
         kernels.linear_batched(o_lat, self.w_uv, heads)
+        if self.gate_entries:
+            kernels.sigmoid_gate(heads.view(n, H * self.v_dim), proj[:, self.off_g: self.off_g + self.gate_width])
         y = ctx.buf("mixer.out", (n, self.hidden), self.dtype)
         kernels.linear(heads.view(n, H * self.v_dim), self.w_o, y)
         return y

@@ -1,10 +1,11 @@
-"""Layer norm with weight and bias, with the residual add fused in on either side.
+"""Layer norm with weight and (unless ``bias=False``) bias, with the residual add fused in on either side.
 
 ``y = (x - mean) / sqrt(var + eps) * w + b`` with ``var`` the mean of the squared deviations, statistics
 in float32 over the float32 stream.  As the norm before a sublayer it adds the pending update while it
 reads (``forward``); the update may itself be waiting for a norm (``NormedUpdate``: a block whose
 sublayers end in a norm), and then the closing norm, the add and this norm are one kernel.  As the norm
-that closes a sublayer it is applied to the sublayer's output and added to the stream (``add_normed``).
+that closes a sublayer it is applied to the sublayer's output and added to the stream (``add_normed``).  A pending
+average over depth (``DepthUpdate``) is taken in the same kernel as the norm that follows it.
 """
 
 from __future__ import annotations
@@ -12,7 +13,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels
-from .base import Norm, NormedUpdate, WeightSpec, register_part, settle_update
+from .base import DepthUpdate, Norm, NormedUpdate, ScaledUpdate, SumUpdate, WeightSpec, register_part, settle_update
 
 
 @register_part("norm", "layernorm")
@@ -20,21 +21,23 @@ class LayerNorm(Norm):
     graph_safe = True
 
     def __init__(self, size: int, eps: float, dtype: torch.dtype, device: torch.device, tensor: str = "weight",
-                 bias_tensor: str | None = None) -> None:
-        """``tensor`` / ``bias_tensor``: names below the part's prefix (the bias defaults to ``tensor + ".b"``)."""
+                 bias_tensor: str | None = None, bias: bool = True) -> None:
+        """``tensor`` / ``bias_tensor``: names below the part's prefix (the bias defaults to ``tensor + ".b"``);
+        ``bias`` False: a weight only."""
         self.size, self.eps = size, float(eps)
         self.dtype, self.device = dtype, device
         self.tensor = tensor
-        self.bias_tensor = bias_tensor or tensor + ".b"
+        self.bias_tensor = (bias_tensor or tensor + ".b") if bias else None
         self.weight: torch.Tensor | None = None
         self.bias: torch.Tensor | None = None
 
     def weight_specs(self) -> list[WeightSpec]:
-        return [WeightSpec(self.tensor, (self.size,), kind="vector32"), WeightSpec(self.bias_tensor, (self.size,), kind="vector32")]
+        return [WeightSpec(name, (self.size,), kind="vector32") for name in (self.tensor, self.bias_tensor) if name is not None]
 
     def load_weights(self, tensors: dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self.tensor].to(device=self.device, dtype=torch.float32).contiguous()
-        self.bias = tensors[self.bias_tensor].to(device=self.device, dtype=torch.float32).contiguous()
+        if self.bias_tensor is not None:
+            self.bias = tensors[self.bias_tensor].to(device=self.device, dtype=torch.float32).contiguous()
 
     def _post(self, delta):
         """(rows or partial sums, the closing norm's (weight, bias, eps) or None) of a pending update; a
@@ -46,6 +49,13 @@ class LayerNorm(Norm):
         return None, None
 
     def forward(self, hidden, out, delta=None, rows=None, write_back=True, settled=False) -> None:
+        if isinstance(delta, DepthUpdate):      # the average over depth and this norm in one kernel
+            kernels.depth_mix(hidden, delta.history, delta.layer, delta.mix, self.dtype, delta=delta.tensor, post=delta.post, out=out,
+                              out_kind="layernorm", weight=self.weight, bias=self.bias, eps=self.eps, rows=rows, write_back=write_back)
+            return
+        if isinstance(delta, (SumUpdate, ScaledUpdate)):
+            settle_update(hidden, delta, self.dtype)
+            delta = None
         if isinstance(delta, NormedUpdate) and delta.bias is not None:
             raise ValueError("a layer norm has no kernel for an update that carries a bias")
         if isinstance(delta, NormedUpdate) and not isinstance(delta.norm, LayerNorm):

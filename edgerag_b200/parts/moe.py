@@ -4,8 +4,8 @@ optionally through a shared expert that every token uses.
     z = W_router x (float32),   s = sigmoid(z),   chosen = the ``top`` largest s (the lower index wins a tie)
     y = sum over chosen e of expert_e(w_e x) + shared(x),      expert(r) = W_down (silu(W_gate r) * (W_up r))
 
-``weights`` says what ``w_e`` is: ``"score"`` (the score itself; ``"score_normed"``, the chosen scores divided by their
-sum, is not built).  With ``scale_input`` the weight multiplies the expert's input (rounded once to the element type),
+``weights`` says what ``w_e`` is: ``"score"`` (the score itself) or ``"score_normed"`` (the chosen scores divided by their
+sum + 1e-20).  With ``scale_input`` the weight multiplies the expert's input (rounded once to the element type),
 otherwise its output: ``y = sum_e w_e expert_e(x)``, the weight applied in float to the down product's sums.  Experts
 have no biases.  The experts' tensors are ``e<i>.{gate, up, down}`` below the part's prefix, the router ``router``, the
 shared expert a feed-forward part of its own under ``shared.``.
@@ -13,7 +13,9 @@ shared expert a feed-forward part of its own under ``shared.``.
 Further options: ``scores = "softmax"`` (the scores are the softmax of the logits over all experts; the choice still
 goes by the largest); ``groups = (count, keep)``: the experts form ``count`` equal groups of neighbours, a group's score
 is its best expert's, and only experts of the ``keep`` best groups can be chosen; ``gated = False`` with ``act =
-"relu_squared"``: experts without a gate branch, ``W_down relu(W_up r)^2`` (tensors ``e<i>.{up, down}``).
+"relu_squared"``: experts without a gate branch, ``W_down relu(W_up r)^2`` (tensors ``e<i>.{up, down}``); ``correction`` (a tensor's name, sigmoid scores): the choice goes
+by ``s + correction``, the weights by ``s``; ``group_score = "top2_sum"``: a group counts as much as the sum of its two best
+experts.
 
 Nothing here goes through the host: the router's kernel leaves, on the device, every expert's list of (token, choice)
 pairs, and the two product kernels walk row tiles of those lists, so the launches of a step depend on its number of
@@ -37,11 +39,15 @@ class RoutedExperts(FeedForward):
                  shared: PartSpec | None = None, weights: str = "score", scale_input: bool = True,
                  names: tuple[str, str, str] = ("gate", "up", "down"), router: str = "router", expert: str = "e{}.",
                  scores: str = "sigmoid", groups: tuple[int, int] | None = None, gated: bool = True,
-                 act: str = "silu") -> None:
+                 act: str = "silu", correction: str | None = None, group_score: str = "best") -> None:
         if not 0 < top <= n_experts:
             raise ValueError(f"routed_experts: top {top} of {n_experts} experts")
-        if weights != "score":
-            raise ValueError("routed_experts: only the scores themselves are built as weights")
+        if weights not in ("score", "score_normed"):
+            raise ValueError(f"routed_experts: weights {weights!r}; known: score, score_normed")
+        if group_score not in kernels.MOE_GROUP_SCORES or (scores != "sigmoid" and (correction or group_score != "best")):
+            raise ValueError("routed_experts: a correction and groups that count their two best go with sigmoid scores")
+        self.normalise, self.correction_name, self.group_score = weights == "score_normed", correction, group_score
+        self.correction: torch.Tensor | None = None
         if scores not in kernels.MOE_SCORES:
             raise ValueError(f"routed_experts: scores {scores!r}; known: {sorted(kernels.MOE_SCORES)}")
         if (gated and act != "silu") or (not gated and act != "relu_squared"):
@@ -63,6 +69,8 @@ class RoutedExperts(FeedForward):
     def weight_specs(self) -> list[WeightSpec]:
         gate, up, down = self.names
         specs = [WeightSpec(self.router_name, (self.n_experts, self.hidden), "vector32")]
+        if self.correction_name is not None:
+            specs.append(WeightSpec(self.correction_name, (self.n_experts,), "vector32"))
         for e in range(self.n_experts):
             pre = self.expert_fmt.format(e)
             if self.gated:
@@ -76,6 +84,8 @@ class RoutedExperts(FeedForward):
         gate, up, down = self.names
         cast = lambda t: t.to(device=self.device, dtype=self.dtype)  # noqa: E731
         self.w_router = tensors[self.router_name].to(device=self.device, dtype=torch.float32).contiguous()
+        if self.correction_name is not None:
+            self.correction = tensors[self.correction_name].to(device=self.device, dtype=torch.float32).contiguous()
         pres = [self.expert_fmt.format(e) for e in range(self.n_experts)]
         if self.gated:
             self.w_gate_up = torch.stack([torch.cat([cast(tensors[p + gate]), cast(tensors[p + up])], 0) for p in pres]).contiguous()
@@ -91,11 +101,13 @@ class RoutedExperts(FeedForward):
         score = ctx.buf("moe.score", (n * top,), torch.float32)
         act = ctx.buf("moe.act", (n * top, self.intermediate), self.dtype)
         parts = ctx.buf("ffn.out_parts", (top + (self.shared is not None), n, self.hidden), torch.float32)
+        route = dict(scores=self.scores, groups=self.groups, correction=self.correction, group_score=self.group_score,
+                     normalise=self.normalise)
         in_score, out_score = (score, None) if self.scale_input else (None, score)
         if kernels.moe_tc_supported(self.dtype, self.hidden, self.intermediate):
             # tensor cores: row tiles sized by the step's tokens, the (scaled) rows gathered once in list order
             tile_rows = kernels.moe_tc_tile_rows(n, self.n_experts, top)
-            kernels.moe_route(x, self.w_router, top, lists, score, tile_rows, scores=self.scores, groups=self.groups)
+            kernels.moe_route(x, self.w_router, top, lists, score, tile_rows, **route)
             xs = ctx.buf("moe.rows", (n * top, self.hidden), self.dtype)
             kernels.moe_tc_gather(x, lists, in_score, self.n_experts, top, xs)
             if self.gated:
@@ -104,11 +116,9 @@ class RoutedExperts(FeedForward):
                 kernels.moe_tc_up_act(xs, self.w_gate_up, lists, top, tile_rows, act)
             kernels.moe_tc_down(act, self.w_down, lists, top, tile_rows, parts, out_score=out_score)
         else:
-            kernels.moe_route(x, self.w_router, top, lists, score, scores=self.scores, groups=self.groups)
+            kernels.moe_route(x, self.w_router, top, lists, score, **route)
             if self.gated:
-                if in_score is None:
-                    raise ValueError("routed_experts: gated experts on the general kernels take their weight on the input")
-                kernels.moe_gate_up(x, self.w_gate_up, lists, score, top, act)
+                kernels.moe_gate_up(x, self.w_gate_up, lists, in_score, top, act)
             else:
                 if in_score is not None:
                     raise ValueError("routed_experts: experts without a gate branch take their weight on the output")

@@ -11,7 +11,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import kernels
-from .base import Norm, NormedUpdate, ScaledUpdate, WeightSpec, register_part, settle_update
+from .base import DepthUpdate, Norm, NormedUpdate, ScaledUpdate, SumUpdate, WeightSpec, register_part, settle_update
 
 
 @register_part("norm", "rmsnorm")
@@ -51,6 +51,13 @@ class RMSNorm(Norm):
                 raise ValueError("a pending update that another kind of norm has to close can only be added to all rows")
             settle_update(hidden, delta, self.dtype)
             delta, settled = None, False
+        if isinstance(delta, DepthUpdate) and self.exact:      # the average over depth and this norm in one kernel
+            kernels.depth_mix(hidden, delta.history, delta.layer, delta.mix, self.dtype, delta=delta.tensor, post=delta.post, out=out,
+                              out_kind="rmsnorm", weight=self.weight, eps=self.eps, rows=rows, write_back=write_back)
+            return
+        if isinstance(delta, (SumUpdate, DepthUpdate)):
+            settle_update(hidden, delta, self.dtype)
+            delta, settled = None, False
         scale = 1.0
         if isinstance(delta, ScaledUpdate):      # the constant rides into the kernel that adds the update
             delta, scale = delta.tensor, delta.scale
@@ -87,6 +94,9 @@ class PassNorm(Norm):
 
     def forward(self, hidden, out, delta=None, rows=None, write_back=True, settled=False) -> None:
         post = bias = None
+        if isinstance(delta, (SumUpdate, DepthUpdate)):
+            settle_update(hidden, delta, self.dtype)
+            delta = None
         if isinstance(delta, NormedUpdate):
             if isinstance(delta.norm, RMSNorm):
                 post, bias, delta = (delta.norm.weight, delta.norm.eps), delta.bias, delta.tensor

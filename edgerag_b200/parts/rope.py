@@ -28,10 +28,23 @@ def rotary_frequencies(base: float, dims: int, scaling: dict | None = None) -> t
     """``f_i = base^(-2i / dims)`` for ``i < dims / 2``, made in float64.  ``scaling = {factor, low, high, original}``
     stretches the long wavelengths: with ``l = 2 pi / f``, a frequency stays where ``l < original / high``, becomes
     ``f / factor`` where ``l > original / low``, and in between is the blend ``(1 - s) f / factor + s f`` with
-    ``s = (original / l - low) / (high - low)``."""
+    ``s = (original / l - low) / (high - low)``.
+
+    ``scaling = {factor, original, fast, slow}`` (YaRN, Peng et al. 2023) tells the pairs apart by the turns they make within
+    ``original`` positions: ``pair(t) = dims * ln(original / (2 pi t)) / (2 ln base)`` is the pair that makes ``t`` turns; up
+    to ``lo = max(floor(pair(fast)), 0)`` a frequency stays, from ``hi = min(ceil(pair(slow)), dims - 1)`` on it becomes
+    ``f / factor``, between them the two are blended linearly in ``i``.  (Its other half is ``rotary_multiplier``.)"""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = float(base) ** (-2.0 * i / max(dims, 1))
-    if scaling:
+    if scaling and "fast" in scaling:
+        factor, original, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+        if not (factor > 0 and original > 0 and fast > 0 and slow > 0) or base <= 0 or base == 1:
+            raise ValueError("rotary scaling needs positive factor, original, fast and slow, and a base other than 1")
+        pair = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))   # noqa: E731
+        lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = f / factor * ramp + f * (1.0 - ramp)
+    elif scaling:
         factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         if not (factor > 0 and high > low and original > 0):
             raise ValueError("rotary scaling needs factor > 0, high > low and original > 0")
@@ -40,6 +53,12 @@ def rotary_frequencies(base: float, dims: int, scaling: dict | None = None) -> t
         blend = (1.0 - s) * f / factor + s * f
         f = torch.where(wavelength < original / high, f, torch.where(wavelength > original / low, f / factor, blend))
     return f
+
+
+def rotary_multiplier(scaling: dict | None) -> float:
+    """What a scaled rotation multiplies cosines and sines by: ``0.1 ln(factor) + 1`` for ``{factor, original, fast, slow}``,
+    1 for everything else."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
 
 
 @register_part("position", "rope_halves")
