@@ -264,3 +264,119 @@ def greedy(w: dict, cfg: dict, prompt: list[int], n_new: int) -> list[int]:
         out.append(int(forward(w, cfg, seq)[-1].argmax()))
         seq.append(out[-1])
     return out
+
+
+# --- configurations and random weights for the tests --------------------------------------------------------------
+
+def mamba_layer(heads=4, vdim=8, state=12, groups=2, conv=4, norm_groups=2, mlp=None) -> dict:
+    return {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv,
+                                        "norm_groups": norm_groups}, "mlp": mlp}
+
+
+def attention_layer(heads=4, kv_heads=2, dim=16, vdim=24, conv=4, scale=None, mlp=None) -> dict:
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv,
+                                           "scale": scale or dim ** -0.5}, "mlp": mlp}
+
+
+def latent_layer(heads=3, dim=8, rot_dim=8, vdim=16, kv_rank=24, q_rank=20, scale=None, base=500.0, scaling=None, kv_from=None,
+                 mlp=None) -> dict:
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank,
+             "scale": scale or (dim + rot_dim) ** -0.5, "rot": {"base": base, "dims": rot_dim}}
+    if scaling:
+        mixer["rot"]["scaling"] = scaling
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+
+
+def dense_mlp(ff=48) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_mlp(ff=16, experts=6, top=2, groups=(3, 2)) -> dict:
+    router = {"experts": experts, "top": top}
+    if groups:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff}, "router": router}
+
+
+def make_config(layers: list[dict], width=32, vocab=97, eps=1e-5, scale=3.0, side=8, softcap=9.0) -> dict:
+    return {"architecture": "Sabolorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale},
+            "token_side": {"dim": side}, "logit_softcap": softcap, "layers": layers}
+
+
+def tensor_shapes(cfg: dict) -> dict[str, tuple[int, ...]]:
+    W, S, n = cfg["width"], cfg["token_side"]["dim"], len(cfg["layers"])
+    shapes: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], W), "final.norm": (W,), "side.embed": (cfg["vocab"], n * S)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        x = p + "mix."
+        shapes.update({p + "norm1": (W,), p + "dwa": (i + 2,), p + "side.gate": (S, W), p + "side.proj": (W, S), p + "side.norm": (W,)})
+        if layer["type"] == "mamba2":
+            H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+            ch = H * P + 2 * G * N
+            shapes.update({x + "in": (H * P + ch + H, W), x + "conv": (ch, m["conv"]), x + "conv.b": (ch,), x + "dt_bias": (H,),
+                           x + "A_log": (H,), x + "D": (H,), x + "norm": (H * P,), x + "o": (W, H * P)})
+        elif layer["type"] == "attention":
+            H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for name, rows in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                shapes.update({x + name: (rows, W), x + name + ".b": (rows,), x + name + ".conv": (rows, m["conv"])})
+            shapes.update({x + "r1": (H,), x + "r2": (H,), x + "o": (W, H * dv)})
+        else:
+            H, d, dr, dv, r, rq = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            shapes.update({x + "dq": (rq, W), x + "dq.norm": (rq,), x + "uq": (H * (d + dr), rq)})
+            if m.get("kv_from") is None:
+                shapes.update({x + "dkv": (r + dr, W), x + "dkv.norm": (r,)})
+            shapes.update({x + "uk": (H * d, r), x + "uv": (H * dv, r), x + "g": (H * dv, W), x + "o": (W, H * dv)})
+        mlp = layer.get("mlp")
+        if not mlp:
+            continue
+        if mlp["kind"] == "dense":
+            shapes.update({p + "mlp.up": (mlp["ff"], W), p + "mlp.down": (W, mlp["ff"])})
+        else:
+            ff, experts = mlp["expert"]["ff"], mlp["router"]["experts"]
+            for e in range(experts):
+                shapes.update({p + f"mlp.e{e}.gate": (ff, W), p + f"mlp.e{e}.up": (ff, W), p + f"mlp.e{e}.down": (W, ff)})
+            shapes.update({p + "mlp.router": (experts, W), p + "mlp.correction": (experts,)})
+    return shapes
+
+
+def random_weights(cfg: dict, seed: int = 0, dtype: torch.dtype = torch.bfloat16) -> dict[str, torch.Tensor]:
+    """Weights of a size that keeps every sublayer's update comparable with the stream."""
+    gen = torch.Generator().manual_seed(seed)
+    normal = lambda shape, std=1.0, mean=0.0: mean + std * torch.randn(shape, generator=gen)                # noqa: E731
+    between = lambda shape, lo, hi: lo + (hi - lo) * torch.rand(shape, generator=gen)                       # noqa: E731
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if name in ("embed", "side.embed"):
+            t = normal(shape)
+        elif leaf == "norm" and ".side." in name:
+            t = normal(shape, 0.1, 0.7)
+        elif leaf in ("norm1", "norm"):
+            t = normal(shape, 0.1, 1.0)
+        elif leaf == "dwa":
+            t = normal(shape, 0.3)
+            t[-1] += 1.0
+        elif leaf == "conv":
+            t = normal(shape, shape[1] ** -0.5)
+        elif leaf == "b":
+            t = normal(shape, 0.3)
+        elif leaf == "dt_bias":
+            t = between(shape, -3.5, -0.5)
+        elif leaf == "A_log":
+            t = between(shape, -4.0, 0.5)
+        elif leaf == "D":
+            t = normal(shape, 0.5, 1.0)
+        elif leaf == "r1":
+            t = between(shape, 0.0, 2.0)
+        elif leaf == "r2":
+            t = between(shape, 0.05, 0.6)
+        elif leaf == "router":
+            t = normal(shape, 2.0 * shape[1] ** -0.5)
+        elif leaf == "correction":
+            t = normal(shape, 0.4, -0.5)
+        else:
+            t = normal(shape, 1.2 * shape[-1] ** -0.5)
+        out[name] = t.to(dtype)
+    return out
