@@ -604,6 +604,32 @@ def pudadra_config(size: dict, n_layers: int) -> dict:
             "logit_scale": 1.0, "layers": layers}
 
 
+#: the Sabolorn sizes beside DESIGN_SIZES: heads of 64 with a quarter as many kv heads, the state-space and latent mixers of
+#: the sizes above, routed experts whose chosen ones are together as wide as the dense feed-forward (top * ff / 4)
+SABOLORN_ROUTER = {"experts": 32, "top": 4, "groups": {"count": 8, "keep": 4}}
+
+
+def sabolorn_config(size: dict, n_layers: int) -> dict:
+    """Layers in the order state-space mixer with a dense feed-forward, attention, latent attention, latent attention on the
+    cache rows of the layer before (these three with routed experts); repeated."""
+    heads = size["width"] // 64
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 64, "scale": 64 ** -0.5, "conv": 4}
+    att = dict(size["att"])
+    latent = dict(att, scale=(att["dim"] + att["rot_dim"]) ** -0.5,
+                  rot={"base": 10000.0, "dims": att["rot_dim"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    moe = {"kind": "moe", "expert": {"ff": size["ff"] // 4}, "router": dict(SABOLORN_ROUTER)}
+    layers = []
+    for i in range(n_layers):
+        if i % 4 == 0:
+            layers.append({"type": "mamba2", "mixer": dict(size["ssm"]), "mlp": {"kind": "dense", "ff": size["ff"]}})
+        elif i % 4 == 1:
+            layers.append({"type": "attention", "mixer": dict(attention), "mlp": moe})
+        else:
+            layers.append({"type": "latent_attention", "mixer": dict(latent, **({"kv_from": i - 1} if i % 4 == 3 else {})), "mlp": moe})
+    return {"architecture": "Sabolorn", "width": size["width"], "vocab": size["vocab"], "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-5}, "token_side": {"dim": size["width"] // 8}, "logit_softcap": 30.0, "layers": layers}
+
+
 def run_designs(args) -> dict:
     """Prefill (one portion of 2,048 tokens) and decode (batch 1 and --batch at a context of 2,048) of one design
     (--design) and of the Llama decoder at the same width, feed-forward size, vocabulary and number of layer
@@ -683,6 +709,8 @@ def run_designs(args) -> dict:
         return run_lozanex(args, measure, n_layers, block, clocks, peak_source, microbench)
     if args.design == "pudadra":
         return run_pudadra(args, measure, n_layers, block, clocks, peak_source, microbench)
+    if args.design == "sabolorn":
+        return run_sabolorn(args, measure, n_layers, block, clocks, peak_source, microbench)
     for name, size in DESIGN_SIZES.items():
         out[name] = {"layers": n_layers, "dokodra": measure(dokodra_config(size, n_layers), size["vocab"]),
                      "llama": measure(llama_config(size, n_layers), size["vocab"])}
@@ -882,6 +910,65 @@ def run_pudadra(args, measure, n_layers: int, block: int, clocks, peak_source: s
             "sizes": out, "kernels": kern, "step_kernels": steps, "clocks": clocks.record()}
 
 
+def run_sabolorn(args, measure, n_layers: int, block: int, clocks, peak_source: str, microbench) -> dict:
+    """Sabolorn beside Dokodra (the framework's other design of state-space and latent-attention layers) at equal width,
+    layer count and feed-forward width per token, then its kernels beside the like kernels of the other designs at equal
+    work, then which kernels a step of each spends its time in."""
+    import subprocess
+    import tempfile
+    import types
+
+    out: dict = {}
+    for name, size in DESIGN_SIZES.items():
+        out[name] = {"layers": n_layers, "sabolorn": measure(sabolorn_config(size, n_layers), size["vocab"]),
+                     "dokodra": measure(dokodra_config(size, n_layers), size["vocab"])}
+    size = DESIGN_SIZES["w2048"]
+    att, ssm = size["att"], size["ssm"]
+    ns = lambda **kw: types.SimpleNamespace(dtype="bfloat16", iters=10, warmup=3, page=block, sequential_pages=False, **kw)  # noqa: E731
+    heads = dict(heads=32, kv_heads=8, head_dim=64)
+    lat = dict(heads=att["heads"], rank=att["kv_rank"], rot=att["rot_dim"], split=0, kernel="mma")
+    scan = dict(heads=ssm["heads"], head_dim=ssm["vdim"], state=ssm["state"], groups=ssm["groups"])
+    moe = dict(width=size["width"], ff=size["ff"] // 4, experts=SABOLORN_ROUTER["experts"], top=SABOLORN_ROUTER["top"])
+    pre = lambda tokens, **kw: microbench.prefill_attention(ns(tokens=tokens, past=0, kernel="tc", key_splits=0, **heads, **kw))  # noqa: E731
+    dec = lambda batch, **kw: microbench.decode_attention(ns(batch=batch, split=0, head_group=0, cold=True, **heads, **kw))  # noqa: E731
+    kern = {}
+    for tokens in (2048, 8192):
+        kern[f"penalised_attention_prefill_{tokens}"] = pre(tokens, penalty=True)
+        kern[f"llama_attention_prefill_{tokens}"] = pre(tokens)
+    for batch, context in ((8, 8192), (64, 2048)):
+        for kernel in ("gqa", "bulk"):
+            kern[f"penalised_attention_decode_b{batch}_ctx{context}_{kernel}"] = dec(batch, context=context, kernel=kernel, penalty=True)
+            kern[f"llama_attention_decode_b{batch}_ctx{context}_{kernel}"] = dec(batch, context=context, kernel=kernel)
+    kern.update({
+        "latent_attention_decode_b8_ctx8192": microbench.latent_attention(ns(batch=8, context=8192, tokens=0, past=0, cold=True, **lat)),
+        "latent_attention_prefill_2048": microbench.latent_attention(ns(batch=1, context=0, tokens=2048, past=0, cold=False, **lat)),
+        "ssm_scan_decode_b64": microbench.ssm_scan(ns(batch=64, tokens=1, **scan)),
+        "ssm_scan_prefill_2048": microbench.ssm_scan(ns(batch=1, tokens=2048, **scan)),
+    })
+    for rows in (8, 64, 2048):
+        kern[f"corrected_experts_{rows}_rows"] = microbench.routed_experts(ns(tokens=rows, corrected=True, groups=(8, 4), **moe))
+        kern[f"lozanex_experts_{rows}_rows"] = microbench.routed_experts(ns(tokens=rows, **moe))
+        kern[f"stream_ops_{rows}_rows"] = microbench.stream_ops(ns(tokens=rows, width=size["width"], layers=n_layers, heads=32, kv_heads=8))
+    steps = {}
+    for name, cfg in (("sabolorn", sabolorn_config(size, 4)), ("dokodra", dokodra_config(size, 4))):
+        with tempfile.NamedTemporaryFile("w", suffix=".json") as f:
+            json.dump(cfg, f)
+            f.flush()
+            done = subprocess.run([sys.executable, "-m", "edgerag_b200.ops.microbench", "step-kernels", "--config-json", f.name,
+                                   "--batch", str(args.batch), "--context", "2048", "--tokens", "2048", "--iters", "4", "--rows", "30"],
+                                  cwd=str(ROOT), env=dict(os.environ, EDGERAG_B200_NO_CHAIN="1"), capture_output=True, text=True)
+        if done.returncode != 0:
+            raise RuntimeError(f"step-kernels of {name} failed: {done.stderr[-400:]}")
+        steps[name] = json.loads(done.stdout.strip().splitlines()[-1])
+    return {"metric": "design_compare", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16",
+            "data": "synthetic", "impl": "ours", "higher_is_better": True,
+            "config": {"designs": ["Sabolorn", "Dokodra"], "prefill_tokens": 2048, "decode_context": 2048,
+                       "decode_batches": sorted({1, args.batch}), "page_tokens": block, "routed_experts": SABOLORN_ROUTER,
+                       "peaks": peak_source,
+                       "l2": "decode: weights and cache larger than L2 at w2048; kernels: caches, weights and stream rows rotated (cold)"},
+            "sizes": out, "kernels": kern, "step_kernels": steps, "clocks": clocks.record()}
+
+
 def _tensors_of(model) -> list:
     import torch
 
@@ -909,7 +996,7 @@ def main() -> int:
                     help="decode: the headline measurement; mixed / continuous: the serving workloads of the "
                          "256M and 500M decoders through Engine.generate; designs: prefill and decode of one design "
                          "(--design) beside the Llama decoder at equal sizes, and its kernels against their rooflines")
-    ap.add_argument("--design", choices=["dokodra", "vokusun", "lozanex", "pudadra"], default="dokodra",
+    ap.add_argument("--design", choices=["dokodra", "vokusun", "lozanex", "pudadra", "sabolorn"], default="dokodra",
                     help="with --workload designs: the design that is measured beside the Llama decoder")
     ap.add_argument("--ref-cpu-check", action="store_true",
                     help="with --impl reference: a dry run of the reference arm's loop at toy sizes on the CPU")

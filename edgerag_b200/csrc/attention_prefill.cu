@@ -33,7 +33,9 @@
 // maximum and sum in scratch, and a second kernel merges the ranges of each row.
 //
 // With `penalty` (float [2][nq]: r1 of every query head, then r2) the scaled score of a key d positions back is lowered by
-// r1 * ln(1 + r2 * d); the kernel is compiled with and without it.
+// r1 * ln(1 + r2 * d); the kernel is compiled with and without it.  A logarithm per score would double the work of the
+// unit that also makes the exponentials; so where every key of a tile is far from every row, the logarithm is taken once
+// for 16 neighbouring keys, at their middle, and continued to the others by the first three terms of its series.
 //
 // Every wait is bounded: a thread that gives up raises a block-wide flag, every other wait of the
 // block then ends too, the block records a code in *status, lets its copies land, frees its TMEM
@@ -74,6 +76,9 @@ constexpr uint32_t kSmemBytes = kSmemTiles + kSmemExchange + 8 * kNumBars + 16 +
 // (P: two bfloat16 per 32-bit column, the row's keys in order: the A operand of the second product)
 constexpr uint32_t kTmemCols = 512;
 constexpr uint32_t kColS = 0, kColO = 256, kColP = 384;
+// From this distance (in keys) on the penalty of 16 neighbouring keys is a series about their middle, at most 7.5 keys away:
+// the first term left out is below (7.5 / 71.5)^4 / 4 < 4e-5 of r1.
+constexpr int kPenaltyFar = 64;
 constexpr float kSumLimit = 1048576.f;   // a tile's sum of P from which on the reference maximum is moved (2^20)
 constexpr uint32_t kIdescS = mma_idesc(BM, BN, false);
 constexpr uint32_t kIdescO = mma_idesc(BM, HD, true);
@@ -326,7 +331,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
       // 1 + r2 * (distance to this thread's first key of the tile); the keys after it are r2 less each (a key behind the
       // row's own is masked: its logarithm, which may be no number, is never used)
       const float pen_at0 = PEN ? fmaf(pen_r2, (float)(my_pos - key0), 1.f) : 0.f;
-      auto lower = [&](int i) { return pen_r1 * __log2f(fmaf(-pen_r2, (float)i, pen_at0)); };   // of key key0 + i, log2 domain
+      auto lower = [&](float at0, int i) { return pen_r1 * fast_log2(fmaf(-pen_r2, (float)i, at0)); };   // of key key0 + i, log2 domain
+      const bool far = PEN && pos0 + t * BM - (tile_key0 + BN - 1) >= kPenaltyFar;
       // some row of the query tile has hidden keys here: keys after its own, or keys before its window that are not kept
       const bool diagonal = tile_key0 + BN - 1 > pos0 + t * BM || (window != 0 && tile_key0 < first_visible_key(pos0 + t * BM + BM - 1, window));
       // The exponentials are taken against the reference maximum of the tiles before, without looking
@@ -342,12 +348,14 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           float m_half = -INFINITY;
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
+            float at0 = pen_at0;
+            if (PEN) asm volatile("" : "+f"(at0));       // (a value of its own: the compiler would keep 64 logarithms for the pass below)
             float s[32];
             tmem_ld32(t_s + 32 * c, s);
             tmem_ld_wait();
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-              if (PEN) s[i] = fmaf(s[i], scale_log2, -lower(32 * c + i));
+              if (PEN) s[i] = fmaf(s[i], scale_log2, -lower(at0, 32 * c + i));
               m_half = fmaxf(m_half, (diagonal && hidden(key0 + 32 * c + i)) ? -INFINITY : s[i]);
             }
           }
@@ -386,9 +394,22 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           tmem_ld_wait();
           if (c + 1 < 4) tmem_ld16(t_s + 16 * (c + 1), s[(c + 1) & 1]);
           float* sc = s[c & 1];
-          if (PEN) {
+          float at0 = pen_at0;
+          if (PEN) asm volatile("" : "+f"(at0));
+          if (PEN && far) {
+            // r1 log2(a - r2 d) = r1 log2 a - (k1 d + k2 d^2 + k3 d^3 + ...), a the argument at the middle of the 16 keys
+            const float a = fmaf(-pen_r2, 16.f * c + 7.5f, at0), inv = __fdividef(pen_r2, a);
+            const float k1 = pen_r1 * 1.4426950408889634f * inv, k2 = 0.5f * k1 * inv, k3 = 0.33333333f * k1 * inv * inv;
+            const float mid = fmaf(-pen_r1, fast_log2(a), -m_ref);
 #pragma unroll
-            for (int i = 0; i < 16; ++i) sc[i] = fmaf(sc[i], scale_log2, -lower(16 * c + i));
+            for (int i = 0; i < 8; ++i) {                     // keys i and 15 - i lie d on either side of the middle
+              const float d = 7.5f - i, even = fmaf(k2, d * d, mid), odd = fmaf(k3, d * d, k1);
+              sc[i] = fmaf(sc[i], scale_log2, fmaf(-d, odd, even));
+              sc[15 - i] = fmaf(sc[15 - i], scale_log2, fmaf(d, odd, even));
+            }
+          } else if (PEN) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) sc[i] = fmaf(sc[i], scale_log2, -lower(at0, 16 * c + i) - m_ref);
           }
           if (diagonal) {
 #pragma unroll
@@ -397,8 +418,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           }
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            const float p0 = fast_exp2(PEN ? sc[2 * i] - m_ref : fmaf(sc[2 * i], scale_log2, -m_ref));
-            const float p1 = fast_exp2(PEN ? sc[2 * i + 1] - m_ref : fmaf(sc[2 * i + 1], scale_log2, -m_ref));
+            const float p0 = fast_exp2(PEN ? sc[2 * i] : fmaf(sc[2 * i], scale_log2, -m_ref));
+            const float p1 = fast_exp2(PEN ? sc[2 * i + 1] : fmaf(sc[2 * i + 1], scale_log2, -m_ref));
             l4[i & 3] += p0 + p1;
             __nv_bfloat162 b = __floats2bfloat162_rn(p0, p1);
             packed[8 * c + i] = *reinterpret_cast<uint32_t*>(&b);

@@ -43,7 +43,7 @@ struct Penalty2 {
   __device__ __forceinline__ void load(const float* table, int head, int n_heads) {
     if (table) { r1 = table[head]; r2 = table[n_heads + head]; }
   }
-  __device__ __forceinline__ float at(int dist) const { return r1 * __log2f(fmaf(r2, (float)dist, 1.f)); }
+  __device__ __forceinline__ float at(int dist) const { return r1 * fast_log2(fmaf(r2, (float)dist, 1.f)); }
 };
 
 __device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {

@@ -184,6 +184,113 @@ depth_mix_kernel(float* __restrict__ hidden, Update delta, const float* __restri
   }
 }
 
+// The same for rows of up to 2,048 V entries of whole 16-byte pieces: a thread owns the groups of four entries threadIdx.x +
+// v * blockDim.x, which stay in registers, and everything it reads (the update, the stream, the history) is asked for before
+// the first sum over the block.
+template <typename T, int V>
+__global__ void __launch_bounds__(512)
+depth_mix_reg_kernel(float* __restrict__ hidden, Update delta, const float* __restrict__ post_w, float post_eps,
+                     float* __restrict__ history, size_t layer_stride, int n_history, const float* __restrict__ mix, int out_kind,
+                     const float* __restrict__ w, const float* __restrict__ b, float eps, T* __restrict__ out, int out_ld,
+                     const int* __restrict__ rows, int width, int write_back) {
+  __shared__ float scratch[32];
+  const int groups = width >> 2;
+  chain_wait();
+  const int o = blockIdx.x, r = rows ? rows[o] : o;
+  const size_t at = (size_t)r * width;
+  const float inv_w = 1.f / (float)width;
+  float d[V][4], x[V][4], acc[V][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int g = threadIdx.x + v * blockDim.x;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) d[v][k] = x[v][k] = acc[v][k] = 0.f;
+    if (g >= groups) continue;
+    load4(hidden + at + 4 * g, x[v]);
+    if (delta.data) load_update<T, 4>(delta, at + 4 * g, d[v]);
+    const float* past = history + at + 4 * g;
+    int j = 0;
+    for (; j + 4 <= n_history; j += 4) {
+      float h[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) load4(past + (size_t)(j + i) * layer_stride, h[i]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float a = mix[j + i];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) acc[v][k] = fmaf(a, h[i][k], acc[v][k]);
+      }
+    }
+    for (; j < n_history; ++j) {
+      float h[4];
+      load4(past + (size_t)j * layer_stride, h);
+      const float a = mix[j];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) acc[v][k] = fmaf(a, h[k], acc[v][k]);
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) ss = fmaf(d[v][k], d[v][k], ss);
+  }
+  const float own = mix[n_history];
+  const float rs = post_w ? rsqrtf(block_sum(ss, scratch) * inv_w + post_eps) : 1.f;
+  float sum = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int g = threadIdx.x + v * blockDim.x;
+    if (g >= groups) continue;
+    if (post_w) {
+      float pw[4];
+      load4(post_w + 4 * g, pw);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) d[v][k] *= rs * pw[k];
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      x[v][k] += d[v][k];
+      acc[v][k] = fmaf(own, x[v][k], acc[v][k]);
+      sum += out_kind == ERB_OUT_RMSNORM ? acc[v][k] * acc[v][k] : acc[v][k];
+    }
+    if (write_back) {
+      store_f<4>(history + (size_t)n_history * layer_stride + at + 4 * g, x[v]);
+      store_f<4>(hidden + at + 4 * g, acc[v]);
+    }
+  }
+  if (!out) return;
+  float mean = 0.f, scale = 1.f;
+  if (out_kind == ERB_OUT_RMSNORM) {
+    scale = rsqrtf(block_sum(sum, scratch) * inv_w + eps);
+  } else if (out_kind == ERB_OUT_LAYERNORM) {
+    mean = block_sum(sum, scratch) * inv_w;
+    float sq = 0.f;
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      if ((int)(threadIdx.x + v * blockDim.x) >= groups) continue;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) sq = fmaf(acc[v][k] - mean, acc[v][k] - mean, sq);
+    }
+    scale = rsqrtf(block_sum(sq, scratch) * inv_w + eps);
+  }
+  T* y = out + (size_t)o * out_ld;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int g = threadIdx.x + v * blockDim.x;
+    if (g >= groups) continue;
+    float res[4];
+    if (out_kind == ERB_OUT_CAST) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) res[k] = acc[v][k];
+    } else {
+      float ww[4], wb[4] = {0.f, 0.f, 0.f, 0.f};
+      load4(w + 4 * g, ww);
+      if (b) load4(b + 4 * g, wb);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) res[k] = (acc[v][k] - mean) * scale * ww[k] + wb[k];
+    }
+    Pack4<T>::store(y + 4 * g, res);
+  }
+}
+
 bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 }  // namespace
@@ -233,6 +340,12 @@ ERB_EXPORT int erb_depth_mix(float* hidden, const void* delta, int n_parts, long
                    aligned16(delta) && aligned16(post_w) && aligned16(history) && aligned16(w) && aligned16(b) && aligned16(out);
   const int groups = vec ? width / 4 : width;
   const int threads = groups >= 512 ? 512 : (groups + 31) / 32 * 32;
+  if (vec && groups <= 4 * 512) {
+    auto reg = groups <= 512 ? depth_mix_reg_kernel<elem_t, 1> : groups <= 1024 ? depth_mix_reg_kernel<elem_t, 2> : depth_mix_reg_kernel<elem_t, 4>;
+    launch_chained(reg, dim3(n_rows), dim3(threads), 0, (cudaStream_t)stream, hidden, u, post_w, post_eps, history, (size_t)layer_stride,
+                   n_history, mix, out_kind, w, b, eps, (elem_t*)out, out_ld, rows, width, write_back);
+    return check_launch("depth_mix");
+  }
   auto kern = vec ? depth_mix_kernel<elem_t, 4> : depth_mix_kernel<elem_t, 1>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

@@ -196,6 +196,11 @@ __device__ __forceinline__ void tma_load_rows(uint32_t dst, const CUtensorMap* m
       ::"r"(dst), "l"(map), "r"(0), "r"(row), "r"(bar) : "memory");
 }
 
+__device__ __forceinline__ float fast_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float fast_exp2(float x) {          // 2^x, one instruction; -inf gives 0
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

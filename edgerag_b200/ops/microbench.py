@@ -73,6 +73,13 @@ def _time(fn, iters: int, warmup: int, rounds: int = 5) -> float:
     return statistics.median(times)
 
 
+def _penalty_of(a) -> torch.Tensor | None:
+    """``--penalty``: a distance penalty ``[2, heads]`` for the attention kernels."""
+    if not getattr(a, "penalty", False):
+        return None
+    return torch.stack([torch.linspace(0.2, 2.0, a.heads), torch.linspace(0.05, 0.5, a.heads)]).cuda()
+
+
 def _paged(batch: int, context: int, nkv: int, d: int, page: int, dtype, shuffle: bool = True):
     """Key and value pools of ``batch`` sequences of ``context`` tokens with their block tables."""
     pages_per = -(-context // page)
@@ -102,6 +109,7 @@ def decode_attention(a) -> dict:
         return caches[state["i"]]
 
     q = torch.randn((a.batch, a.heads * a.head_dim), device="cuda").to(dtype)
+    pen = _penalty_of(a)
     out = torch.empty_like(q)
     pos = torch.full((a.batch,), a.context - 1, dtype=torch.int32, device="cuda")
     tok = torch.arange(a.batch, dtype=torch.int32, device="cuda")
@@ -122,18 +130,19 @@ def decode_attention(a) -> dict:
     scale = a.head_dim ** -0.5
     if a.kernel == "gqa":
         fn = lambda: kernels.attention_decode_gqa(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
-                                                  status, split_keys=a.split, window=window, keep_first=keep, chunk=chunk)
+                                                  status, split_keys=a.split, window=window, keep_first=keep, chunk=chunk, penalty=pen)
     elif a.kernel == "bulk":
         fn = lambda: kernels.attention_decode_bulk(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
                                                    status, split_keys=a.split, head_group=a.head_group, window=window, keep_first=keep,
-                                                   chunk=chunk)
+                                                   chunk=chunk, penalty=pen)
     else:
         fn = lambda: kernels.attention_decode(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
-                                              split_keys=a.split, window=window, keep_first=keep, chunk=chunk)
+                                              split_keys=a.split, window=window, keep_first=keep, chunk=chunk, penalty=pen)
     us = _time(fn, max(a.iters, 2 * reps), a.warmup)
     return {"case": "decode-attention", "kernel": a.kernel, "split": a.split, "head_group": a.head_group, "us": round(us, 2),
             "bytes": nbytes, "gbs": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / HBM_GBS, 4),
-            "status": int(status), "from_dram": bool(a.cold) or nbytes > 126e6, "window": window, "keep_first": keep, "chunk": chunk}
+            "status": int(status), "from_dram": bool(a.cold) or nbytes > 126e6, "window": window, "keep_first": keep, "chunk": chunk,
+            "penalty": pen is not None}
 
 
 def prefill_attention(a) -> dict:
@@ -146,6 +155,7 @@ def prefill_attention(a) -> dict:
     pos = torch.arange(a.past, total, dtype=torch.int32, device="cuda")
     starts = torch.tensor([0, a.tokens], dtype=torch.int32, device="cuda")
     seq_of = torch.zeros(a.tokens, dtype=torch.int32, device="cuda")
+    pen = _penalty_of(a)
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
     scale = a.head_dim ** -0.5
     window, keep, chunk = getattr(a, "window", 0), getattr(a, "keep_first", 0), getattr(a, "chunk", 0)
@@ -157,10 +167,10 @@ def prefill_attention(a) -> dict:
         part_o, part_ml = torch.empty(need_o, device="cuda"), torch.empty(need_ml, device="cuda")
         fn = lambda: kernels.attention_prefill_tc(qkv, kp, vp, tables, starts, pos, out, blocks, a.heads, scale, status,  # noqa: E731
                                                   key_splits=ranges, part_o=part_o, part_ml=part_ml, window=window, keep_first=keep,
-                                                  chunk=chunk)
+                                                  chunk=chunk, penalty=pen)
     else:
         fn = lambda: kernels.attention_rows(qkv, kp, vp, tables, seq_of, pos, out, a.heads, scale, window=window,  # noqa: E731
-                                            keep_first=keep, chunk=chunk)
+                                            keep_first=keep, chunk=chunk, penalty=pen)
     us = _time(fn, a.iters, a.warmup)
     if window > 0:      # (query, key) pairs that are seen: the window's keys and the kept ones before it
         p = torch.arange(a.past, total, dtype=torch.float64)
@@ -173,7 +183,8 @@ def prefill_attention(a) -> dict:
         pairs = a.tokens * a.past + a.tokens * (a.tokens + 1) / 2
     flops = 4.0 * a.heads * a.head_dim * pairs
     return {"case": "prefill-attention", "kernel": a.kernel, "us": round(us, 2), "tflops": round(flops / us / 1e6, 1),
-            "frac_bf16": round(flops / us / 1e6 / BF16_TFLOPS, 4), "status": int(status), "window": window, "keep_first": keep, "chunk": chunk}
+            "frac_bf16": round(flops / us / 1e6 / BF16_TFLOPS, 4), "status": int(status), "window": window, "keep_first": keep, "chunk": chunk,
+            "penalty": pen is not None}
 
 
 def linear(a) -> dict:
@@ -537,19 +548,25 @@ def routed_experts(a) -> dict:
     tile_rows = kernels.moe_tc_tile_rows(n, E, top) if tc else 0
     if getattr(a, "ungated", False):
         return _routed_experts_ungated(a, x, router, wgu, wd, lists, score, act, parts, tc, tile_rows, rotate, reps, item)
-    kernels.moe_route(x, router, top, lists, score, tile_rows)
+    # --corrected: chosen by score + correction among the best groups, normalised weights that multiply the experts' outputs
+    how = {}
+    if getattr(a, "corrected", False):
+        how = dict(groups=tuple(a.groups) if getattr(a, "groups", None) else None, correction=torch.randn(E, device="cuda") * 0.3,
+                   group_score="top2_sum", normalise=True)
+    in_score, out_score = (None, score) if how else (score, None)
+    kernels.moe_route(x, router, top, lists, score, tile_rows, **how)
     used = int((lists[2 * n * top: 2 * n * top + E] > 0).sum())     # experts that some row chose
-    us_route = _time(lambda: kernels.moe_route(x, router, top, lists, score, tile_rows), a.iters, a.warmup)
+    us_route = _time(lambda: kernels.moe_route(x, router, top, lists, score, tile_rows, **how), a.iters, a.warmup)
     us_gather = 0.0
     if tc:
         xs = torch.empty((n * top, h), dtype=dtype, device="cuda")
-        kernels.moe_tc_gather(x, lists, score, E, top, xs)
-        us_gather = _time(lambda: kernels.moe_tc_gather(x, lists, score, E, top, xs), a.iters, a.warmup)
+        kernels.moe_tc_gather(x, lists, in_score, E, top, xs)
+        us_gather = _time(lambda: kernels.moe_tc_gather(x, lists, in_score, E, top, xs), a.iters, a.warmup)
         us_up = _time(lambda: kernels.moe_tc_gate_up(xs, wgu[rotate()], lists, top, tile_rows, act), max(a.iters, 2 * reps), a.warmup)
-        us_down = _time(lambda: kernels.moe_tc_down(act, wd[rotate()], lists, top, tile_rows, parts), max(a.iters, 2 * reps), a.warmup)
+        us_down = _time(lambda: kernels.moe_tc_down(act, wd[rotate()], lists, top, tile_rows, parts, out_score=out_score), max(a.iters, 2 * reps), a.warmup)
     else:
-        us_up = _time(lambda: kernels.moe_gate_up(x, wgu[rotate()], lists, score, top, act), max(a.iters, 2 * reps), a.warmup)
-        us_down = _time(lambda: kernels.moe_down(act, wd[rotate()], lists, top, parts), max(a.iters, 2 * reps), a.warmup)
+        us_up = _time(lambda: kernels.moe_gate_up(x, wgu[rotate()], lists, in_score, top, act), max(a.iters, 2 * reps), a.warmup)
+        us_down = _time(lambda: kernels.moe_down(act, wd[rotate()], lists, top, parts, out_score=out_score), max(a.iters, 2 * reps), a.warmup)
     # the dense feed-forward of the same arithmetic per token
     dgu = [(torch.randn((2 * top * ff, h), device="cuda") * 0.02).to(dtype) for _ in range(max(1, reps // 4))]
     dd = [(torch.randn((h, top * ff), device="cuda") * 0.02).to(dtype) for _ in range(max(1, reps // 4))]
@@ -605,6 +622,58 @@ def _routed_experts_ungated(a, x, router, wgu, wd, lists, score, act, parts, tc,
             "gather_us": round(us_gather, 2), "up": line(us_up, bytes_up), "down": line(us_down, bytes_down)}
 
 
+def stream_ops(a) -> dict:
+    """The kernels on the residual stream between layers, over ``tokens`` rows: the average over ``layers`` earlier results
+    with the norms on either side of it (bound by the float rows it reads and writes), the sum of a layer's two updates with
+    the rounded copy, the convolution of q, k and v with the cache write, and, for comparison, the plain add with a layer norm."""
+    dtype = torch.bfloat16 if a.dtype == "bfloat16" else torch.float32
+    item = 2 if dtype == torch.bfloat16 else 4
+    n, h, L = a.tokens, a.width, a.layers
+    row_bytes = n * h
+    reps = max(1, int(300e6 // (row_bytes * 4 * (L + 1))) + 1)
+    hist = [torch.randn((L + 1, n, h), device="cuda") for _ in range(reps)]
+    hidden = [torch.randn((n, h), device="cuda") for _ in range(reps)]
+    y, out = torch.randn((n, h), device="cuda").to(dtype), torch.empty((n, h), device="cuda", dtype=dtype)
+    parts = torch.randn((4, n, h), device="cuda")
+    w, mix = torch.randn(h, device="cuda"), torch.randn(L + 1, device="cuda")
+    state = {"i": 0}
+
+    def turn():
+        state["i"] = (state["i"] + 1) % reps
+        return state["i"]
+
+    def depth():
+        i = turn()
+        kernels.depth_mix(hidden[i], hist[i], L - 1, mix, dtype, delta=y, post=(w, 1e-5), out=out, out_kind="layernorm", weight=w, eps=1e-5)
+
+    def line(us, nbytes):
+        return {"us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / HBM_GBS, 4)}
+
+    iters = max(a.iters, 2 * reps)
+    res = {"case": "stream-ops", "tokens": n, "width": h, "layers": L,
+           "depth_mix": line(_time(depth, iters, a.warmup), row_bytes * (4 * (L + 3) + 2 * item)),
+           "sum_updates": line(_time(lambda: kernels.sum_updates(hidden[turn()], y, parts, dtype, out=out), iters, a.warmup),
+                               row_bytes * (8 + 16 + 2 * item)),
+           "add_layernorm": line(_time(lambda: kernels.add_layernorm(hidden[turn()], w, None, out, 1e-5, delta=y), iters, a.warmup),
+                                 row_bytes * (8 + 2 * item))}
+    H, G, D, taps, page = a.heads, a.kv_heads, 64, 4, 16
+    C = (H + 2 * G) * D
+    proj, q = torch.randn((n, C), device="cuda").to(dtype), torch.empty((n, H * D), device="cuda", dtype=dtype)
+    seqs = 1 if n > 64 else n                       # one prompt portion, or single tokens
+    starts = torch.tensor([0, n] if seqs == 1 else list(range(n + 1)), dtype=torch.int32, device="cuda")
+    seq_of = torch.zeros(n, dtype=torch.int32, device="cuda") if seqs == 1 else torch.arange(n, dtype=torch.int32, device="cuda")
+    slots = torch.randperm(n).to(torch.int32).cuda()
+    pages = [torch.empty((-(-n // page), G, page, D), device="cuda", dtype=dtype) for _ in range(2)]
+    record = torch.zeros((seqs, taps - 1, C), device="cuda")
+    bias, cw = torch.randn(C, device="cuda"), torch.randn((taps, C), device="cuda")
+    st = torch.arange(seqs, dtype=torch.int32, device="cuda")
+    conv = lambda: kernels.qkv_conv(proj, q, H, G, D, taps=taps, bias=bias, weight=cw, conv_state=record, seq_of_token=seq_of,   # noqa: E731
+                                    seq_starts=starts, state_slots=st, n_seqs=seqs, first_portion=seqs if n <= 64 else 0,
+                                    slots=slots, k_pages=pages[0], v_pages=pages[1], page_size=page)
+    res["qkv_conv"] = line(_time(conv, a.iters, a.warmup), n * C * 2 * item + 2 * record.numel() * 4)
+    return res
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="edgerag_b200.ops.microbench", description=__doc__.split("\n\n")[0])
     sub = ap.add_subparsers(dest="case", required=True)
@@ -622,6 +691,7 @@ def main(argv=None) -> int:
     att.add_argument("--keep-first", type=int, default=0, help="with a window: first keys that stay visible")
     att.add_argument("--chunk", type=int, default=0, help="instead of a window: a query sees its own run of this many positions")
     att.add_argument("--sequential-pages", action="store_true", help="pages in order instead of shuffled")
+    att.add_argument("--penalty", action="store_true", help="a penalty that grows with the logarithm of the distance")
     d = sub.add_parser("decode-attention", parents=[common, att])
     d.add_argument("--batch", type=int, default=8)
     d.add_argument("--context", type=int, default=8192)
@@ -708,14 +778,21 @@ def main(argv=None) -> int:
     re.add_argument("--top", type=int, default=4)
     re.add_argument("--general", action="store_true", help="the products on CUDA cores (what float32 runs) instead of tensor cores")
     re.add_argument("--ungated", action="store_true", help="experts without a gate branch, softmax scores, the weight on the output")
-    re.add_argument("--groups", type=int, nargs=2, default=None, help="with --ungated: (count, keep) of the router's groups")
+    re.add_argument("--corrected", action="store_true", help="a correction per expert in the choice, normalised weights on the output")
+    re.add_argument("--groups", type=int, nargs=2, default=None, help="with --ungated or --corrected: (count, keep) of the router's groups")
+    so = sub.add_parser("stream-ops", parents=[common])
+    so.add_argument("--tokens", type=int, default=2048)
+    so.add_argument("--width", type=int, default=2048)
+    so.add_argument("--layers", type=int, default=8, help="results that the average over depth takes besides the newest")
+    so.add_argument("--heads", type=int, default=32)
+    so.add_argument("--kv-heads", type=int, default=8)
     a = ap.parse_args(argv)
     if not torch.cuda.is_available():
         print("microbench needs a CUDA device", file=sys.stderr)
         return 1
     fn = {"decode-attention": decode_attention, "prefill-attention": prefill_attention, "linear": linear,
           "step-kernels": step_kernels, "step-timeline": step_timeline, "latent-attention": latent_attention,
-          "ssm-scan": ssm_scan, "delta-scan": delta_scan, "routed-experts": routed_experts, "diff-attention": diff_attention}[a.case]
+          "ssm-scan": ssm_scan, "delta-scan": delta_scan, "routed-experts": routed_experts, "diff-attention": diff_attention, "stream-ops": stream_ops}[a.case]
     load_peaks(a.peaks)
     result = fn(a)
     result["peaks"] = PEAKS_FROM

@@ -704,7 +704,7 @@ def test_router_with_correction_and_gated_experts_on_both_product_paths(sizes, d
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("width", [32, 70, 512, 2048, 5000])
+@pytest.mark.parametrize("width", [32, 70, 512, 2048, 3000, 5000, 9000])
 def test_stream_kernels_between_layers(width, dtype):
     """The sum of two updates, the side input's gate, and the average over depth with the norms on either side of it: every
     form of update, layer norm without and with bias, RMS norm, plain cast, a selection of rows."""
