@@ -35,10 +35,94 @@ namespace {
 
 constexpr int kRouteThreads = 512;
 
+// A warp picks one token's experts from their logits z (shared or global memory): `choice` and `score` (the token's `top` entries).
+// cv and gm: shared memory for an entry per expert each.
+__device__ __forceinline__ void choose_experts(const float* z, float* cv, float* gm, int n_experts, int top, int* __restrict__ choice,
+                                               float* __restrict__ score, int score_kind, int n_groups, int keep_groups,
+                                               const float* __restrict__ correction, int group_kind, int normalise) {
+  const int lane = threadIdx.x & 31;
+  // softmax scores: the maximum and the denominator over all experts, before any expert is ruled out
+  float z_top = 0.f, denom = 1.f;
+  if (score_kind == ERB_SCORE_SOFTMAX) {
+    float mx = -INFINITY;
+    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, z[e]);
+    z_top = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < n_experts; e += 32) sum += expf(z[e] - z_top);
+    denom = warp_sum(sum);
+  }
+  // What the choice goes by: the logits (the scores rise with them), or sigmoid scores plus correction.
+  const bool by_score = correction != nullptr || group_kind == ERB_GROUP_TOP2_SUM;
+  for (int e = lane; e < n_experts; e += 32)
+    cv[e] = by_score ? 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f) : z[e];
+  __syncwarp();
+  // groups of neighbouring experts: a group counts as much as its best expert or as the sum of its two best; the experts
+  // of all but the `keep_groups` best groups are ruled out (the lower group wins a tie)
+  if (n_groups > 1 && keep_groups < n_groups) {
+    const int per = n_experts / n_groups;
+    for (int g = lane; g < n_groups; g += 32) {
+      float mx = -INFINITY, second = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = cv[e];
+        second = fmaxf(second, fminf(mx, v));
+        mx = fmaxf(mx, v);
+      }
+      gm[g] = group_kind == ERB_GROUP_TOP2_SUM && per > 1 ? mx + second : mx;
+    }
+    __syncwarp();
+    for (int c = 0; c < keep_groups; ++c) {
+      float best = -INFINITY;
+      int arg = 0x7fffffff;
+      for (int g = lane; g < n_groups; g += 32) {
+        const float v = gm[g];
+        if (v > best) { best = v; arg = g; }     // (a group already kept holds NaN: never greater)
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+      }
+      if (lane == 0 && arg < n_groups) gm[arg] = __int_as_float(0x7fc00000);
+      __syncwarp();
+    }
+    for (int e = lane; e < n_experts; e += 32)
+      if (gm[e / per] == gm[e / per]) cv[e] = -INFINITY;      // not NaN: the group was not kept
+    __syncwarp();
+  }
+  float total = 0.f;
+  for (int c = 0; c < top; ++c) {
+    float best = -INFINITY;
+    int arg = 0x7fffffff;
+    for (int e = lane; e < n_experts; e += 32) {
+      const float zv = cv[e];
+      if (zv > best) { best = zv; arg = e; }     // rising e within a lane: the first maximum stays
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+    }
+    if (arg >= n_experts) arg = c;                // (no expert compares: logits that are no numbers; any choice does)
+    if (lane == 0) {
+      const float s = score_kind == ERB_SCORE_SOFTMAX ? expf(z[arg] - z_top) / denom : 1.f / (1.f + expf(-z[arg]));
+      choice[c] = arg;
+      score[c] = s;
+      cv[arg] = -INFINITY;
+      total += s;
+    }
+    __syncwarp();
+  }
+  if (normalise && lane == 0)
+    for (int c = 0; c < top; ++c) score[c] /= total + 1e-20f;
+}
+
 // One block per kRouteTokens tokens.  Shared memory: their logits, then their rows as floats.  A warp takes an expert at
 // a time and reads its router row once for all the block's tokens; a lane sums the entries 4 lane .. 4 lane + 3 of every
 // run of 128, then the lanes are added: one order of sums per token whatever the batch.  Then a warp per token picks.
 constexpr int kRouteTokens = 4;
+constexpr int kRouteFewPairs = 512, kRouteFewExperts = 256;   // up to which one block picks and makes the lists
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_router, int n_tokens, int width, int n_experts,
@@ -92,83 +176,8 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
   if (warp >= n_here) return;
   const int t = t0 + warp;
   float* z = z_s + warp * e_pad;
-  // softmax scores: the maximum and the denominator over all experts, before any expert is ruled out
-  float z_top = 0.f, denom = 1.f;
-  if (score_kind == ERB_SCORE_SOFTMAX) {
-    float mx = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, z[e]);
-    z_top = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < n_experts; e += 32) sum += expf(z[e] - z_top);
-    denom = warp_sum(sum);
-  }
-  // What the choice goes by: the logits (the scores rise with them), or sigmoid scores plus correction.
-  float* cv = c_s + warp * e_pad;
-  const bool by_score = correction != nullptr || group_kind == ERB_GROUP_TOP2_SUM;
-  for (int e = lane; e < n_experts; e += 32)
-    cv[e] = by_score ? 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f) : z[e];
-  __syncwarp();
-  // groups of neighbouring experts: a group counts as much as its best expert or as the sum of its two best; the experts
-  // of all but the `keep_groups` best groups are ruled out (the lower group wins a tie)
-  if (n_groups > 1 && keep_groups < n_groups) {
-    float* gm = g_s + warp * e_pad;
-    const int per = n_experts / n_groups;
-    for (int g = lane; g < n_groups; g += 32) {
-      float mx = -INFINITY, second = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) {
-        const float v = cv[e];
-        second = fmaxf(second, fminf(mx, v));
-        mx = fmaxf(mx, v);
-      }
-      gm[g] = group_kind == ERB_GROUP_TOP2_SUM && per > 1 ? mx + second : mx;
-    }
-    __syncwarp();
-    for (int c = 0; c < keep_groups; ++c) {
-      float best = -INFINITY;
-      int arg = 0x7fffffff;
-      for (int g = lane; g < n_groups; g += 32) {
-        const float v = gm[g];
-        if (v > best) { best = v; arg = g; }     // (a group already kept holds NaN: never greater)
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-      }
-      if (lane == 0 && arg < n_groups) gm[arg] = __int_as_float(0x7fc00000);
-      __syncwarp();
-    }
-    for (int e = lane; e < n_experts; e += 32)
-      if (gm[e / per] == gm[e / per]) cv[e] = -INFINITY;      // not NaN: the group was not kept
-    __syncwarp();
-  }
-  float total = 0.f;
-  for (int c = 0; c < top; ++c) {
-    float best = -INFINITY;
-    int arg = 0x7fffffff;
-    for (int e = lane; e < n_experts; e += 32) {
-      const float zv = cv[e];
-      if (zv > best) { best = zv; arg = e; }     // rising e within a lane: the first maximum stays
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-    }
-    if (arg >= n_experts) arg = c;                // (no expert compares: logits that are no numbers; any choice does)
-    if (lane == 0) {
-      const float s = score_kind == ERB_SCORE_SOFTMAX ? expf(z[arg] - z_top) / denom : 1.f / (1.f + expf(-z[arg]));
-      choice[(size_t)t * top + c] = arg;
-      score[(size_t)t * top + c] = s;
-      cv[arg] = -INFINITY;
-      total += s;
-    }
-    __syncwarp();
-  }
-  if (normalise && lane == 0)
-    for (int c = 0; c < top; ++c) score[(size_t)t * top + c] /= total + 1e-20f;
+  choose_experts(z, c_s + warp * e_pad, g_s + warp * e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, score_kind,
+                 n_groups, keep_groups, correction, group_kind, normalise);
 }
 
 // One block per expert e builds the expert's part of the lists on its own: a histogram of all choices in shared memory
@@ -219,6 +228,113 @@ __global__ void __launch_bounds__(256) moe_lists_kernel(const int* __restrict__ 
       base_s += all;
     }
     __syncthreads();
+  }
+}
+
+// Few tokens.  With a block per kRouteTokens tokens a handful of blocks would each stream the whole router matrix; here a warp
+// takes one expert for kRouteTokens tokens and writes their logits, summed exactly as in moe_route_kernel, so that a token's
+// choice does not depend on which of the two made it.  grid (token groups, experts / 4).
+template <typename T>
+__global__ void __launch_bounds__(128)
+moe_logits_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_router, int n_tokens, int width, int n_experts,
+                  float* __restrict__ logits) {
+  chain_wait();
+  const int t0 = blockIdx.x * kRouteTokens, lane = threadIdx.x & 31, e = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (e >= n_experts) return;
+  const int n_here = min(kRouteTokens, n_tokens - t0);
+  const float* w = w_router + (size_t)e * width;
+  const T* rows[kRouteTokens];
+  float acc[kRouteTokens];
+#pragma unroll
+  for (int j = 0; j < kRouteTokens; ++j) {
+    rows[j] = x + (size_t)(t0 + min(j, n_here - 1)) * ld;
+    acc[j] = 0.f;
+  }
+  const bool pack = ((uintptr_t)x & 15) == 0 && (ld & 3) == 0;
+  const int whole = (width & 3) == 0 && pack ? width & ~127 : 0;
+#pragma unroll 4
+  for (int k = 4 * lane; k < whole; k += 128) {
+    const float4 wv = *reinterpret_cast<const float4*>(w + k);
+#pragma unroll
+    for (int j = 0; j < kRouteTokens; ++j) {
+      float xv[4];
+      Pack4<T>::load(rows[j] + k, xv);
+      acc[j] = fmaf(xv[0], wv.x, acc[j]);
+      acc[j] = fmaf(xv[1], wv.y, acc[j]);
+      acc[j] = fmaf(xv[2], wv.z, acc[j]);
+      acc[j] = fmaf(xv[3], wv.w, acc[j]);
+    }
+  }
+  // (unaligned rows take the same order entry by entry)
+  const int order4 = (width & 3) == 0 ? width & ~127 : 0;
+  for (int k = whole + 4 * lane; k < order4; k += 128)
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < kRouteTokens; ++j) acc[j] = fmaf(Elem<T>::load(rows[j] + k + i), w[k + i], acc[j]);
+  for (int k = order4 + lane; k < width; k += 32) {
+    const float wv = w[k];
+#pragma unroll
+    for (int j = 0; j < kRouteTokens; ++j) acc[j] = fmaf(Elem<T>::load(rows[j] + k), wv, acc[j]);
+  }
+#pragma unroll
+  for (int j = 0; j < kRouteTokens; ++j) {
+    const float total = warp_sum(acc[j]);
+    if (lane == 0 && j < n_here) logits[(size_t)(t0 + j) * n_experts + e] = total;
+  }
+}
+
+// ... and one block picks for all of them, a warp a token at a time, and builds the lists: thread e walks the pairs (parked in
+// shared memory) for expert e, so an expert's pairs come out in rising order as in moe_lists_kernel.
+__global__ void __launch_bounds__(kRouteThreads)
+moe_choose_lists_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top, int* __restrict__ choice,
+                        float* __restrict__ score, int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ tiles,
+                        int* __restrict__ order, int tile_rows, int score_kind, int n_groups, int keep_groups,
+                        const float* __restrict__ correction, int group_kind, int normalise) {
+  chain_wait();
+  extern __shared__ float z_s[];                 // per warp: logits, what the choice goes by, the groups' values
+  constexpr int kWarps = kRouteThreads / 32;
+  __shared__ int pair_s[kRouteFewPairs];
+  const int e_pad = (n_experts + 3) & ~3, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int* count_s = reinterpret_cast<int*>(z_s + 3 * kWarps * e_pad);      // [n_experts], then [n_experts] offsets
+  int* off_s = count_s + e_pad;
+  float* z = z_s + 3 * warp * e_pad;
+  for (int t = warp; t < n_tokens; t += kWarps) {
+    for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * n_experts + e];
+    __syncwarp();
+    choose_experts(z, z + e_pad, z + 2 * e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, score_kind, n_groups,
+                   keep_groups, correction, group_kind, normalise);
+    __syncwarp();
+    for (int c = lane; c < top; c += 32) pair_s[t * top + c] = choice[(size_t)t * top + c];
+    __syncwarp();
+  }
+  __syncthreads();
+  const int n_pairs = n_tokens * top;
+  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
+    int n = 0;
+#pragma unroll 4
+    for (int i = 0; i < n_pairs; ++i) n += pair_s[i] == e;
+    count_s[e] = n;
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int off = 0, tl = 0;
+    for (int e = 0; e < n_experts; ++e) {
+      counts[e] = count_s[e];
+      offsets[e] = off_s[e] = off;
+      tiles[e] = tl;
+      off += count_s[e];
+      tl += (count_s[e] + tile_rows - 1) / tile_rows;
+    }
+    offsets[n_experts] = off;
+    tiles[n_experts] = tl;
+    counts[n_experts] = 0;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
+    int at = off_s[e];
+    const int stop = at + count_s[e];
+    for (int i = 0; at < stop; ++i)
+      if (pair_s[i] == e) order[at++] = i;
   }
 }
 
@@ -328,10 +444,15 @@ moe_product_kernel(const T* __restrict__ a, int lda, const T* __restrict__ weigh
 
 ERB_EXPORT int erb_moe_tile_rows() { return kTM; }
 
+// Whether a step of this many tokens is routed by the pair of kernels for few tokens (then `logits` is [n_tokens][n_experts]).
+ERB_EXPORT int erb_moe_route_few(int n_tokens, int n_experts, int top) {
+  return n_tokens <= 64 && n_tokens * top <= kRouteFewPairs && n_experts <= kRouteFewExperts;
+}
+
 ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n_tokens, int width, int n_experts, int top,
                              int* choice, float* score, int* counts, int* offsets, int* tiles, int* order, int tile_rows,
                              int score_kind, int n_groups, int keep_groups, const float* correction, int group_kind,
-                             int normalise, void* stream) {
+                             int normalise, float* logits, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   if (width <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || n_experts > 8192)
     return fail(ERB_ERR_ARG, "moe_route: %d of %d experts", top, n_experts);
@@ -344,6 +465,21 @@ ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n
     return fail(ERB_ERR_ARG, "moe_route: a correction and groups that count their two best go with sigmoid scores");
   cudaStream_t s = (cudaStream_t)stream;
   const int n_pairs = n_tokens * top;
+  if (logits && erb_moe_route_few(n_tokens, n_experts, top)) {
+    launch_chained(moe_logits_kernel<elem_t>, dim3((n_tokens + kRouteTokens - 1) / kRouteTokens, (n_experts + 3) / 4), dim3(128), 0, s,
+                   (const elem_t*)x, ld, w_router, n_tokens, width, n_experts, logits);
+    int rc = check_launch("moe_logits");
+    if (rc) return rc;
+    const size_t smem = sizeof(float) * (3 * (kRouteThreads / 32) + 2) * (size_t)((n_experts + 3) & ~3);
+    if (smem > 40 * 1024) {
+      cudaError_t err = cudaFuncSetAttribute(moe_choose_lists_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (err != cudaSuccess) return fail(ERB_ERR_CUDA, "moe_route: %s", cudaGetErrorString(err));
+    }
+    launch_chained(moe_choose_lists_kernel, dim3(1), dim3(kRouteThreads), smem, s, (const float*)logits, n_tokens, n_experts, top, choice,
+                   score, counts, offsets, tiles, order, tile_rows > 0 ? tile_rows : kTM, score_kind, n_groups, keep_groups, correction,
+                   group_kind, normalise);
+    return check_launch("moe_choose_lists");
+  }
   const size_t route_smem = sizeof(float) * kRouteTokens * (3 * (size_t)((n_experts + 3) & ~3) + width);
   if (route_smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(moe_route_kernel<elem_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)route_smem);

@@ -122,7 +122,7 @@ _SIGNATURES = {
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "erb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "erb_moe_route": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "erb_moe_tc_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "erb_moe_tc_gate_up": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                            c_void_p, c_void_p],
@@ -1406,9 +1406,16 @@ MOE_SCORES = {"sigmoid": 0, "softmax": 1}
 MOE_GROUP_SCORES = {"best": 0, "top2_sum": 1}
 
 
+@functools.lru_cache(maxsize=4096)
+def moe_route_few(n_tokens: int, n_experts: int, top: int, dtype: torch.dtype = torch.bfloat16) -> bool:
+    """Whether a step of this many tokens is routed by the pair of kernels for few tokens (``moe_route`` with ``logits``)."""
+    return bool(native.load("moe", _ELEM[dtype]).erb_moe_route_few(int(n_tokens), int(n_experts), int(top)))
+
+
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Tensor, score: torch.Tensor,
               tile_rows: int = 0, scores: str = "sigmoid", groups: tuple[int, int] | None = None,
-              correction: torch.Tensor | None = None, group_score: str = "best", normalise: bool = False) -> None:
+              correction: torch.Tensor | None = None, group_score: str = "best", normalise: bool = False,
+              logits: torch.Tensor | None = None) -> None:
     """Route every row of ``x`` (element type, row-strided view allowed): logits ``w_router x`` in float (``w_router``
     float ``[experts, width]``), the ``top`` largest chosen (the lower index wins a tie), ``score`` float ``[tokens *
     top]`` their sigmoids; ``lists`` (int32, ``moe_lists_ints`` entries) receives the choices and, per expert, the list
@@ -1419,7 +1426,11 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     only experts of the ``keep`` best groups can be chosen.  With ``correction`` (float ``[experts]``, sigmoid scores) the
     choice goes by score + correction, while ``score`` stays without it; ``group_score = "top2_sum"``: a group counts as
     much as the sum of its two best experts (in what the choice goes by); ``normalise``: the chosen scores are divided by
-    their sum (+ 1e-20)."""
+    their sum (+ 1e-20).  ``logits`` (float scratch ``[tokens, experts]``, where ``moe_route_few`` says so): the pair of
+    kernels for few tokens is used, with the same results to the bit."""
+    _need(logits, "logits", torch.float32)
+    if logits is not None and tuple(logits.shape) != (x.shape[0], w_router.shape[0]):
+        raise KernelError("moe_route: logits are [tokens, experts]")
     _need(correction, "correction", torch.float32)
     if correction is not None and correction.numel() != w_router.shape[0]:
         raise KernelError("moe_route: one correction per expert")
@@ -1436,7 +1447,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     _call(_fn("moe", _elem(x), "erb_moe_route"), x.data_ptr(), x.stride(0) if n > 1 else width, w_router.data_ptr(), n, width,
           n_experts, int(top), choice.data_ptr(), score.data_ptr(), counts.data_ptr(), offsets.data_ptr(), tiles.data_ptr(),
           order.data_ptr(), int(tile_rows), MOE_SCORES[scores], int(n_groups), int(keep), _ptr(correction),
-          MOE_GROUP_SCORES[group_score], int(bool(normalise)), _stream())
+          MOE_GROUP_SCORES[group_score], int(bool(normalise)),
+          _ptr(logits), _stream())
 
 
 def moe_tc_supported(dtype: torch.dtype, width: int, ff: int) -> bool:

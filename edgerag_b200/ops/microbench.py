@@ -553,7 +553,12 @@ def routed_experts(a) -> dict:
     if getattr(a, "corrected", False):
         how = dict(groups=tuple(a.groups) if getattr(a, "groups", None) else None, correction=torch.randn(E, device="cuda") * 0.3,
                    group_score="top2_sum", normalise=True)
+    if kernels.moe_route_few(n, E, top, dtype):
+        how_few = {"logits": torch.empty((n, E), device="cuda")}
+    else:
+        how_few = {}
     in_score, out_score = (None, score) if how else (score, None)
+    how.update(how_few)
     kernels.moe_route(x, router, top, lists, score, tile_rows, **how)
     used = int((lists[2 * n * top: 2 * n * top + E] > 0).sum())     # experts that some row chose
     us_route = _time(lambda: kernels.moe_route(x, router, top, lists, score, tile_rows, **how), a.iters, a.warmup)

@@ -103,6 +103,8 @@ class RoutedExperts(FeedForward):
         parts = ctx.buf("ffn.out_parts", (top + (self.shared is not None), n, self.hidden), torch.float32)
         route = dict(scores=self.scores, groups=self.groups, correction=self.correction, group_score=self.group_score,
                      normalise=self.normalise)
+        if kernels.moe_route_few(n, self.n_experts, top, self.dtype):
+            route["logits"] = ctx.buf("moe.logits", (n, self.n_experts), torch.float32)
         in_score, out_score = (score, None) if self.scale_input else (None, score)
         if kernels.moe_tc_supported(self.dtype, self.hidden, self.intermediate):
             # tensor cores: row tiles sized by the step's tokens, the (scaled) rows gathered once in list order

@@ -654,7 +654,7 @@ def test_router_with_correction_and_gated_experts_on_both_product_paths(sizes, d
     corr = torch.where(torch.rand(E, generator=g) < 0.5, -2.0, -1.0) + 0.3 * torch.randn(E, generator=g)
     w_gu = (torch.randn(E, 2 * ff, width, generator=g) / math.sqrt(width)).to(tdt)
     w_down = (torch.randn(E, width, ff, generator=g) / math.sqrt(ff)).to(tdt)
-    for n in (5, 200):
+    for n in (5, 64, 200):
         x = torch.randn(n, width, generator=g).to(tdt)
         s = torch.sigmoid(x.double() @ w_router.double().T)
         chosen = plain.routed_choice(x.double(), w_router, corr, router)
@@ -675,6 +675,15 @@ def test_router_with_correction_and_gated_experts_on_both_product_paths(sizes, d
         how = dict(groups=groups, correction=corr.float().cuda(), group_score="top2_sum", normalise=True)
         k.moe_route(x.cuda(), w_router.cuda(), top, lists, score, tile_rows, **how)
         got_c, got_s = lists[: n * top].reshape(n, top).cpu(), score.reshape(n, top).cpu()
+        if k.moe_route_few(n, E, top, tdt):           # the kernels for few tokens: the same choices, weights and lists to the bit
+            lists2, score2 = torch.zeros_like(lists), torch.zeros_like(score)
+            k.moe_route(x.cuda(), w_router.cuda(), top, lists2, score2, tile_rows, logits=torch.empty(n, E, device="cuda"), **how)
+            assert torch.equal(lists, lists2) and torch.equal(score, score2)
+            for scores, gr in (("sigmoid", groups), ("softmax", groups)):
+                k.moe_route(x.cuda(), w_router.cuda(), top, lists2, score2, tile_rows, scores=scores, groups=gr)
+                l3, s3 = torch.zeros_like(lists), torch.zeros_like(score)
+                k.moe_route(x.cuda(), w_router.cuda(), top, l3, s3, tile_rows, scores=scores, groups=gr, logits=torch.empty(n, E, device="cuda"))
+                assert torch.equal(l3, lists2) and torch.equal(s3, score2), scores
         assert torch.equal(got_c[clear].long(), chosen[clear]), "choices"
         assert torch.allclose(got_s[clear].double(), weight[clear], rtol=2e-5, atol=1e-7), "weights: the scores without correction, over their sum"
         want = torch.zeros(n, width, dtype=torch.float64)          # the update from the engine's own choices
