@@ -1682,9 +1682,32 @@ __global__ void sigmoid_gate_kernel(T* __restrict__ x, int ld_x, const T* __rest
     Elem<T>::store(row + i, Elem<T>::load(row + i) / (1.f + expf(-Elem<T>::load(g + i))));
 }
 
+// The same, four neighbouring entries a thread.
+template <typename T>
+__global__ void __launch_bounds__(256)
+sigmoid_gate_vec4_kernel(T* __restrict__ x, int ld_x, const T* __restrict__ gate, int ld_g, int groups, size_t total) {
+  chain_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / groups;
+    const int c = 4 * (int)(i - t * groups);
+    float v[4], g[4];
+    Pack4<T>::load(x + t * ld_x + c, v);
+    Pack4<T>::load(gate + t * ld_g + c, g);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v[k] = v[k] / (1.f + expf(-g[k]));
+    Pack4<T>::store(x + t * ld_x + c, v);
+  }
+}
+
 ERB_EXPORT int erb_sigmoid_gate(void* x, int ld_x, const void* gate, int ld_g, int n_rows, int width, void* stream) {
   if (n_rows <= 0 || width <= 0) return ERB_OK;
   if (ld_x < width || ld_g < width) return fail(ERB_ERR_ARG, "sigmoid_gate: strides must cover a row");
+  if (width % 4 == 0 && ld_x % 4 == 0 && ld_g % 4 == 0 && (((uintptr_t)x | (uintptr_t)gate) & 15) == 0) {
+    const size_t total = (size_t)n_rows * (width / 4), blocks = (total + 255) / 256;
+    launch_chained(sigmoid_gate_vec4_kernel<elem_t>, dim3((unsigned)(blocks < 148 * 32 ? blocks : 148 * 32)), dim3(256), 0,
+                   (cudaStream_t)stream, (elem_t*)x, ld_x, (const elem_t*)gate, ld_g, width / 4, total);
+    return check_launch("sigmoid_gate");
+  }
   int y = (width + 1023) / 1024;
   if (y > 64) y = 64;
   launch_chained(sigmoid_gate_kernel<elem_t>, dim3(n_rows, y), dim3(256), 0, (cudaStream_t)stream, (elem_t*)x, ld_x,

@@ -35,11 +35,36 @@ namespace {
 
 constexpr int kRouteThreads = 512;
 
-// A warp picks one token's experts from their logits z (shared or global memory): `choice` and `score` (the token's `top` entries).
-// cv and gm: shared memory for an entry per expert each.
-__device__ __forceinline__ void choose_experts(const float* z, float* cv, float* gm, int n_experts, int top, int* __restrict__ choice,
-                                               float* __restrict__ score, int score_kind, int n_groups, int keep_groups,
-                                               const float* __restrict__ correction, int group_kind, int normalise) {
+// Floats as unsigned numbers in the same order; what is no number counts as the least.
+__device__ __forceinline__ unsigned order_key(float v) {
+  if (v != v) return 0u;
+  const unsigned u = __float_as_uint(v);
+  return (u >> 31) ? ~u : u | 0x80000000u;
+}
+
+// The largest of keys[0 .. n) over the warp, the lower index on a tie (-1: all are zero); the winner's key becomes zero.
+__device__ __forceinline__ int take_largest(unsigned* keys, int n) {
+  const int lane = threadIdx.x & 31;
+  unsigned best = 0u;
+  int arg = 0x7fffffff;
+  for (int e = lane; e < n; e += 32) {
+    const unsigned k = keys[e];
+    if (k > best) { best = k; arg = e; }         // rising e within a lane: the first maximum stays
+  }
+  const unsigned top = __reduce_max_sync(0xffffffffu, best);
+  if (top == 0u) return -1;
+  const int winner = (int)__reduce_min_sync(0xffffffffu, best == top ? (unsigned)arg : 0x7fffffffu);
+  if ((winner & 31) == lane) keys[winner] = 0u;
+  __syncwarp();
+  return winner;
+}
+
+// A warp picks one token's experts from their logits z (shared memory): `choice` and `score` (the token's `top` entries; `pairs`,
+// if given, receives the choices too).  keys and gkeys: shared memory for an entry per expert each.
+__device__ __forceinline__ void choose_experts(const float* z, unsigned* keys, unsigned* gkeys, int n_experts, int top,
+                                               int* __restrict__ choice, float* __restrict__ score, int* pairs, int score_kind,
+                                               int n_groups, int keep_groups, const float* __restrict__ correction, int group_kind,
+                                               int normalise) {
   const int lane = threadIdx.x & 31;
   // softmax scores: the maximum and the denominator over all experts, before any expert is ruled out
   float z_top = 0.f, denom = 1.f;
@@ -53,9 +78,8 @@ __device__ __forceinline__ void choose_experts(const float* z, float* cv, float*
   }
   // What the choice goes by: the logits (the scores rise with them), or sigmoid scores plus correction.
   const bool by_score = correction != nullptr || group_kind == ERB_GROUP_TOP2_SUM;
-  for (int e = lane; e < n_experts; e += 32)
-    cv[e] = by_score ? 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f) : z[e];
-  __syncwarp();
+  auto value = [&](int e) { return by_score ? 1.f / (1.f + expf(-z[e])) + (correction ? correction[e] : 0.f) : z[e]; };
+  for (int e = lane; e < n_experts; e += 32) keys[e] = order_key(value(e));
   // groups of neighbouring experts: a group counts as much as its best expert or as the sum of its two best; the experts
   // of all but the `keep_groups` best groups are ruled out (the lower group wins a tie)
   if (n_groups > 1 && keep_groups < n_groups) {
@@ -63,66 +87,45 @@ __device__ __forceinline__ void choose_experts(const float* z, float* cv, float*
     for (int g = lane; g < n_groups; g += 32) {
       float mx = -INFINITY, second = -INFINITY;
       for (int e = g * per; e < (g + 1) * per; ++e) {
-        const float v = cv[e];
+        const float v = value(e);
         second = fmaxf(second, fminf(mx, v));
         mx = fmaxf(mx, v);
       }
-      gm[g] = group_kind == ERB_GROUP_TOP2_SUM && per > 1 ? mx + second : mx;
+      gkeys[g] = max(1u, order_key(group_kind == ERB_GROUP_TOP2_SUM && per > 1 ? mx + second : mx));
     }
     __syncwarp();
-    for (int c = 0; c < keep_groups; ++c) {
-      float best = -INFINITY;
-      int arg = 0x7fffffff;
-      for (int g = lane; g < n_groups; g += 32) {
-        const float v = gm[g];
-        if (v > best) { best = v; arg = g; }     // (a group already kept holds NaN: never greater)
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-      }
-      if (lane == 0 && arg < n_groups) gm[arg] = __int_as_float(0x7fc00000);
-      __syncwarp();
-    }
+    for (int c = 0; c < keep_groups; ++c) take_largest(gkeys, n_groups);
     for (int e = lane; e < n_experts; e += 32)
-      if (gm[e / per] == gm[e / per]) cv[e] = -INFINITY;      // not NaN: the group was not kept
-    __syncwarp();
+      if (gkeys[e / per] != 0u) keys[e] = 0u;                // (a group that was taken has the key zero)
   }
-  float total = 0.f;
+  __syncwarp();
+  float mine = 0.f, sum = 0.f;                               // of choice c, lane c % 32 keeps the score
   for (int c = 0; c < top; ++c) {
-    float best = -INFINITY;
-    int arg = 0x7fffffff;
-    for (int e = lane; e < n_experts; e += 32) {
-      const float zv = cv[e];
-      if (zv > best) { best = zv; arg = e; }     // rising e within a lane: the first maximum stays
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-      if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-    }
-    if (arg >= n_experts) arg = c;                // (no expert compares: logits that are no numbers; any choice does)
-    if (lane == 0) {
-      const float s = score_kind == ERB_SCORE_SOFTMAX ? expf(z[arg] - z_top) / denom : 1.f / (1.f + expf(-z[arg]));
+    int arg = take_largest(keys, n_experts);
+    if (arg < 0) arg = c;                                    // (no expert compares: logits that are no numbers; any choice does)
+    if ((c & 31) == lane) {
+      mine = score_kind == ERB_SCORE_SOFTMAX ? expf(z[arg] - z_top) / denom : 1.f / (1.f + expf(-z[arg]));
+      sum += mine;
       choice[c] = arg;
-      score[c] = s;
-      cv[arg] = -INFINITY;
-      total += s;
+      if (pairs) pairs[c] = arg;
+      if (!normalise || top > 32) score[c] = mine;
     }
-    __syncwarp();
   }
-  if (normalise && lane == 0)
-    for (int c = 0; c < top; ++c) score[c] /= total + 1e-20f;
+  if (!normalise) return;
+  const float total = warp_sum(sum) + 1e-20f;
+  if (top <= 32) {
+    if (lane < top) score[lane] = mine / total;
+  } else {
+    for (int c = lane; c < top; c += 32) score[c] /= total;
+  }
 }
 
 // One block per kRouteTokens tokens.  Shared memory: their logits, then their rows as floats.  A warp takes an expert at
 // a time and reads its router row once for all the block's tokens; a lane sums the entries 4 lane .. 4 lane + 3 of every
 // run of 128, then the lanes are added: one order of sums per token whatever the batch.  Then a warp per token picks.
 constexpr int kRouteTokens = 4;
-constexpr int kRouteFewPairs = 512, kRouteFewExperts = 256;   // up to which one block picks and makes the lists
+// up to which one block picks and makes the lists (one token a warp: from 32 tokens on the other kernels are as fast)
+constexpr int kRouteFewTokens = 16, kRouteFewPairs = 512, kRouteFewExperts = 256;
 template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_router, int n_tokens, int width, int n_experts,
@@ -176,8 +179,9 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
   if (warp >= n_here) return;
   const int t = t0 + warp;
   float* z = z_s + warp * e_pad;
-  choose_experts(z, c_s + warp * e_pad, g_s + warp * e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, score_kind,
-                 n_groups, keep_groups, correction, group_kind, normalise);
+  choose_experts(z, reinterpret_cast<unsigned*>(c_s) + warp * e_pad, reinterpret_cast<unsigned*>(g_s) + warp * e_pad, n_experts, top,
+                 choice + (size_t)t * top, score + (size_t)t * top, nullptr, score_kind, n_groups, keep_groups, correction, group_kind,
+                 normalise);
 }
 
 // One block per expert e builds the expert's part of the lists on its own: a histogram of all choices in shared memory
@@ -252,7 +256,7 @@ moe_logits_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_r
   }
   const bool pack = ((uintptr_t)x & 15) == 0 && (ld & 3) == 0;
   const int whole = (width & 3) == 0 && pack ? width & ~127 : 0;
-#pragma unroll 4
+#pragma unroll 8
   for (int k = 4 * lane; k < whole; k += 128) {
     const float4 wv = *reinterpret_cast<const float4*>(w + k);
 #pragma unroll
@@ -283,8 +287,8 @@ moe_logits_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_r
   }
 }
 
-// ... and one block picks for all of them, a warp a token at a time, and builds the lists: thread e walks the pairs (parked in
-// shared memory) for expert e, so an expert's pairs come out in rising order as in moe_lists_kernel.
+// ... and one block picks for all of them, a warp a token at a time, and builds the lists: the first warp walks the pairs (parked
+// in shared memory) 32 at a time in rising order, so an expert's pairs come out in rising order as in moe_lists_kernel.
 __global__ void __launch_bounds__(kRouteThreads)
 moe_choose_lists_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top, int* __restrict__ choice,
                         float* __restrict__ score, int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ tiles,
@@ -298,43 +302,49 @@ moe_choose_lists_kernel(const float* __restrict__ logits, int n_tokens, int n_ex
   int* count_s = reinterpret_cast<int*>(z_s + 3 * kWarps * e_pad);      // [n_experts], then [n_experts] offsets
   int* off_s = count_s + e_pad;
   float* z = z_s + 3 * warp * e_pad;
+  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count_s[e] = 0;
   for (int t = warp; t < n_tokens; t += kWarps) {
     for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * n_experts + e];
     __syncwarp();
-    choose_experts(z, z + e_pad, z + 2 * e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, score_kind, n_groups,
-                   keep_groups, correction, group_kind, normalise);
-    __syncwarp();
-    for (int c = lane; c < top; c += 32) pair_s[t * top + c] = choice[(size_t)t * top + c];
+    unsigned* keys = reinterpret_cast<unsigned*>(z + e_pad);
+    choose_experts(z, keys, keys + e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, pair_s + t * top, score_kind,
+                   n_groups, keep_groups, correction, group_kind, normalise);
     __syncwarp();
   }
   __syncthreads();
   const int n_pairs = n_tokens * top;
-  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
-    int n = 0;
-#pragma unroll 4
-    for (int i = 0; i < n_pairs; ++i) n += pair_s[i] == e;
-    count_s[e] = n;
-  }
+  for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) atomicAdd(&count_s[pair_s[i]], 1);
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (warp != 0) return;
+  {                                               // running sums over the experts, 32 at a time
     int off = 0, tl = 0;
-    for (int e = 0; e < n_experts; ++e) {
-      counts[e] = count_s[e];
-      offsets[e] = off_s[e] = off;
-      tiles[e] = tl;
-      off += count_s[e];
-      tl += (count_s[e] + tile_rows - 1) / tile_rows;
+    for (int e0 = 0; e0 < n_experts; e0 += 32) {
+      const int e = e0 + lane, n = e < n_experts ? count_s[e] : 0, t = (n + tile_rows - 1) / tile_rows;
+      int on = n, ot = t;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, on, d), b = __shfl_up_sync(0xffffffffu, ot, d);
+        if (lane >= d) { on += a; ot += b; }
+      }
+      if (e < n_experts) {
+        counts[e] = n;
+        offsets[e] = off_s[e] = off + on - n;
+        tiles[e] = tl + ot - t;
+      }
+      off += __shfl_sync(0xffffffffu, on, 31);
+      tl += __shfl_sync(0xffffffffu, ot, 31);
     }
-    offsets[n_experts] = off;
-    tiles[n_experts] = tl;
-    counts[n_experts] = 0;
+    if (lane == 0) { offsets[n_experts] = off; tiles[n_experts] = tl; counts[n_experts] = 0; }
   }
-  __syncthreads();
-  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
-    int at = off_s[e];
-    const int stop = at + count_s[e];
-    for (int i = 0; at < stop; ++i)
-      if (pair_s[i] == e) order[at++] = i;
+  __syncwarp();
+  for (int i0 = 0; i0 < n_pairs; i0 += 32) {
+    const int i = i0 + lane, e = i < n_pairs ? pair_s[i] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    const int before = __popc(same & ((1u << lane) - 1u));
+    if (e >= 0) order[off_s[e] + before] = i;
+    __syncwarp();
+    if (e >= 0 && before == 0) off_s[e] += __popc(same);
+    __syncwarp();
   }
 }
 
@@ -446,7 +456,7 @@ ERB_EXPORT int erb_moe_tile_rows() { return kTM; }
 
 // Whether a step of this many tokens is routed by the pair of kernels for few tokens (then `logits` is [n_tokens][n_experts]).
 ERB_EXPORT int erb_moe_route_few(int n_tokens, int n_experts, int top) {
-  return n_tokens <= 64 && n_tokens * top <= kRouteFewPairs && n_experts <= kRouteFewExperts;
+  return n_tokens <= kRouteFewTokens && n_tokens * top <= kRouteFewPairs && n_experts <= kRouteFewExperts;
 }
 
 ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n_tokens, int width, int n_experts, int top,

@@ -654,7 +654,7 @@ def test_router_with_correction_and_gated_experts_on_both_product_paths(sizes, d
     corr = torch.where(torch.rand(E, generator=g) < 0.5, -2.0, -1.0) + 0.3 * torch.randn(E, generator=g)
     w_gu = (torch.randn(E, 2 * ff, width, generator=g) / math.sqrt(width)).to(tdt)
     w_down = (torch.randn(E, width, ff, generator=g) / math.sqrt(ff)).to(tdt)
-    for n in (5, 64, 200):
+    for n in (5, 16, 200):
         x = torch.randn(n, width, generator=g).to(tdt)
         s = torch.sigmoid(x.double() @ w_router.double().T)
         chosen = plain.routed_choice(x.double(), w_router, corr, router)
@@ -782,6 +782,9 @@ def test_layer_norm_without_bias_and_entrywise_gate(dtype):
         got = y.clone().cuda()
         k.sigmoid_gate(got, z.cuda()[:, width:])
         assert (got.double().cpu() - y.double() * torch.sigmoid(z.double()[:, width:])).abs().max() < tol * 3
+        got = y.clone().cuda()
+        k.sigmoid_gate(got, z.cuda()[:, 2: width + 2])                  # (a view that is not 16-byte aligned)
+        assert (got.double().cpu() - y.double() * torch.sigmoid(z.double()[:, 2: width + 2])).abs().max() < tol * 3
 
 
 @pytest.mark.gpu
