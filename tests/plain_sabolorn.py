@@ -301,17 +301,22 @@ def moe_mlp(ff=16, experts=6, top=2, groups=(3, 2)) -> dict:
 
 
 def make_config(layers: list[dict], width=32, vocab=97, eps=1e-5, scale=3.0, side=8, softcap=9.0) -> dict:
-    return {"architecture": "Sabolorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale},
-            "token_side": {"dim": side}, "logit_softcap": softcap, "layers": layers}
+    out = {"architecture": "Sabolorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": scale},
+           "logit_softcap": softcap, "layers": layers}
+    return {**out, "token_side": {"dim": side}} if side else out
 
 
 def tensor_shapes(cfg: dict) -> dict[str, tuple[int, ...]]:
-    W, S, n = cfg["width"], cfg["token_side"]["dim"], len(cfg["layers"])
-    shapes: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], W), "final.norm": (W,), "side.embed": (cfg["vocab"], n * S)}
+    W, S, n = cfg["width"], (cfg.get("token_side") or {}).get("dim", 0), len(cfg["layers"])
+    shapes: dict[str, tuple[int, ...]] = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
+    if S:
+        shapes["side.embed"] = (cfg["vocab"], n * S)
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.", layer["mixer"]
         x = p + "mix."
-        shapes.update({p + "norm1": (W,), p + "dwa": (i + 2,), p + "side.gate": (S, W), p + "side.proj": (W, S), p + "side.norm": (W,)})
+        shapes.update({p + "norm1": (W,), p + "dwa": (i + 2,)})
+        if S:
+            shapes.update({p + "side.gate": (S, W), p + "side.proj": (W, S), p + "side.norm": (W,)})
         if layer["type"] == "mamba2":
             H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
             ch = H * P + 2 * G * N
