@@ -58,11 +58,13 @@ class KVGroupSpec:
 
 @dataclass(frozen=True)
 class StateSpec:
-    """A per-request record of fixed size kept by a mixer (``shape`` per request, float32 unless said)."""
+    """A per-request record of fixed size kept by a part (``shape`` per request, float32 unless said)."""
 
     name: str
     shape: tuple[int, ...]
     dtype: str = "float32"
+    #: the part leaves rows with a negative state slot alone, so that a step may hold filler rows
+    fillers: bool = False
 
 
 @dataclass

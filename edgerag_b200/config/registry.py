@@ -81,6 +81,9 @@ def _register_builtin() -> None:
     from ..models.sabolorn import SabolornConfig, sabolorn_plan
 
     register_architecture(["Sabolorn", "sabolorn"], SabolornConfig.from_dict, sabolorn_plan)
+    from ..models.kikarax import KikaraxConfig, kikarax_plan
+
+    register_architecture(["Kikarax", "kikarax"], KikaraxConfig.from_dict, kikarax_plan)
 
 
 _register_builtin()

@@ -11,7 +11,9 @@
 // distance.  A negative `window` stands for a mask of chunks: the query sees the keys from the start of its own run of
 // -window positions (runs counted from position 0 of the sequence) up to itself.  Query head h reads kv head h / (nq / nkv).
 // With `penalty` (float [2][nq]: r1 of every query head, then r2) the scaled score of a key d positions back is lowered by
-// r1 * ln(1 + r2 * d).
+// r1 * ln(1 + r2 * d).  With `softcap` c > 0 the scaled score s becomes c * tanh(s / c); a launch takes one of the two.
+// With `gate` (rows of nq * D entries, `gate_stride` apart, row t for output row t) every output entry is multiplied by the
+// sigmoid of its entry of the gate before it is rounded.
 //
 // Both kernels give every thread its own keys and its own online-softmax state (running max,
 // denominator, float accumulator of D values), so the inner loop has no cross-thread traffic;
@@ -48,7 +50,7 @@ struct LaneState {
   }
   // Visit one key: k and v point at the D elements of the key and the value row.
   template <typename T>
-  __device__ __forceinline__ void visit(const float* q_smem, const T* k, const T* v, float scale, float lower) {
+  __device__ __forceinline__ void visit(const float* q_smem, const T* k, const T* v, float scale, float lower, float softcap) {
     constexpr int N = Vec<T>::N;
     float s = 0.f;
 #pragma unroll
@@ -59,6 +61,7 @@ struct LaneState {
       for (int i = 0; i < N; ++i) s = fmaf(q_smem[d0 + i], kk[i], s);
     }
     s = fmaf(s, scale, -lower);
+    if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     float p;
     if (s > m) {
       const float alpha = expf(m - s);  // exp(-inf) = 0 on the first key
@@ -129,7 +132,8 @@ attention_rows_kernel(const T* __restrict__ q, int q_row_stride, const T* __rest
                       const T* __restrict__ v_pages, const int* __restrict__ block_tables, int max_pages,
                       const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                       T* __restrict__ out, int out_row_stride, int n_tokens, int nq, int nkv,
-                      int page_size, int window, int keep_first, float scale, const float* __restrict__ penalty) {
+                      int page_size, int window, int keep_first, float scale, const float* __restrict__ penalty, float softcap,
+                      const T* __restrict__ gate, int gate_stride) {
   chain_wait();
   extern __shared__ float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -154,12 +158,12 @@ attention_rows_kernel(const T* __restrict__ q, int q_row_stride, const T* __rest
   for (int k = lane; k < kept; k += 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k), softcap);
   }
   for (int k = k_lo + lane; k <= pos; k += 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k), softcap);
   }
   float m_w, l_w, o[(D + 31) / 32];
   warp_merge<D>(st, stage, m_w, l_w, o);
@@ -168,7 +172,7 @@ attention_rows_kernel(const T* __restrict__ q, int q_row_stride, const T* __rest
 #pragma unroll
   for (int i = 0; i < (D + 31) / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) Elem<T>::store(o_row + d, o[i] * inv);
+    if (d < D) Elem<T>::store(o_row + d, gate ? sigmoid_mul(o[i] * inv, Elem<T>::load(gate + (size_t)t * gate_stride + h * D + d)) : o[i] * inv);
   }
 }
 
@@ -188,7 +192,8 @@ attention_decode_split_kernel(const T* __restrict__ q, int q_row_stride, const T
                               int max_pages, const int* __restrict__ token_of_seq,
                               const int* __restrict__ positions, float* __restrict__ part_acc,
                               float* __restrict__ part_ml, int max_splits, int nq, int nkv, int page_size,
-                              int window, int keep_first, int split_keys, float scale, const float* __restrict__ penalty) {
+                              int window, int keep_first, int split_keys, float scale, const float* __restrict__ penalty,
+                              float softcap) {
   chain_wait();
   extern __shared__ float smem[];
   float* q_s = smem;                                   // D
@@ -218,12 +223,12 @@ attention_decode_split_kernel(const T* __restrict__ q, int q_row_stride, const T
   for (int k = (int)threadIdx.x; k < kept; k += kDecodeWarps * 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k), softcap);
   }
   for (int k = begin + (int)threadIdx.x; k < end; k += kDecodeWarps * 32) {
     const int page = bt[k / page_size];
     const size_t row = (((size_t)page * nkv + kvh) * page_size + (k % page_size)) * D;
-    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k));
+    st.template visit<T>(q_s, k_pages + row, v_pages + row, scale, pen.at(pos - k), softcap);
   }
   float m_w, l_w, o[(D + 31) / 32];
   warp_merge<D>(st, stage + warp * 32 * (D + 1), m_w, l_w, o);
@@ -269,7 +274,7 @@ __global__ void attention_decode_combine_kernel(const float* __restrict__ part_a
                                                 const int* __restrict__ token_of_seq,
                                                 const int* __restrict__ positions, T* __restrict__ out,
                                                 int out_row_stride, int max_splits, int nq, int head_dim,
-                                                int window, int split_keys) {
+                                                int window, int split_keys, const T* __restrict__ gate, int gate_stride) {
   chain_wait();
   const int h = blockIdx.x, seq = blockIdx.y;
   const int t = token_of_seq[seq];
@@ -289,7 +294,7 @@ __global__ void attention_decode_combine_kernel(const float* __restrict__ part_a
     float sum = 0.f;
     for (int s = 0; s < n_splits; ++s)
       sum += part_acc[(base + s) * head_dim + d] * expf(part_ml[(base + s) * 2] - m);
-    Elem<T>::store(o_row + d, sum * inv);
+    Elem<T>::store(o_row + d, gate ? sigmoid_mul(sum * inv, Elem<T>::load(gate + (size_t)t * gate_stride + h * head_dim + d)) : sum * inv);
   }
 }
 
@@ -297,7 +302,7 @@ template <typename T, int D>
 int launch_rows(const void* q, int q_row_stride, const void* k_pages, const void* v_pages,
                 const int* block_tables, int max_pages, const int* seq_of_token, const int* positions,
                 void* out, int out_row_stride, int n_tokens, int nq, int nkv, int page_size, int window,
-                int keep_first, float scale, const float* penalty, cudaStream_t s) {
+                int keep_first, float scale, const float* penalty, float softcap, const void* gate, int gate_stride, cudaStream_t s) {
   const size_t smem = (size_t)(kRowWarps * D + kRowWarps * 32 * (D + 1)) * sizeof(float);
   auto kern = attention_rows_kernel<T, D>;
   if (smem > 48 * 1024) {
@@ -307,7 +312,7 @@ int launch_rows(const void* q, int q_row_stride, const void* k_pages, const void
   dim3 grid((n_tokens + kRowWarps - 1) / kRowWarps, nq);
   launch_chained(kern, dim3(grid), dim3(kRowWarps * 32), smem, s, (const T*)q, q_row_stride, (const T*)k_pages, (const T*)v_pages,
       block_tables, max_pages, seq_of_token, positions, (T*)out, out_row_stride, n_tokens, nq, nkv,
-      page_size, window, keep_first, scale, penalty);
+      page_size, window, keep_first, scale, penalty, softcap, (const T*)gate, gate_stride);
   return check_launch("attention_rows");
 }
 
@@ -315,7 +320,8 @@ template <typename T, int D>
 int launch_decode(const void* q, int q_row_stride, const void* k_pages, const void* v_pages,
                   const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                   void* out, int out_row_stride, float* part_acc, float* part_ml, int max_splits, int n_seqs,
-                  int nq, int nkv, int page_size, int window, int keep_first, int split_keys, float scale, const float* penalty, cudaStream_t s) {
+                  int nq, int nkv, int page_size, int window, int keep_first, int split_keys, float scale, const float* penalty,
+                  float softcap, const void* gate, int gate_stride, cudaStream_t s) {
   const size_t smem =
       (size_t)(D + kDecodeWarps * 32 * (D + 1) + kDecodeWarps * (D + 2)) * sizeof(float);
   auto kern = attention_decode_split_kernel<T, D>;
@@ -326,11 +332,11 @@ int launch_decode(const void* q, int q_row_stride, const void* k_pages, const vo
   dim3 grid(max_splits, nq, n_seqs);
   launch_chained(kern, dim3(grid), dim3(kDecodeWarps * 32), smem, s, (const T*)q, q_row_stride, (const T*)k_pages,
       (const T*)v_pages, block_tables, max_pages, token_of_seq, positions, part_acc, part_ml, max_splits,
-      nq, nkv, page_size, window, keep_first, split_keys, scale, penalty);
+      nq, nkv, page_size, window, keep_first, split_keys, scale, penalty, softcap);
   int rc = check_launch("attention_decode_split");
   if (rc) return rc;
   launch_chained(attention_decode_combine_kernel<T>, dim3(dim3(nq, n_seqs)), dim3(64), 0, s, part_acc, part_ml, token_of_seq,
-      positions, (T*)out, out_row_stride, max_splits, nq, D, window, split_keys);
+      positions, (T*)out, out_row_stride, max_splits, nq, D, window, split_keys, (const T*)gate, gate_stride);
   return check_launch("attention_decode_combine");
 }
 
@@ -366,13 +372,15 @@ ERB_EXPORT int erb_attention_rows(const void* q, int q_row_stride, const void* k
                                   const int* block_tables, int max_pages, const int* seq_of_token,
                                   const int* positions, void* out, int out_row_stride, int n_tokens, int nq,
                                   int nkv, int head_dim, int page_size, int window, int keep_first, float scale,
-                                  const float* penalty, void* stream) {
+                                  const float* penalty, float softcap, const void* gate, int gate_stride, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
+  if (penalty && softcap > 0.f) return fail(ERB_ERR_UNSUPPORTED, "attention_rows: a penalty and a cap of the scores exclude each other");
   int rc = check_common("attention_rows", nq, nkv, head_dim, page_size, max_pages);
   if (rc) return rc;
   cudaStream_t s = (cudaStream_t)stream;
   ERB_DISPATCH_D(launch_rows, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, seq_of_token,
-                 positions, out, out_row_stride, n_tokens, nq, nkv, page_size, window, window > 0 ? keep_first : 0, scale, penalty, s)
+                 positions, out, out_row_stride, n_tokens, nq, nkv, page_size, window, window > 0 ? keep_first : 0, scale, penalty,
+                 softcap, gate, gate_stride, s)
   return fail(ERB_ERR_UNSUPPORTED, "attention_rows: head_dim %d", head_dim);
 }
 
@@ -384,8 +392,10 @@ ERB_EXPORT int erb_attention_decode(const void* q, int q_row_stride, const void*
                                     const int* token_of_seq, const int* positions, void* out,
                                     int out_row_stride, float* part_acc, float* part_ml, int max_splits,
                                     int n_seqs, int nq, int nkv, int head_dim, int page_size, int window,
-                                    int keep_first, int split_keys, float scale, const float* penalty, void* stream) {
+                                    int keep_first, int split_keys, float scale, const float* penalty, float softcap,
+                                    const void* gate, int gate_stride, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
+  if (penalty && softcap > 0.f) return fail(ERB_ERR_UNSUPPORTED, "attention_decode: a penalty and a cap of the scores exclude each other");
   int rc = check_common("attention_decode", nq, nkv, head_dim, page_size, max_pages);
   if (rc) return rc;
   if (max_splits <= 0 || split_keys <= 0 || !part_acc || !part_ml)
@@ -394,7 +404,7 @@ ERB_EXPORT int erb_attention_decode(const void* q, int q_row_stride, const void*
   cudaStream_t s = (cudaStream_t)stream;
   ERB_DISPATCH_D(launch_decode, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                  positions, out, out_row_stride, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size,
-                 window, window > 0 ? keep_first : 0, split_keys, scale, penalty, s)
+                 window, window > 0 ? keep_first : 0, split_keys, scale, penalty, softcap, gate, gate_stride, s)
   return fail(ERB_ERR_UNSUPPORTED, "attention_decode: head_dim %d", head_dim);
 }
 
@@ -457,5 +467,5 @@ ERB_EXPORT int erb_attention_decode_static(const void* q, int q_row_stride, cons
   float* part_ml = base + (size_t)n_seqs * nq * max_splits * head_dim;
   return erb_attention_decode(q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                               positions, out, out_row_stride, part_acc, part_ml, max_splits, n_seqs, nq, nkv,
-                              head_dim, page_size, window, 0, split_keys, scale, nullptr, stream);
+                              head_dim, page_size, window, 0, split_keys, scale, nullptr, 0.f, nullptr, 0, stream);
 }

@@ -37,6 +37,14 @@
 // unit that also makes the exponentials; so where every key of a tile is far from every row, the logarithm is taken once
 // for 16 neighbouring keys, at their middle, and continued to the others by the first three terms of its series.
 //
+// With a cap of the scores (`softcap` c > 0) the scaled score s becomes c * tanh(s / c), again in a form of the kernel of its
+// own.  The exact form takes two more operations of the unit that makes the exponentials; so 16 neighbouring scores of a warp's
+// rows that are all below the cap take a polynomial of tanh on the multipliers instead (relative error below 1e-6, as the
+// exact form's).  The cap is monotonic: a search for a maximum looks at the scores as they are and caps what it found.
+//
+// With `gate` (row t, `gate_stride` apart, nq * 64 entries, for output row t) every output entry is multiplied by the sigmoid of
+// its entry of the gate before it is rounded.
+//
 // Every wait is bounded: a thread that gives up raises a block-wide flag, every other wait of the
 // block then ends too, the block records a code in *status, lets its copies land, frees its TMEM
 // and returns.
@@ -83,7 +91,13 @@ constexpr float kSumLimit = 1048576.f;   // a tile's sum of P from which on the 
 constexpr uint32_t kIdescS = mma_idesc(BM, BN, false);
 constexpr uint32_t kIdescO = mma_idesc(BM, HD, true);
 
-template <bool PEN>
+// What is done to a scaled score before the softmax.
+constexpr int kScorePlain = 0, kScorePenalty = 1, kScoreCap = 2;
+// tanh(x) = x (t0 + t1 y + ... + t5 y^5), y = x^2 <= 1: the minimax polynomial of tanh(x) / x in y (relative error 6e-7)
+constexpr float kTanh0 = 0.99999941f, kTanh1 = -0.33329042f, kTanh2 = 0.13281434f, kTanh3 = -0.051605674f, kTanh4 = 0.016743115f,
+                kTanh5 = -0.0030670603f;
+
+template <int SCORE>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                          const __nv_bfloat16* __restrict__ q, int q_row_stride,
@@ -91,7 +105,10 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
                          const int* __restrict__ positions, __nv_bfloat16* __restrict__ out, int out_row_stride,
                          int n_seqs, int nq, int nkv, int page_size, float scale_log2, int* __restrict__ status,
                          int key_splits, float* __restrict__ part_o, float* __restrict__ part_ml, int window, int keep_first,
-                         const float* __restrict__ penalty) {
+                         const float* __restrict__ penalty, float cap_in, float cap_out, const __nv_bfloat16* __restrict__ gate,
+                         int gate_stride) {
+  // cap_in: the raw score's factor to x = s / c; cap_out: c log2(e)
+  constexpr bool PEN = SCORE == kScorePenalty, CAP = SCORE == kScoreCap;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;             // the swizzle repeats every 1024 bytes
@@ -363,7 +380,9 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           named_barrier(pair_barrier, 64);
           // (scale > 0: the maximum of the scaled scores.  A range of keys may begin with a tile of which a row
           // sees nothing: its reference then stays at a finite floor, so that exp2(-inf - reference) is 0, not NaN.)
-          const float m_tile = fmaxf(fmaxf(m_half, *partners) * (PEN ? 1.f : scale_log2), -1e30f);
+          const float m_raw = fmaxf(m_half, *partners);
+          const float m_tile = CAP ? capped_score(m_raw * (cap_in * 2.8853900817779268f), cap_out)
+                                   : fmaxf(m_raw * (PEN ? 1.f : scale_log2), -1e30f);
           float alpha = 1.f;
           if (m_tile > m_ref) {
             alpha = fast_exp2(m_ref - m_tile);                          // 0 on the first tile
@@ -411,6 +430,28 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
             for (int i = 0; i < 16; ++i) sc[i] = fmaf(sc[i], scale_log2, -lower(at0, 16 * c + i) - m_ref);
           }
+          if (CAP) {
+            float big = 0.f;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) big = fmaxf(big, fabsf(sc[i]));
+            if (__any_sync(0xffffffffu, !(big * cap_in <= 1.f))) {
+              const float x_in = cap_in * 2.8853900817779268f;
+#pragma unroll
+              for (int i = 0; i < 16; ++i) sc[i] = capped_score(sc[i] * x_in, cap_out) - m_ref;
+            } else {
+              const float out = cap_in * cap_out;
+#pragma unroll
+              for (int i = 0; i < 16; ++i) {
+                const float x = sc[i] * cap_in, y = x * x;
+                float p = fmaf(kTanh5, y, kTanh4);
+                p = fmaf(p, y, kTanh3);
+                p = fmaf(p, y, kTanh2);
+                p = fmaf(p, y, kTanh1);
+                p = fmaf(p, y, kTanh0);
+                sc[i] = fmaf(sc[i] * out, p, -m_ref);
+              }
+            }
+          }
           if (diagonal) {
 #pragma unroll
             for (int i = 0; i < 16; ++i)
@@ -418,8 +459,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           }
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            const float p0 = fast_exp2(PEN ? sc[2 * i] : fmaf(sc[2 * i], scale_log2, -m_ref));
-            const float p1 = fast_exp2(PEN ? sc[2 * i + 1] : fmaf(sc[2 * i + 1], scale_log2, -m_ref));
+            const float p0 = fast_exp2(PEN || CAP ? sc[2 * i] : fmaf(sc[2 * i], scale_log2, -m_ref));
+            const float p1 = fast_exp2(PEN || CAP ? sc[2 * i + 1] : fmaf(sc[2 * i + 1], scale_log2, -m_ref));
             l4[i & 3] += p0 + p1;
             __nv_bfloat162 b = __floats2bfloat162_rn(p0, p1);
             packed[8 * c + i] = *reinterpret_cast<uint32_t*>(&b);
@@ -471,12 +512,24 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
         tmem_ld32(t_o, acc);
         tmem_ld_wait();
         if (row < rows_t[t]) {
+          const __nv_bfloat16* g_row = gate ? gate + (size_t)(q0 + t * BM + row) * gate_stride + h * HD + half * 32 : nullptr;
+#pragma unroll
+          for (int d = 0; d < 32; ++d) acc[d] *= inv;
+          if (g_row) {
+#pragma unroll
+            for (int d = 0; d < 32; d += 8) {
+              float z[8];
+              load8(g_row + d, z);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) acc[d + i] = sigmoid_mul(acc[d + i], z[i]);
+            }
+          }
 #pragma unroll
           for (int d = 0; d < 32; d += 8) {
             uint32_t w[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-              __nv_bfloat162 b = __floats2bfloat162_rn(acc[d + 2 * i] * inv, acc[d + 2 * i + 1] * inv);
+              __nv_bfloat162 b = __floats2bfloat162_rn(acc[d + 2 * i], acc[d + 2 * i + 1]);
               w[i] = *reinterpret_cast<uint32_t*>(&b);
             }
             *reinterpret_cast<uint4*>(dst + d) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -508,7 +561,8 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 // range that saw no key has sum 0.  One warp per (token, head), a lane for two neighbouring elements.
 __global__ void __launch_bounds__(128)
 attention_prefill_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
-                               int out_row_stride, int first_row, int n_rows, int nq, int key_splits) {
+                               int out_row_stride, int first_row, int n_rows, int nq, int key_splits,
+                               const __nv_bfloat16* __restrict__ gate, int gate_stride) {
   chain_wait();
   const int pair = (int)(blockIdx.x * 4 + (threadIdx.x >> 5)), lane = threadIdx.x & 31;
   if (pair >= n_rows * nq) return;
@@ -527,7 +581,14 @@ attention_prefill_merge_kernel(const float* __restrict__ part_o, const float* __
     o1 += o.y * w;
   }
   const float inv = 1.f / l;
-  *reinterpret_cast<__nv_bfloat162*>(out + (size_t)row * out_row_stride + (size_t)h * HD + 2 * lane) = __floats2bfloat162_rn(o0 * inv, o1 * inv);
+  o0 *= inv;
+  o1 *= inv;
+  if (gate) {
+    const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)row * gate_stride + h * HD + 2 * lane));
+    o0 = sigmoid_mul(o0, z.x);
+    o1 = sigmoid_mul(o1, z.y);
+  }
+  *reinterpret_cast<__nv_bfloat162*>(out + (size_t)row * out_row_stride + (size_t)h * HD + 2 * lane) = __floats2bfloat162_rn(o0, o1);
 }
 
 }  // namespace
@@ -556,8 +617,10 @@ ERB_EXPORT int erb_attention_prefill_tc(const void* q, int q_row_stride, const v
                                         int n_seqs, int n_blocks, int nq, int nkv, int head_dim, int page_size,
                                         float scale, int* status, int key_splits, int first_row, int n_rows,
                                         float* part_o, float* part_ml, int window, int keep_first, const float* penalty,
-                                        void* stream) {
+                                        float softcap, const void* gate, int gate_stride, void* stream) {
   if (n_seqs <= 0 || n_blocks <= 0) return ERB_OK;
+  if (penalty && softcap > 0.f) return fail(ERB_ERR_UNSUPPORTED, "attention_prefill_tc: a penalty and a cap of the scores exclude each other");
+  if (gate && (gate_stride % 8 || ((uintptr_t)gate & 15))) return fail(ERB_ERR_UNSUPPORTED, "attention_prefill_tc: gate rows must be 16-byte aligned");
   if (key_splits < 1 || key_splits > 64 || (key_splits > 1 && (!part_o || !part_ml || first_row < 0 || n_rows <= 0 || ((uintptr_t)part_o & 15))))
     return fail(ERB_ERR_ARG, "attention_prefill_tc: bad split arguments");
   if (!erb_attention_prefill_tc_supported(head_dim, page_size))
@@ -576,20 +639,24 @@ ERB_EXPORT int erb_attention_prefill_tc(const void* q, int q_row_stride, const v
   if ((rc = pool_map(&mk, k_pages, pool_rows, (unsigned)page_size, "attention_prefill_tc")) ||
       (rc = pool_map(&mv, v_pages, pool_rows, (unsigned)page_size, "attention_prefill_tc")))
     return rc;
-  auto kern = penalty ? attention_prefill_kernel<true> : attention_prefill_kernel<false>;
-  static bool configured[2] = {false, false};
-  if (!configured[penalty != nullptr]) {
+  const int score = penalty ? kScorePenalty : softcap > 0.f ? kScoreCap : kScorePlain;
+  auto kern = score == kScorePenalty ? attention_prefill_kernel<kScorePenalty>
+              : score == kScoreCap   ? attention_prefill_kernel<kScoreCap>
+                                     : attention_prefill_kernel<kScorePlain>;
+  static bool configured[3] = {false, false, false};
+  if (!configured[score]) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemBytes);
     if (e != cudaSuccess) return fail(ERB_ERR_CUDA, "attention_prefill_tc: %s", cudaGetErrorString(e));
-    configured[penalty != nullptr] = true;
+    configured[score] = true;
   }
   const float scale_log2 = scale * 1.4426950408889634f;
   launch_chained(kern, dim3(nq, n_blocks, key_splits), dim3(kThreads), kSmemBytes, (cudaStream_t)stream, mk, mv,
                  (const __nv_bfloat16*)q, q_row_stride, block_tables, max_pages, seq_starts, positions,
                  (__nv_bfloat16*)out, out_row_stride, n_seqs, nq, nkv, page_size, scale_log2, status, key_splits, part_o, part_ml,
-                 window, window > 0 && keep_first > 0 ? keep_first : 0, penalty);
+                 window, window > 0 && keep_first > 0 ? keep_first : 0, penalty, softcap > 0.f ? scale / softcap : 0.f,
+                 softcap * 1.4426950408889634f, (const __nv_bfloat16*)gate, gate_stride);
   if ((rc = check_launch("attention_prefill_tc")) || key_splits == 1) return rc;
   launch_chained(attention_prefill_merge_kernel, dim3((n_rows * nq + 3) / 4), dim3(128), 0, (cudaStream_t)stream, part_o, part_ml,
-                 (__nv_bfloat16*)out, out_row_stride, first_row, n_rows, nq, key_splits);
+                 (__nv_bfloat16*)out, out_row_stride, first_row, n_rows, nq, key_splits, (const __nv_bfloat16*)gate, gate_stride);
   return check_launch("attention_prefill_merge");
 }

@@ -27,7 +27,9 @@ ERB_DEFINE_LAST_ERROR(erb_last_error)
 // splits in order.  bfloat16, head size 32, 64 or 128.
 //
 // Both kernels take an optional penalty on the distance (`penalty`, float [2][nq]: r1 of every query head, then r2):
-// the scaled score of a key d positions back is lowered by r1 * ln(1 + r2 * d).
+// the scaled score of a key d positions back is lowered by r1 * ln(1 + r2 * d); or a cap of the scores (`softcap` c > 0):
+// the scaled score s becomes c * tanh(s / c).  With `gate` (row t, `gate_stride` apart, nq * D entries, for output row t)
+// every output entry is multiplied by the sigmoid of its entry of the gate before it is rounded.
 // =============================================================================================
 namespace {
 
@@ -45,6 +47,11 @@ struct Penalty2 {
   }
   __device__ __forceinline__ float at(int dist) const { return r1 * fast_log2(fmaf(r2, (float)dist, 1.f)); }
 };
+
+// An output entry, times the sigmoid of its entry of the gate where there is one (`gate` points at the token's row).
+__device__ __forceinline__ __nv_bfloat16 gated(float v, const __nv_bfloat16* gate, int col) {
+  return __float2bfloat16_rn(gate ? sigmoid_mul(v, __bfloat162float(gate[col])) : v);
+}
 
 __device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
@@ -74,7 +81,7 @@ constexpr int kMergeWarps = 9;            // warps of the largest block that mer
 template <int D>
 __device__ __forceinline__ void merge_splits_if_last(int* counter, const float* part_acc, const float* part_ml,
                                                      size_t head0, int n_heads, int n_splits, int max_splits,
-                                                     __nv_bfloat16* o) {
+                                                     __nv_bfloat16* o, const __nv_bfloat16* gate) {
   __shared__ int s_last;
   __shared__ float s_w[kMergeWarps][kCombineMaxSplits];     // the splits' weights, per warp
   __threadfence();
@@ -123,7 +130,7 @@ __device__ __forceinline__ void merge_splits_if_last(int* counter, const float* 
       for (int i = 0; i < V; ++i) sum[i] += x[i] * w[sp];
     }
 #pragma unroll
-    for (int i = 0; i < V; ++i) o[(size_t)h * D + lane * V + i] = __float2bfloat16_rn(sum[i] * inv);
+    for (int i = 0; i < V; ++i) o[(size_t)h * D + lane * V + i] = gated(sum[i] * inv, gate, h * D + lane * V + i);
     __syncwarp();
   }
 }
@@ -137,7 +144,8 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
                              float* __restrict__ part_acc, float* __restrict__ part_ml, int max_splits, int nq,
                              int nkv, int page_size, int split_keys, float scale_log2, int hg,
                              __nv_bfloat16* __restrict__ out, int out_row_stride, int* __restrict__ status,
-                             int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty) {
+                             int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty, float softcap,
+                             const __nv_bfloat16* __restrict__ gate, int gate_stride) {
   // Everything up to chain_wait() below reads only what earlier steps or the host wrote (the batch's
   // metadata, keys and values of earlier tokens), so it runs while the kernel before this one (the
   // one that rotates q and writes this step's keys and values) is still at work.
@@ -259,6 +267,8 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
 #pragma unroll
     for (int i = 0; i < 8; ++i) qr[g][i] = tmp[i] * scale_log2;
   }
+  const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
+  const __nv_bfloat16* gate_row = gate ? gate + (size_t)t * gate_stride : nullptr;
   Penalty2 pen[R];
 #pragma unroll
   for (int g = 0; g < R; ++g) pen[g].load(penalty, (serves ? kvh : kvh0) * R + g, nq);
@@ -324,6 +334,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
 #pragma unroll
         for (int u = 0; u < kKeysPerGroup; ++u) {
           if (penalty) sc[g][u] -= pen[g].at(pos - (key0 + u));
+          if (softcap > 0.f) sc[g][u] = capped_score(sc[g][u] * cap_in, cap_out);
           if (hidden[u]) sc[g][u] = -INFINITY;     // keys past the end of the split or before the window
           m_new = fmaxf(m_new, sc[g][u]);
         }
@@ -399,7 +410,8 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
       l += merge[(w * R + g) * (D + 2) + D + 1] * f;
     }
     if (max_splits == 1) {      // the only split: this is the result (what the combine kernel would make of it)
-      out[(size_t)t * out_row_stride + (size_t)((kvh0 + head) * R + g) * D + d] = __float2bfloat16_rn(sum * (1.f / l));
+      const int col = ((kvh0 + head) * R + g) * D + d;
+      out[(size_t)t * out_row_stride + col] = gated(sum * (1.f / l), gate_row, col);
       continue;
     }
     const size_t slot = ((size_t)seq * nq + (kvh0 + head) * R + g) * max_splits + split;
@@ -409,7 +421,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
   if (max_splits > 1 && counters)
     merge_splits_if_last<D>(counters + (size_t)seq * gridDim.y + blockIdx.y, part_acc, part_ml,
                             (size_t)seq * nq + (size_t)kvh0 * R, hg_here * R, min(pos / split_keys - first_split + 1, max_splits), max_splits,
-                            out + (size_t)t * out_row_stride + (size_t)kvh0 * R * D);
+                            out + (size_t)t * out_row_stride + (size_t)kvh0 * R * D, gate_row ? gate_row + kvh0 * R * D : nullptr);
 }
 
 // Merges the splits of each (sequence, head).  The partial maxima are in the log2 domain.  The
@@ -419,7 +431,8 @@ __global__ void __launch_bounds__(64)
 attention_decode_bulk_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                      const int* __restrict__ token_of_seq, const int* __restrict__ positions,
                                      __nv_bfloat16* __restrict__ out, int out_row_stride, int max_splits,
-                                     int nq, int head_dim, int split_keys, int window) {
+                                     int nq, int head_dim, int split_keys, int window, const __nv_bfloat16* __restrict__ gate,
+                                     int gate_stride) {
   chain_wait();
   __shared__ float s_w[kCombineMaxSplits];
   __shared__ float s_red[2];
@@ -446,7 +459,7 @@ attention_decode_bulk_combine_kernel(const float* __restrict__ part_acc, const f
     float sum = 0.f;
 #pragma unroll 8
     for (int s = 0; s < n_splits; ++s) sum += part_acc[(base + s) * head_dim + d] * s_w[s];
-    o[d] = __float2bfloat16_rn(sum * inv);
+    o[d] = gated(sum * inv, gate ? gate + (size_t)t * gate_stride : nullptr, h * head_dim + d);
   }
 }
 
@@ -479,7 +492,7 @@ int launch_decode_bulk(const void* q, int q_row_stride, const void* k_pages, con
                        const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                        float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int page_size,
                        int split_keys, float scale_log2, void* out, int out_row_stride, int* status, int* counters, int head_group,
-                       int window, int keep_first, const float* penalty, cudaStream_t s) {
+                       int window, int keep_first, const float* penalty, float softcap, const void* gate, int gate_stride, cudaStream_t s) {
   const int hg = decode_head_group(nkv, D, page_size, split_keys, head_group);
   if (hg <= 0) return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: %d heads per block with pages of %d and splits of %d", head_group, page_size, split_keys);
   constexpr int STAGE_BYTES = kDecWarps * (32 / (D / 8)) * kKeysPerGroup * D * 2;
@@ -497,7 +510,7 @@ int launch_decode_bulk(const void* q, int q_row_stride, const void* k_pages, con
   launch_chained(kern, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kDecThreads), smem, s, (const __nv_bfloat16*)q, q_row_stride,
       (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_tables, max_pages, token_of_seq, positions,
       part_acc, part_ml, max_splits, nq, nkv, page_size, split_keys, scale_log2, hg, (__nv_bfloat16*)out, out_row_stride, status, counters,
-      window, keep_first, penalty);
+      window, keep_first, penalty, softcap, (const __nv_bfloat16*)gate, gate_stride);
   return check_launch("attention_decode_bulk");
 }
 
@@ -506,12 +519,13 @@ int dispatch_group(int r, const void* q, int q_row_stride, const void* k_pages, 
                    const int* block_tables, int max_pages, const int* token_of_seq, const int* positions,
                    float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int page_size,
                    int split_keys, float scale_log2, void* out, int out_row_stride, int* status, int* counters, int head_group,
-                   int window, int keep_first, const float* penalty, cudaStream_t s) {
+                   int window, int keep_first, const float* penalty, float softcap, const void* gate, int gate_stride, cudaStream_t s) {
 #define ERB_R(RR)                                                                                              \
   case RR: return launch_decode_bulk<D, RR>(q, q_row_stride, k_pages, v_pages, block_tables, max_pages,        \
                                             token_of_seq, positions, part_acc, part_ml, max_splits, n_seqs, nq, \
                                             nkv, page_size, split_keys, scale_log2, out, out_row_stride,       \
-                                            status, counters, head_group, window, keep_first, penalty, s);
+                                            status, counters, head_group, window, keep_first, penalty, softcap, gate, \
+                                            gate_stride, s);
   switch (r) { ERB_R(1) ERB_R(2) ERB_R(3) ERB_R(4) ERB_R(5) ERB_R(6) ERB_R(7) ERB_R(8) }
 #undef ERB_R
   return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: %d query heads per kv head (at most %d)", r, kMaxGroup);
@@ -576,7 +590,8 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             float* __restrict__ part_acc, float* __restrict__ part_ml, int max_splits, int nq,
                             int nkv, int page_size, int split_keys, float scale_log2, int hg,
                             __nv_bfloat16* __restrict__ out, int out_row_stride, int* __restrict__ status,
-                            int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty) {
+                            int* __restrict__ counters, int window, int keep_first, const float* __restrict__ penalty, float softcap,
+                            const __nv_bfloat16* __restrict__ gate, int gate_stride) {
   constexpr int D = 64;
   const int R = nq / nkv;
   extern __shared__ uint8_t smem_raw[];
@@ -695,6 +710,8 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       qa[ks][1] = real ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * j + 8) : 0u;
     }
   }
+  const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
+  const __nv_bfloat16* gate_row = gate ? gate + (size_t)t * gate_stride : nullptr;
   Penalty2 pen;
   if (serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
   float o[8][4];
@@ -754,6 +771,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           const bool seen = key < n_here && !(key_abs0 + key < k_lo && key_abs0 + key >= keep_first);
           sc[b][i] *= scale_log2;
           if (penalty) sc[b][i] -= pen.at(pos - (key_abs0 + key));
+          if (softcap > 0.f) sc[b][i] = capped_score(sc[b][i] * cap_in, cap_out);
           if (!seen) sc[b][i] = -INFINITY;
           m_new = fmaxf(m_new, sc[b][i]);
         }
@@ -813,7 +831,8 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       l += merge[(w * R + gq) * (D + 2) + D + 1] * f;
     }
     if (max_splits == 1) {      // the only split: this is the result (what the combine kernel would make of it)
-      out[(size_t)t * out_row_stride + (size_t)((kvh0 + head) * R + gq) * D + d] = __float2bfloat16_rn(sum * (1.f / l));
+      const int col = ((kvh0 + head) * R + gq) * D + d;
+      out[(size_t)t * out_row_stride + col] = gated(sum * (1.f / l), gate_row, col);
       continue;
     }
     const size_t slot = ((size_t)seq * nq + (kvh0 + head) * R + gq) * max_splits + split;
@@ -823,7 +842,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   if (max_splits > 1 && counters)
     merge_splits_if_last<D>(counters + (size_t)seq * gridDim.y + blockIdx.y, part_acc, part_ml,
                             (size_t)seq * nq + (size_t)kvh0 * R, hg_here * R, min(pos / split_keys - first_split + 1, max_splits), max_splits,
-                            out + (size_t)t * out_row_stride + (size_t)kvh0 * R * D);
+                            out + (size_t)t * out_row_stride + (size_t)kvh0 * R * D, gate_row ? gate_row + kvh0 * R * D : nullptr);
 }
 
 }  // namespace
@@ -844,8 +863,10 @@ ERB_EXPORT int erb_attention_decode_gqa(const void* q, int q_row_stride, const v
                                         const int* token_of_seq, const int* positions, void* out, int out_row_stride,
                                         float* part_acc, float* part_ml, int max_splits, int n_seqs, int nq, int nkv,
                                         int head_dim, int page_size, int split_keys, float scale, int* status,
-                                        int* counters, int window, int keep_first, const float* penalty, void* stream) {
+                                        int* counters, int window, int keep_first, const float* penalty, float softcap,
+                                        const void* gate, int gate_stride, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
+  if (penalty && softcap > 0.f) return fail(ERB_ERR_UNSUPPORTED, "attention_decode_gqa: a penalty and a cap of the scores exclude each other");
   keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   if (!erb_attention_decode_gqa_supported(nq, nkv, head_dim, page_size, split_keys))
     return fail(ERB_ERR_UNSUPPORTED, "attention_decode_gqa: %d/%d heads of %d, pages of %d, splits of %d", nq, nkv,
@@ -882,11 +903,11 @@ ERB_EXPORT int erb_attention_decode_gqa(const void* q, int q_row_stride, const v
   launch_chained(attention_decode_gqa_kernel, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kGqaThreads), smem, s,
                  mk, mv, mkl, mvl, (const __nv_bfloat16*)q, q_row_stride, block_tables, max_pages, token_of_seq, positions,
                  part_acc, part_ml, max_splits, nq, nkv, page_size, split_keys, scale_log2, hg, (__nv_bfloat16*)out, out_row_stride,
-                 status, counters, window, keep_first, penalty);
+                 status, counters, window, keep_first, penalty, softcap, (const __nv_bfloat16*)gate, gate_stride);
   // a single split wrote the result itself; with counters the block that finishes last merges the splits
   if ((rc = check_launch("attention_decode_gqa")) || max_splits == 1 || counters) return rc;
   launch_chained(attention_decode_bulk_combine_kernel, dim3(dim3(nq, n_seqs)), dim3(64), 0, s, part_acc, part_ml, token_of_seq, positions,
-      (__nv_bfloat16*)out, out_row_stride, max_splits, nq, head_dim, split_keys, window);
+      (__nv_bfloat16*)out, out_row_stride, max_splits, nq, head_dim, split_keys, window, (const __nv_bfloat16*)gate, gate_stride);
   return check_launch("attention_decode_bulk_combine");
 }
 
@@ -914,8 +935,10 @@ ERB_EXPORT int erb_attention_decode_bulk(const void* q, int q_row_stride, const 
                                          const int* positions, void* out, int out_row_stride, float* part_acc,
                                          float* part_ml, int max_splits, int n_seqs, int nq, int nkv, int head_dim,
                                          int page_size, int split_keys, float scale, int* status, int* counters,
-                                         int head_group, int window, int keep_first, const float* penalty, void* stream) {
+                                         int head_group, int window, int keep_first, const float* penalty, float softcap,
+                                         const void* gate, int gate_stride, void* stream) {
   if (n_seqs <= 0) return ERB_OK;
+  if (penalty && softcap > 0.f) return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: a penalty and a cap of the scores exclude each other");
   if (nq <= 0 || nkv <= 0 || nq % nkv) return fail(ERB_ERR_ARG, "attention_decode_bulk: bad head counts");
   keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   if (max_splits <= 0 || split_keys <= 0 || !part_acc || !part_ml || !status || page_size <= 0)
@@ -932,18 +955,18 @@ ERB_EXPORT int erb_attention_decode_bulk(const void* q, int q_row_stride, const 
   switch (head_dim) {
     case 32: rc = dispatch_group<32>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                      positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size, split_keys,
-                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
+                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, softcap, gate, gate_stride, s); break;
     case 64: rc = dispatch_group<64>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                      positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size, split_keys,
-                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
+                                     scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, softcap, gate, gate_stride, s); break;
     case 128: rc = dispatch_group<128>(r, q, q_row_stride, k_pages, v_pages, block_tables, max_pages, token_of_seq,
                                        positions, part_acc, part_ml, max_splits, n_seqs, nq, nkv, page_size,
-                                       split_keys, scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, s); break;
+                                       split_keys, scale_log2, out, out_row_stride, status, counters, head_group, window, keep_first, penalty, softcap, gate, gate_stride, s); break;
     default: return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: head_dim %d (takes 32, 64, 128)", head_dim);
   }
   // a single split wrote the result itself; with counters the block that finishes last merges the splits
   if (rc || max_splits == 1 || counters) return rc;
   launch_chained(attention_decode_bulk_combine_kernel, dim3(dim3(nq, n_seqs)), dim3(64), 0, s, part_acc, part_ml, token_of_seq, positions,
-      (__nv_bfloat16*)out, out_row_stride, max_splits, nq, head_dim, split_keys, window);
+      (__nv_bfloat16*)out, out_row_stride, max_splits, nq, head_dim, split_keys, window, (const __nv_bfloat16*)gate, gate_stride);
   return check_launch("attention_decode_bulk_combine");
 }

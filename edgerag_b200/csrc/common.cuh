@@ -123,6 +123,15 @@ __device__ __forceinline__ float silu_mul(float g, float u) {
 #endif
 }
 
+// x * sigmoid(z) in float (an entry of an output gate), in the forms of silu_mul.
+__device__ __forceinline__ float sigmoid_mul(float x, float z) {
+#if ERB_ELEM == 1
+  return __fdividef(x, 1.f + __expf(-z));
+#else
+  return x / (1.f + expf(-z));
+#endif
+}
+
 // gelu(g) * u with the tanh form of gelu, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))), in float.  Every
 // kernel that gates this way calls this, so that they agree to the bit.
 __device__ __forceinline__ float gelu_tanh_mul(float g, float u) {

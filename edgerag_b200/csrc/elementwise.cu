@@ -45,6 +45,100 @@ ERB_EXPORT int erb_embed_rows(void* hidden, const void* table, const void* embed
 }
 
 // ---------------------------------------------------------------------------------------------
+// Embedding as a sum: hidden[t, :] = scale * table[id] + bigram[row] + pos[position], each of the last two where there is one
+// (`scale` multiplies the first alone; rows of given embeddings may stand in for the table's, as above).
+//   row = (id of the token before * mul_prev + id * mul_cur) mod buckets;  row `buckets` for a sequence's first token
+// The token before is the row before in the batch, or, for the first token of a sequence's portion, the last id of its portion
+// before, which is kept per state slot in `last_id`.  The block of a portion's first token reads it and then leaves the portion's
+// own last id there; rows of a negative slot have no record.  An id, or a position outside [0, n_pos), flags *status.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void embed_sum_kernel(float* __restrict__ hidden, const T* __restrict__ table, const T* __restrict__ embeds,
+                                 const int* __restrict__ ids, const int* __restrict__ embed_row, int hidden_size, int vocab,
+                                 int n_embed_rows, int* __restrict__ status, float scale, const T* __restrict__ bigram, int buckets,
+                                 long long mul_prev, long long mul_cur, const int* __restrict__ seq_of_token,
+                                 const int* __restrict__ seq_starts, const int* __restrict__ state_slots, int* __restrict__ last_id,
+                                 const int* __restrict__ positions, const T* __restrict__ pos_table, int n_pos, int vec) {
+  chain_wait();
+  const int t = blockIdx.x;
+  const int er = embed_row ? embed_row[t] : -1;
+  const int id = er >= 0 ? 0 : ids[t], p = positions[t];
+  const T* src = nullptr;
+  if (er >= 0) {
+    if (er < n_embed_rows && embeds) src = embeds + (size_t)er * hidden_size;
+  } else if (id >= 0 && id < vocab) {
+    src = table + (size_t)id * hidden_size;
+  }
+  const T* at = nullptr;
+  if (pos_table) {
+    if (p >= 0 && p < n_pos) at = pos_table + (size_t)p * hidden_size;
+    else src = nullptr;
+  }
+  const T* pair = nullptr;
+  if (bigram) {
+    const int s = seq_of_token[t], first = seq_starts[s];
+    long long row = buckets;
+    if (t > first) {
+      row = p > 0 ? ((long long)max(ids[t - 1], 0) * mul_prev + (long long)max(id, 0) * mul_cur) % buckets : buckets;
+    } else {
+      const int slot = state_slots[s];
+      const int before = slot >= 0 ? last_id[slot] : 0;
+      if (p > 0) row = ((long long)max(before, 0) * mul_prev + (long long)max(id, 0) * mul_cur) % buckets;
+      __syncthreads();                                       // (every thread has read the record)
+      if (threadIdx.x == 0 && slot >= 0) last_id[slot] = ids[seq_starts[s + 1] - 1];
+    }
+    pair = bigram + (size_t)row * hidden_size;
+  }
+  if (!src && threadIdx.x == 0) atomicCAS(status, 0, 1 + t);
+  float* dst = hidden + (size_t)t * hidden_size;
+  if (vec) {
+    for (int i = 4 * threadIdx.x; i < hidden_size; i += 4 * blockDim.x) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f}, w[4];
+      if (src) {
+        Pack4<T>::load(src + i, v);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[k] *= scale;
+        if (pair) {
+          Pack4<T>::load(pair + i, w);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) v[k] += w[k];
+        }
+        if (at) {
+          Pack4<T>::load(at + i, w);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) v[k] += w[k];
+        }
+      }
+      *reinterpret_cast<float4*>(dst + i) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < hidden_size; i += blockDim.x)
+    dst[i] = src ? Elem<T>::load(src + i) * scale + (pair ? Elem<T>::load(pair + i) : 0.f) + (at ? Elem<T>::load(at + i) : 0.f) : 0.f;
+}
+
+// `bigram` holds buckets + 1 rows (null: none), `pos_table` n_pos rows (null: none).
+ERB_EXPORT int erb_embed_sum(void* hidden, const void* table, const void* embeds, const int* ids, const int* embed_row, int n_tokens,
+                             int hidden_size, int vocab, int n_embed_rows, int* status, float scale, const void* bigram, int buckets,
+                             long long mul_prev, long long mul_cur, const int* seq_of_token, const int* seq_starts,
+                             const int* state_slots, int* last_id, const int* positions, const void* pos_table, int n_pos,
+                             void* stream) {
+  if (n_tokens <= 0) return ERB_OK;
+  if (hidden_size <= 0 || vocab <= 0 || !positions || (bigram && (buckets <= 0 || mul_prev < 0 || mul_cur < 0)))
+    return fail(ERB_ERR_ARG, "embed_sum: bad sizes");
+  if (bigram && (!seq_of_token || !seq_starts || !state_slots || !last_id))
+    return fail(ERB_ERR_ARG, "embed_sum: pairs of tokens need the batch's sequences and their records");
+  const uintptr_t bits = (uintptr_t)hidden | (uintptr_t)table | (uintptr_t)embeds | (uintptr_t)bigram | (uintptr_t)pos_table;
+  const int vec = hidden_size % 4 == 0 && (bits & 15) == 0;
+  const int threads = hidden_size >= 1024 ? 256 : 128;
+  launch_chained(embed_sum_kernel<elem_t>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream, (float*)hidden,
+      (const elem_t*)table, (const elem_t*)embeds, ids, embed_row, hidden_size, vocab, n_embed_rows, status, scale,
+      (const elem_t*)bigram, buckets, mul_prev, mul_cur, seq_of_token, seq_starts, state_slots, last_id, positions,
+      (const elem_t*)pos_table, n_pos, vec);
+  return check_launch("embed_sum");
+}
+
+// ---------------------------------------------------------------------------------------------
 // Residual add + RMSNorm.
 //   r = hidden[row] (+ dscale * delta[row])   in float, stored back when `write_back` (dscale: a constant of the model
 //                                             that multiplies every update of its stream; 1 for most)
@@ -675,11 +769,12 @@ ERB_EXPORT int erb_resolve_ids(int* ids, int n, const int* fed, int n_fed, void*
 // A gated unit with bounded branches: with g = min(gate, limit) and u = clamp(up, -limit, limit),
 //   out[t, i] = g * sigmoid(alpha * g) * (u + shift),      gate = gate_up[t, i], up = gate_up[t, I + i],
 // computed in float.  limit <= 0 leaves both branches unbounded; (alpha, shift) = (1, 0) is SwiGLU.  `act` 1 puts
-// the tanh form of gelu in the place of g * sigmoid(alpha * g) (see glu_gate).
+// the tanh form of gelu in the place of g * sigmoid(alpha * g) (see glu_gate).  `row_scale` (a float per row, or null) multiplies
+// the row before it is rounded.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void glu_bounded_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total,
-                                   float limit, float alpha, float shift, int act) {
+                                   float limit, float alpha, float shift, int act, const float* __restrict__ row_scale) {
   chain_wait();
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total) return;
@@ -687,13 +782,13 @@ __global__ void glu_bounded_kernel(const T* __restrict__ gate_up, T* __restrict_
   const int i = (int)(idx % inter);
   const T* row = gate_up + t * 2 * (size_t)inter;
   const float g = Elem<T>::load(row + i), u = Elem<T>::load(row + inter + i);
-  Elem<T>::store(out + idx, glu_gate(g, u, act, limit, alpha, shift));
+  Elem<T>::store(out + idx, glu_gate(g, u, act, limit, alpha, shift) * (row_scale ? row_scale[t] : 1.f));
 }
 
 // The same on 16-byte groups (the intermediate size a multiple of the group, rows 16-byte aligned).
 template <typename T>
 __global__ void glu_bounded_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t groups,
-                                       float limit, float alpha, float shift, int act) {
+                                       float limit, float alpha, float shift, int act, const float* __restrict__ row_scale) {
   chain_wait();
   constexpr int N = Vec16<T>::N;
   const size_t gidx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -705,24 +800,25 @@ __global__ void glu_bounded_vec_kernel(const T* __restrict__ gate_up, T* __restr
   float g[N], u[N];
   Vec16<T>::load(row + i, g);
   Vec16<T>::load(row + inter + i, u);
+  const float factor = row_scale ? row_scale[t] : 1.f;
 #pragma unroll
-  for (int j = 0; j < N; ++j) g[j] = glu_gate(g[j], u[j], act, limit, alpha, shift);
+  for (int j = 0; j < N; ++j) g[j] = glu_gate(g[j], u[j], act, limit, alpha, shift) * factor;
   Vec16<T>::store(out + t * (size_t)inter + i, g);
 }
 
 ERB_EXPORT int erb_glu_bounded(const void* gate_up, void* out, int n_tokens, int inter, float limit, float alpha,
-                               float shift, int act, void* stream) {
+                               float shift, int act, const float* row_scale, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   if (inter <= 0) return fail(ERB_ERR_ARG, "glu_bounded: bad intermediate size");
   const size_t total = (size_t)n_tokens * inter;
   if (inter % Vec16<elem_t>::N == 0 && !((uintptr_t)gate_up & 15) && !((uintptr_t)out & 15)) {
     const size_t groups = total / Vec16<elem_t>::N;
     launch_chained(glu_bounded_vec_kernel<elem_t>, dim3((unsigned)((groups + 255) / 256)), dim3(256), 0, (cudaStream_t)stream,
-                   (const elem_t*)gate_up, (elem_t*)out, inter, groups, limit, alpha, shift, act);
+                   (const elem_t*)gate_up, (elem_t*)out, inter, groups, limit, alpha, shift, act, row_scale);
     return check_launch("glu_bounded");
   }
   launch_chained(glu_bounded_kernel<elem_t>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, (cudaStream_t)stream,
-                 (const elem_t*)gate_up, (elem_t*)out, inter, total, limit, alpha, shift, act);
+                 (const elem_t*)gate_up, (elem_t*)out, inter, total, limit, alpha, shift, act, row_scale);
   return check_launch("glu_bounded");
 }
 
@@ -1525,6 +1621,9 @@ ERB_EXPORT int erb_bias_rows(float* y, const float* vec, int n_rows, int width, 
 //   the first rot_dim entries of every q and k head are turned, entry i with entry i + rot_dim / 2, by position * inv_freq[i]
 //   q goes back in place, k and v to the token's cache slot (page * page_size + offset; negative or no pages: not written).
 // `has_kv` 0: the row holds queries only (a layer that reads another layer's keys and values).
+// Values may be blended with an earlier layer's: `first` holds that layer's values of the step's tokens as [token][nkv * v_dim]
+// (true head sizes, the entries as the projection left them).  blend_write: this is that layer, it leaves its values there; else
+// with `blend` (one float l) the cached value is (1 - l) v + l * first.
 // One block per token.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
@@ -1533,7 +1632,8 @@ qkv_whole_norm_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_b
                       const float* __restrict__ v_bias, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
                       float q_count, float k_count, float eps, const int* __restrict__ positions,
                       const float* __restrict__ inv_freq, int rot_dim, const int* __restrict__ slots, T* __restrict__ k_pages,
-                      T* __restrict__ v_pages, int nq, int nkv, int D, int page_size, int has_kv) {
+                      T* __restrict__ v_pages, int nq, int nkv, int D, int page_size, int has_kv, T* __restrict__ first,
+                      const float* __restrict__ blend, int blend_write, int v_dim) {
   chain_wait();
   extern __shared__ float wn_smem[];      // (nq + nkv) * D floats, then 32 of scratch
   const int qw = nq * D, kw = has_kv ? nkv * D : 0;
@@ -1585,10 +1685,18 @@ qkv_whole_norm_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_b
       Elem<T>::store(dst + i, src[i] * rs * (nw ? nw[i] : 1.f));
     }
   }
-  if (slot >= 0 && v_pages) {
+  const bool stores_v = slot >= 0 && v_pages;
+  if (stores_v || (has_kv && first && blend_write)) {
+    const float l = first && !blend_write ? *blend : 0.f;
     for (int i = threadIdx.x; i < kw; i += blockDim.x) {
       const int hh = i / D, e = i % D;
-      const float v = Elem<T>::load(row + qw + kw + i) + (v_bias ? v_bias[i] : 0.f);
+      float v = Elem<T>::load(row + qw + kw + i) + (v_bias ? v_bias[i] : 0.f);
+      if (first && e < v_dim) {
+        T* kept = first + (size_t)t * nkv * v_dim + hh * v_dim + e;
+        if (blend_write) Elem<T>::store(kept, v);
+        else v = fmaf(l, Elem<T>::load(kept), (1.f - l) * v);
+      }
+      if (!stores_v) continue;
       Elem<T>::store(v_pages + (((size_t)page * nkv + hh) * page_size + offset) * D + e, v);
     }
   }
@@ -1598,8 +1706,10 @@ ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const 
                                   const float* q_norm, const float* k_norm, int q_count, int k_count, float eps,
                                   const int* positions, const float* inv_freq, int rot_dim, const int* slots, void* k_pages,
                                   void* v_pages, int n_tokens, int nq, int nkv, int head_dim, int page_size, int has_kv,
-                                  void* stream) {
+                                  void* first, const float* blend, int blend_write, int v_dim, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
+  if (first && (!has_kv || v_dim <= 0 || v_dim > head_dim || (!blend_write && !blend)))
+    return fail(ERB_ERR_ARG, "qkv_whole_norm: blended values need values, their size and the blend");
   if (nq <= 0 || nkv <= 0 || head_dim <= 0 || rot_dim < 0 || rot_dim % 2 || rot_dim > head_dim || (rot_dim && !inv_freq) ||
       q_count <= 0 || k_count <= 0 || page_size <= 0)
     return fail(ERB_ERR_ARG, "qkv_whole_norm: bad sizes (rot_dim %d of head_dim %d)", rot_dim, head_dim);
@@ -1613,7 +1723,7 @@ ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const 
   }
   launch_chained(kern, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, (elem_t*)qkv, ld, q_bias, k_bias, v_bias, q_norm,
                  k_norm, (float)q_count, (float)k_count, eps, positions, inv_freq, rot_dim, slots, (elem_t*)k_pages,
-                 (elem_t*)v_pages, nq, nkv, head_dim, page_size, has_kv);
+                 (elem_t*)v_pages, nq, nkv, head_dim, page_size, has_kv, (elem_t*)first, blend, blend_write, v_dim);
   return check_launch("qkv_whole_norm");
 }
 

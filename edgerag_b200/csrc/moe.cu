@@ -4,7 +4,9 @@
 //   1. route:   z = W_router x (float), s = sigmoid(z); the `top` experts with the largest z (the lower index wins a tie);
 //               per token the chosen experts and their scores s.  A (token, choice) is a "pair", numbered token * top + choice.
 //               With a correction per expert the choice goes by s + correction; a group of experts counts as much as its
-//               best expert or as the sum of its two best; the chosen scores may be divided by their sum.
+//               best expert or as the sum of its two best; the chosen scores may be divided by their sum and are multiplied
+//               by a constant.  A row of the router beyond its experts' gives one more logit per token, whose sigmoid is left
+//               for the caller (what a shared expert's output is multiplied by).
 //   2. lists:   one block per expert counts all choices, makes its offset (and its offset in row tiles) and writes the
 //               pair numbers of its expert in rising order behind the offset.
 //   3. gate/up: for every expert the rows of its pairs, each row the token's input times the pair's score (rounded to T
@@ -64,7 +66,7 @@ __device__ __forceinline__ int take_largest(unsigned* keys, int n) {
 __device__ __forceinline__ void choose_experts(const float* z, unsigned* keys, unsigned* gkeys, int n_experts, int top,
                                                int* __restrict__ choice, float* __restrict__ score, int* pairs, int score_kind,
                                                int n_groups, int keep_groups, const float* __restrict__ correction, int group_kind,
-                                               int normalise) {
+                                               int normalise, float weight) {
   const int lane = threadIdx.x & 31;
   // softmax scores: the maximum and the denominator over all experts, before any expert is ruled out
   float z_top = 0.f, denom = 1.f;
@@ -108,15 +110,15 @@ __device__ __forceinline__ void choose_experts(const float* z, unsigned* keys, u
       sum += mine;
       choice[c] = arg;
       if (pairs) pairs[c] = arg;
-      if (!normalise || top > 32) score[c] = mine;
+      if (!normalise || top > 32) score[c] = normalise ? mine : mine * weight;
     }
   }
   if (!normalise) return;
   const float total = warp_sum(sum) + 1e-20f;
   if (top <= 32) {
-    if (lane < top) score[lane] = mine / total;
+    if (lane < top) score[lane] = mine / total * weight;
   } else {
-    for (int c = lane; c < top; c += 32) score[c] /= total;
+    for (int c = lane; c < top; c += 32) score[c] = score[c] / total * weight;
   }
 }
 
@@ -130,10 +132,11 @@ template <typename T>
 __global__ void __launch_bounds__(kRouteThreads)
 moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_router, int n_tokens, int width, int n_experts,
                  int top, int* __restrict__ choice, float* __restrict__ score, int score_kind, int n_groups, int keep_groups,
-                 const float* __restrict__ correction, int group_kind, int normalise) {
+                 const float* __restrict__ correction, int group_kind, int normalise, float weight, float* __restrict__ side_gate) {
   chain_wait();
-  extern __shared__ float z_s[];                 // [kRouteTokens][n_experts padded to 4] logits, the same again for the
-  const int e_pad = (n_experts + 3) & ~3;        // groups' values and for what the choice goes by, then [kRouteTokens][width]
+  const int n_rows = n_experts + (side_gate != nullptr);
+  extern __shared__ float z_s[];                 // [kRouteTokens][n_rows padded to 4] logits, the same again for the
+  const int e_pad = (n_rows + 3) & ~3;           // groups' values and for what the choice goes by, then [kRouteTokens][width]
   float* g_s = z_s + kRouteTokens * e_pad;
   float* c_s = g_s + kRouteTokens * e_pad;
   float* x_s = c_s + kRouteTokens * e_pad;
@@ -147,7 +150,7 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
   }
   __syncthreads();
   const int whole = (width & 3) == 0 ? width & ~127 : 0;       // entries read as float4 by whole warps
-  for (int e = warp; e < n_experts; e += kRouteThreads / 32) {
+  for (int e = warp; e < n_rows; e += kRouteThreads / 32) {
     const float* w = w_router + (size_t)e * width;
     float acc[kRouteTokens];
 #pragma unroll
@@ -179,9 +182,10 @@ moe_route_kernel(const T* __restrict__ x, int ld, const float* __restrict__ w_ro
   if (warp >= n_here) return;
   const int t = t0 + warp;
   float* z = z_s + warp * e_pad;
+  if (side_gate && lane == 0) side_gate[t] = 1.f / (1.f + expf(-z[n_experts]));
   choose_experts(z, reinterpret_cast<unsigned*>(c_s) + warp * e_pad, reinterpret_cast<unsigned*>(g_s) + warp * e_pad, n_experts, top,
                  choice + (size_t)t * top, score + (size_t)t * top, nullptr, score_kind, n_groups, keep_groups, correction, group_kind,
-                 normalise);
+                 normalise, weight);
 }
 
 // One block per expert e builds the expert's part of the lists on its own: a histogram of all choices in shared memory
@@ -293,8 +297,10 @@ __global__ void __launch_bounds__(kRouteThreads)
 moe_choose_lists_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top, int* __restrict__ choice,
                         float* __restrict__ score, int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ tiles,
                         int* __restrict__ order, int tile_rows, int score_kind, int n_groups, int keep_groups,
-                        const float* __restrict__ correction, int group_kind, int normalise) {
+                        const float* __restrict__ correction, int group_kind, int normalise, float weight,
+                        float* __restrict__ side_gate) {
   chain_wait();
+  const int n_rows = n_experts + (side_gate != nullptr);     // logits per token
   extern __shared__ float z_s[];                 // per warp: logits, what the choice goes by, the groups' values
   constexpr int kWarps = kRouteThreads / 32;
   __shared__ int pair_s[kRouteFewPairs];
@@ -304,11 +310,12 @@ moe_choose_lists_kernel(const float* __restrict__ logits, int n_tokens, int n_ex
   float* z = z_s + 3 * warp * e_pad;
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count_s[e] = 0;
   for (int t = warp; t < n_tokens; t += kWarps) {
-    for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * n_experts + e];
+    for (int e = lane; e < n_experts; e += 32) z[e] = logits[(size_t)t * n_rows + e];
+    if (side_gate && lane == 0) side_gate[t] = 1.f / (1.f + expf(-logits[(size_t)t * n_rows + n_experts]));
     __syncwarp();
     unsigned* keys = reinterpret_cast<unsigned*>(z + e_pad);
     choose_experts(z, keys, keys + e_pad, n_experts, top, choice + (size_t)t * top, score + (size_t)t * top, pair_s + t * top, score_kind,
-                   n_groups, keep_groups, correction, group_kind, normalise);
+                   n_groups, keep_groups, correction, group_kind, normalise, weight);
     __syncwarp();
   }
   __syncthreads();
@@ -454,7 +461,8 @@ moe_product_kernel(const T* __restrict__ a, int lda, const T* __restrict__ weigh
 
 ERB_EXPORT int erb_moe_tile_rows() { return kTM; }
 
-// Whether a step of this many tokens is routed by the pair of kernels for few tokens (then `logits` is [n_tokens][n_experts]).
+// Whether a step of this many tokens is routed by the pair of kernels for few tokens (then `logits` is [n_tokens][n_experts], with a
+// row of the router for the shared expert's gate [n_tokens][n_experts + 1]).
 ERB_EXPORT int erb_moe_route_few(int n_tokens, int n_experts, int top) {
   return n_tokens <= kRouteFewTokens && n_tokens * top <= kRouteFewPairs && n_experts <= kRouteFewExperts;
 }
@@ -462,7 +470,7 @@ ERB_EXPORT int erb_moe_route_few(int n_tokens, int n_experts, int top) {
 ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n_tokens, int width, int n_experts, int top,
                              int* choice, float* score, int* counts, int* offsets, int* tiles, int* order, int tile_rows,
                              int score_kind, int n_groups, int keep_groups, const float* correction, int group_kind,
-                             int normalise, float* logits, void* stream) {
+                             int normalise, float weight, float* side_gate, float* logits, void* stream) {
   if (n_tokens <= 0) return ERB_OK;
   if (width <= 0 || n_experts <= 0 || top <= 0 || top > n_experts || n_experts > 8192)
     return fail(ERB_ERR_ARG, "moe_route: %d of %d experts", top, n_experts);
@@ -474,10 +482,10 @@ ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n
       (score_kind != ERB_SCORE_SIGMOID && (correction || group_kind != ERB_GROUP_BEST)))
     return fail(ERB_ERR_ARG, "moe_route: a correction and groups that count their two best go with sigmoid scores");
   cudaStream_t s = (cudaStream_t)stream;
-  const int n_pairs = n_tokens * top;
+  const int n_pairs = n_tokens * top, n_rows = n_experts + (side_gate != nullptr);
   if (logits && erb_moe_route_few(n_tokens, n_experts, top)) {
-    launch_chained(moe_logits_kernel<elem_t>, dim3((n_tokens + kRouteTokens - 1) / kRouteTokens, (n_experts + 3) / 4), dim3(128), 0, s,
-                   (const elem_t*)x, ld, w_router, n_tokens, width, n_experts, logits);
+    launch_chained(moe_logits_kernel<elem_t>, dim3((n_tokens + kRouteTokens - 1) / kRouteTokens, (n_rows + 3) / 4), dim3(128), 0, s,
+                   (const elem_t*)x, ld, w_router, n_tokens, width, n_rows, logits);
     int rc = check_launch("moe_logits");
     if (rc) return rc;
     const size_t smem = sizeof(float) * (3 * (kRouteThreads / 32) + 2) * (size_t)((n_experts + 3) & ~3);
@@ -487,10 +495,10 @@ ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n
     }
     launch_chained(moe_choose_lists_kernel, dim3(1), dim3(kRouteThreads), smem, s, (const float*)logits, n_tokens, n_experts, top, choice,
                    score, counts, offsets, tiles, order, tile_rows > 0 ? tile_rows : kTM, score_kind, n_groups, keep_groups, correction,
-                   group_kind, normalise);
+                   group_kind, normalise, weight, side_gate);
     return check_launch("moe_choose_lists");
   }
-  const size_t route_smem = sizeof(float) * kRouteTokens * (3 * (size_t)((n_experts + 3) & ~3) + width);
+  const size_t route_smem = sizeof(float) * kRouteTokens * (3 * (size_t)((n_rows + 3) & ~3) + width);
   if (route_smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(moe_route_kernel<elem_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)route_smem);
     if (err != cudaSuccess) return fail(ERB_ERR_CUDA, "moe_route: %s", cudaGetErrorString(err));
@@ -498,7 +506,7 @@ ERB_EXPORT int erb_moe_route(const void* x, int ld, const float* w_router, int n
   if (route_smem > 200 * 1024) return fail(ERB_ERR_UNSUPPORTED, "moe_route: rows of %d entries with %d experts", width, n_experts);
   launch_chained(moe_route_kernel<elem_t>, dim3((n_tokens + kRouteTokens - 1) / kRouteTokens), dim3(kRouteThreads), route_smem, s,
                  (const elem_t*)x, ld, w_router, n_tokens, width, n_experts, top, choice, score, score_kind, n_groups, keep_groups,
-                 correction, group_kind, normalise);
+                 correction, group_kind, normalise, weight, side_gate);
   int rc = check_launch("moe_route");
   if (rc) return rc;
   launch_chained(moe_lists_kernel, dim3(n_experts), dim3(256), sizeof(int) * n_experts, s, (const int*)choice, n_pairs, n_experts,

@@ -201,11 +201,19 @@ __device__ __forceinline__ float fast_log2(float x) {
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float fast_rcp(float x) {           // 1 / x, one instruction; inf gives 0
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float fast_exp2(float x) {          // 2^x, one instruction; -inf gives 0
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// A capped score in the log2 domain: for a scaled score s, x = 2 log2(e) s / c and c2 = c log2(e) this is log2(e) c tanh(s / c),
+// as c2 (1 - 2 / (1 + 2^x)); its error is a few units in the last place of c2, whatever s is.
+__device__ __forceinline__ float capped_score(float x, float c2) { return fmaf(-2.f * c2, fast_rcp(1.f + fast_exp2(x)), c2); }
 
 // Tensor maps over a page pool seen as [rows = pages * kv heads * page_size][64 bfloat16] with boxes
 // of `box_rows` rows and the 128-byte swizzle.  Encoding is a host-side computation; the maps are

@@ -129,6 +129,8 @@ class Engine:
         layout = model.cache_layout
         itemsize = 2 if self.dtype == torch.bfloat16 else 4
         max_len = options.max_model_len or getattr(config, "max_position_embeddings", None) or 8192
+        if getattr(model, "max_positions", None) is not None:     # (a table of positions ends there)
+            max_len = min(max_len, model.max_positions)
         self.max_model_len = max_len
         if options.num_blocks is not None:
             num_pages = options.num_blocks

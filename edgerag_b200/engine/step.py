@@ -245,6 +245,9 @@ class ModelRunner:
                 raise StepError(f"request {e.request_id!r}: embeds must be [n, {hidden}]")
             if e.tokens is not None and not all(0 <= int(t) < vocab for t in e.tokens):
                 raise StepError(f"request {e.request_id!r}: a token id is outside [0, {vocab})")
+            limit = getattr(self.model, "max_positions", None)
+            if limit is not None and self.cache.requests[e.request_id].num_tokens + n > limit:
+                raise StepError(f"request {e.request_id!r}: the model has no position from {limit} on")
             if any(not 0 <= int(w) < n for w in e.want):
                 raise StepError(f"request {e.request_id!r}: a wanted place is outside its {n} tokens")
         total = sum(e.n_tokens for e in entries)
@@ -272,7 +275,7 @@ class ModelRunner:
         graphable = self.graphs_enabled and all(e.embeds is None for e in ordered)
         # Filler rows between the single tokens and the portions (None in `rows`): see `pad_decodes`.
         n_fill = 0
-        if self.pad_decodes and n_decode and all(e.embeds is None for e in ordered) and not self.cache.layout.states:
+        if self.pad_decodes and n_decode and all(e.embeds is None for e in ordered) and all(s.fillers for s in self.cache.layout.states):
             n_fill = _fill_to(n_decode) - n_decode
             if total + n_fill > self.max_step_tokens:
                 n_fill = 0
@@ -308,13 +311,14 @@ class ModelRunner:
         for s, (orig, e) in enumerate(zip(origins, rows)):
             if e is None:
                 # a filler: token 0 at position 0 of a sequence whose table names page 0 only; it reads that
-                # page's first key (whatever it holds: the row's results go nowhere) and has no cache slot
+                # page's first key (whatever it holds: the row's results go nowhere) and has no cache slot and no state slot
                 seq_of_token[t0] = s
                 token_of_seq[s] = t0
                 seq_starts[s + 1] = t0 + 1
+                state_slots[s] = -1
                 ctx.host_q_len.append(1)
                 ctx.host_positions_last.append(0)
-                ctx.host_state_slots.append(0)
+                ctx.host_state_slots.append(-1)
                 t0 += 1
                 continue
             rc = self.cache.requests[e.request_id]

@@ -59,6 +59,9 @@ class DecoderModel:
             getattr(getattr(b.mixer, "position", None), "graph_safe", True) for b in self.blocks)
         #: some part looks at the tokens' ids: rows of embeddings cannot stand in for them
         self.needs_token_ids = any(part.needs_token_ids for _, part in self._owners)
+        limits = [part.max_positions for _, part in self._owners if part.max_positions is not None]
+        #: positions that some part has no row for start here (None: no such part)
+        self.max_positions = min(limits) if limits else None
         self.logits_stride = -(-plan.vocab_size // 8) * 8  # rows of the logits buffer start 32-byte aligned
 
     # --- cache needs ------------------------------------------------------------------------------
@@ -92,7 +95,9 @@ class DecoderModel:
                     layout.placement[cl] = (g, counts[g])
                     counts[g] += 1
                 else:
-                    layout.states.append(StateSpec(f"{item.name}@{cl}", tuple(item.shape), item.dtype))
+                    layout.states.append(StateSpec(f"{item.name}@{cl}", tuple(item.shape), item.dtype, item.fillers))
+        for item in getattr(self.embedding, "state_specs", list)():
+            layout.states.append(StateSpec(f"{item.name}@embedding", tuple(item.shape), item.dtype, item.fillers))
         layout.groups = [KVGroupSpec(c, *k) for k, c in zip(keys, counts)]
         return layout
 

@@ -25,6 +25,8 @@ _ELEM = {torch.float32: "float32", torch.bfloat16: "bfloat16"}
 _SIGNATURES = {
     "erb_embed_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                        c_void_p, c_float, c_void_p],
+    "erb_embed_sum": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+                      c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "erb_add_rmsnorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int,
                         c_float, c_void_p],
     "erb_residual_add": [c_void_p, c_void_p, c_longlong, c_float, c_void_p],
@@ -40,7 +42,7 @@ _SIGNATURES = {
     "erb_linear_skinny": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "erb_linear_skinny_glu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "erb_linear_skinny_glu_bounded": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                      c_float, c_int, c_void_p],
+                                      c_float, c_int, c_void_p, c_void_p],
     "erb_linear_skinny_rope": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "erb_linear_tc": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -55,20 +57,23 @@ _SIGNATURES = {
     "erb_linear_tc_rope": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "erb_attention_rows": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_float,
+                           c_void_p, c_int, c_void_p],
     "erb_attention_decode": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                              c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+                             c_int, c_int, c_int, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p],
     "erb_attention_prefill_tc": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
-                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_int,
+                                 c_void_p],
     "erb_attention_decode_bulk": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                   c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+                                  c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int,
+                                  c_void_p],
     "erb_attention_decode_gqa": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
-    "erb_glu_bounded": [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
+                                 c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p],
+    "erb_glu_bounded": [c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p],
     "erb_add_layernorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float,
                           c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "erb_cast_rows": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -117,12 +122,12 @@ _SIGNATURES = {
     "erb_bias_rows": [c_void_p, c_void_p, c_int, c_int, c_void_p],
     "erb_qkv_whole_norm": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float,
                            c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                           c_void_p],
+                           c_void_p, c_void_p, c_int, c_int, c_void_p],
     "erb_delta_scan": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "erb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "erb_moe_route": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
+                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p],
     "erb_moe_tc_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "erb_moe_tc_gate_up": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                            c_void_p, c_void_p],
@@ -218,6 +223,38 @@ def embed_rows(hidden: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, sta
     _call(_fn("elementwise", _elem(table), "erb_embed_rows"), hidden.data_ptr(), table.data_ptr(),
           _ptr(embeds), ids.data_ptr(), _ptr(embed_row), n, h, table.shape[0],
           0 if embeds is None else embeds.shape[0], status.data_ptr(), float(scale), _stream())
+
+
+def embed_sum(hidden: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, status: torch.Tensor, positions: torch.Tensor, *,
+              scale: float = 1.0, embeds: torch.Tensor | None = None, embed_row: torch.Tensor | None = None,
+              pairs: torch.Tensor | None = None, pair_hash: tuple[int, int, int] | None = None, last_id: torch.Tensor | None = None,
+              seq_of_token: torch.Tensor | None = None, seq_starts: torch.Tensor | None = None,
+              state_slots: torch.Tensor | None = None, pos_table: torch.Tensor | None = None) -> None:
+    """``embed_rows`` with more terms: ``hidden[t] = scale * table[id] + pairs[row] + pos_table[positions[t]]`` (the last two where
+    given).  ``pair_hash = (buckets, mul_prev, mul_cur)``: ``row = (id of the token before * mul_prev + id * mul_cur) mod buckets``,
+    row ``buckets`` for position 0; ``pairs`` has ``buckets + 1`` rows.  The token before a portion's first one is the state record
+    ``last_id`` (int32 ``[slots, 1]``) of its sequence, which afterwards holds the portion's last token; a negative slot has none."""
+    n, h = hidden.shape
+    _need(hidden, "hidden", torch.float32); _need(table, "table"); _need(ids, "ids", torch.int32)
+    _need(status, "status", torch.int32); _need(embed_row, "embed_row", torch.int32); _need(positions, "positions", torch.int32)
+    _need(embeds, "embeds", table.dtype); _need(pairs, "pairs", table.dtype); _need(pos_table, "pos_table", table.dtype)
+    if table.shape[1] != h or ids.numel() < n or positions.numel() < n or any(t is not None and t.shape[1] != h for t in (embeds, pairs, pos_table)):
+        raise KernelError("embed_sum: shapes disagree")
+    if embeds is not None and (embed_row is None or pairs is not None):
+        raise KernelError("embed_sum: embeds need embed_row and exclude rows of token pairs")
+    buckets = mul_prev = mul_cur = 0
+    if pairs is not None:
+        for name, t in (("last_id", last_id), ("seq_of_token", seq_of_token), ("seq_starts", seq_starts), ("state_slots", state_slots)):
+            if t is None:
+                raise KernelError(f"embed_sum: rows of token pairs need {name}")
+            _need(t, name, torch.int32)
+        buckets, mul_prev, mul_cur = (int(v) for v in pair_hash)
+        if pairs.shape[0] != buckets + 1:
+            raise KernelError("embed_sum: the table of pairs has a row per bucket and one more")
+    _call(_fn("elementwise", _elem(table), "erb_embed_sum"), hidden.data_ptr(), table.data_ptr(), _ptr(embeds), ids.data_ptr(),
+          _ptr(embed_row), n, h, table.shape[0], 0 if embeds is None else embeds.shape[0], status.data_ptr(), float(scale), _ptr(pairs),
+          buckets, mul_prev, mul_cur, _ptr(seq_of_token), _ptr(seq_starts), _ptr(state_slots), _ptr(last_id), positions.data_ptr(),
+          _ptr(pos_table), 0 if pos_table is None else pos_table.shape[0], _stream())
 
 
 def add_rmsnorm(hidden: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float,
@@ -367,14 +404,22 @@ def qkv_whole_norm(qkv: torch.Tensor, positions: torch.Tensor, n_q_heads: int, n
                    q_count: int, k_count: int, eps: float, q_bias: torch.Tensor | None = None, k_bias: torch.Tensor | None = None,
                    v_bias: torch.Tensor | None = None, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
                    inv_freq: torch.Tensor | None = None, rot_dim: int = 0, has_kv: bool = True, slots: torch.Tensor | None = None,
-                   k_pages: torch.Tensor | None = None, v_pages: torch.Tensor | None = None, page_size: int = 16) -> None:
+                   k_pages: torch.Tensor | None = None, v_pages: torch.Tensor | None = None, page_size: int = 16,
+                   first_values: torch.Tensor | None = None, blend: torch.Tensor | None = None) -> None:
     """Rows ``[q heads | k heads | v heads]`` (``head_dim`` entries a head; with ``has_kv`` False the queries only) made
     ready for attention where the norm of queries and keys runs over a token's whole projection: biases added, ``q *
     rsqrt(sum(q^2) / q_count + eps) * q_norm`` (all entries of the row at once; ``q_count`` is the true number of
     entries where heads are padded with zeros), k likewise, entries ``i`` and ``i + rot_dim / 2`` of the first
     ``rot_dim`` of every q and k head turned by ``position * inv_freq[i]``; q goes back in place, k and v (plus bias)
-    to the tokens' cache slots.  All in float."""
+    to the tokens' cache slots.  All in float.  ``first_values`` ``[tokens, n_kv_heads * true value size]``: without ``blend`` the
+    rows' values are also left there; with it (one float ``l``) the cached values are ``(1 - l) v + l first_values``."""
     _need(qkv, "qkv", contiguous=False); _need(positions, "positions", torch.int32)
+    _need(first_values, "first_values", qkv.dtype); _need(blend, "blend", torch.float32)
+    v_dim = 0
+    if first_values is not None:
+        v_dim = first_values.shape[1] // n_kv_heads
+        if not has_kv or first_values.shape != (qkv.shape[0], n_kv_heads * v_dim) or not 0 < v_dim <= head_dim:
+            raise KernelError("qkv_whole_norm: first_values are [tokens, kv heads * value size]")
     for name, t in (("q_bias", q_bias), ("k_bias", k_bias), ("v_bias", v_bias), ("q_norm", q_norm), ("k_norm", k_norm),
                     ("inv_freq", inv_freq)):
         _need(t, name, torch.float32)
@@ -394,7 +439,7 @@ def qkv_whole_norm(qkv: torch.Tensor, positions: torch.Tensor, n_q_heads: int, n
     _call(_fn("elementwise", _elem(qkv), "erb_qkv_whole_norm"), qkv.data_ptr(), qkv.stride(0) if n > 1 else qkv.shape[1],
           _ptr(q_bias), _ptr(k_bias), _ptr(v_bias), _ptr(q_norm), _ptr(k_norm), int(q_count), int(k_count), float(eps),
           positions.data_ptr(), _ptr(inv_freq), int(rot_dim), _ptr(slots), _ptr(k_pages), _ptr(v_pages), n, n_q_heads,
-          n_kv_heads, head_dim, int(page_size), int(bool(has_kv)), _stream())
+          n_kv_heads, head_dim, int(page_size), int(bool(has_kv)), _ptr(first_values), _ptr(blend), int(blend is None), v_dim, _stream())
 
 
 def cast_rows(src: torch.Tensor, dst: torch.Tensor) -> None:
@@ -505,16 +550,20 @@ GLU_ACTS = {"sigmoid": 0, "gelu_tanh": 1}
 
 
 def glu_bounded(gate_up: torch.Tensor, out: torch.Tensor, limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0,
-                act: str = "sigmoid") -> None:
+                act: str = "sigmoid", row_scale: torch.Tensor | None = None) -> None:
     """out[t, i] = g * sigmoid(alpha * g) * (u + shift) with g = min(gate_up[t, i], limit) and
     u = clamp(gate_up[t, I + i], -limit, limit); ``limit <= 0`` bounds nothing.  ``act="gelu_tanh"``:
-    ``0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))`` in the place of ``g * sigmoid(alpha * g)``."""
+    ``0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))`` in the place of ``g * sigmoid(alpha * g)``.  ``row_scale``: a float per row
+    that multiplies the row before it is rounded."""
+    _need(row_scale, "row_scale", torch.float32)
+    if row_scale is not None and row_scale.numel() < out.shape[0]:
+        raise KernelError("glu_bounded: one row_scale per row")
     _need(gate_up, "gate_up"); _need(out, "out", gate_up.dtype)
     n, inter = out.shape
     if gate_up.shape != (n, 2 * inter):
         raise KernelError("glu_bounded: gate_up must be [tokens, 2 * intermediate]")
     _call(_fn("elementwise", _elem(out), "erb_glu_bounded"), gate_up.data_ptr(), out.data_ptr(), n, inter, float(limit),
-          float(alpha), float(shift), GLU_ACTS[act], _stream())
+          float(alpha), float(shift), GLU_ACTS[act], _ptr(row_scale), _stream())
 
 
 def softcap(logits: torch.Tensor, cap: float, dtype: torch.dtype) -> None:
@@ -809,11 +858,15 @@ def linear_glu_supported(a: torch.Tensor, weight: torch.Tensor, max_rows: int = 
     return a.shape[0] <= max_rows and weight.shape[0] % 2 == 0 and linear_few_rows_supported(a, weight, lda)
 
 
-def linear_glu(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bounded: tuple | None = None) -> None:
+def linear_glu(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bounded: tuple | None = None,
+               row_scale: torch.Tensor | None = None) -> None:
     """out[M, N] = silu(a @ gate^T) * (a @ up^T) for ``weight = [gate; up]`` of shape [2N, K], in one
     launch; equal to ``linear`` into an [M, 2N] buffer followed by ``swiglu`` (each product is rounded
     to bfloat16 before the gate).  ``bounded = (limit, alpha, shift[, act])``: the gate of ``glu_bounded`` instead,
-    equal to ``linear`` followed by ``glu_bounded``."""
+    equal to ``linear`` followed by ``glu_bounded`` (``row_scale``: as there, with ``bounded`` only)."""
+    _need(row_scale, "row_scale", torch.float32)
+    if row_scale is not None and (bounded is None or row_scale.numel() < a.shape[0]):
+        raise KernelError("linear_glu: one row_scale per row, and it goes with bounded")
     _need(a, "a", torch.bfloat16, contiguous=False); _need(weight, "weight", torch.bfloat16)
     _need(out, "out", torch.bfloat16, contiguous=False)
     m, k = a.shape
@@ -826,7 +879,7 @@ def linear_glu(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bounded
         limit, alpha, shift = bounded[:3]
         act = bounded[3] if len(bounded) > 3 else "sigmoid"
         _call(_fn("gemm", "bfloat16", "erb_linear_skinny_glu_bounded"), a.data_ptr(), weight.data_ptr(), out.data_ptr(), m, n, k,
-              lda, k, ldo, float(limit), float(alpha), float(shift), GLU_ACTS[act], _stream())
+              lda, k, ldo, float(limit), float(alpha), float(shift), GLU_ACTS[act], _ptr(row_scale), _stream())
         return
     _call(_fn("gemm", "bfloat16", "erb_linear_skinny_glu"), a.data_ptr(), weight.data_ptr(), out.data_ptr(), m, n, k,
           lda, k, ldo, _stream())
@@ -1415,7 +1468,7 @@ def moe_route_few(n_tokens: int, n_experts: int, top: int, dtype: torch.dtype = 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Tensor, score: torch.Tensor,
               tile_rows: int = 0, scores: str = "sigmoid", groups: tuple[int, int] | None = None,
               correction: torch.Tensor | None = None, group_score: str = "best", normalise: bool = False,
-              logits: torch.Tensor | None = None) -> None:
+              logits: torch.Tensor | None = None, weight: float = 1.0, side_gate: torch.Tensor | None = None) -> None:
     """Route every row of ``x`` (element type, row-strided view allowed): logits ``w_router x`` in float (``w_router``
     float ``[experts, width]``), the ``top`` largest chosen (the lower index wins a tie), ``score`` float ``[tokens *
     top]`` their sigmoids; ``lists`` (int32, ``moe_lists_ints`` entries) receives the choices and, per expert, the list
@@ -1427,12 +1480,17 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     choice goes by score + correction, while ``score`` stays without it; ``group_score = "top2_sum"``: a group counts as
     much as the sum of its two best experts (in what the choice goes by); ``normalise``: the chosen scores are divided by
     their sum (+ 1e-20).  ``logits`` (float scratch ``[tokens, experts]``, where ``moe_route_few`` says so): the pair of
-    kernels for few tokens is used, with the same results to the bit."""
-    _need(logits, "logits", torch.float32)
+    kernels for few tokens is used, with the same results to the bit.  ``weight`` multiplies the scores at last.  ``side_gate``
+    (float ``[tokens]``): ``w_router`` has one row more than there are experts, and the sigmoid of its logit is left there
+    (``logits`` then are ``[tokens, experts + 1]``)."""
+    _need(logits, "logits", torch.float32); _need(side_gate, "side_gate", torch.float32)
+    n_experts = w_router.shape[0] - (side_gate is not None)
+    if side_gate is not None and side_gate.numel() < x.shape[0]:
+        raise KernelError("moe_route: one side_gate per token")
     if logits is not None and tuple(logits.shape) != (x.shape[0], w_router.shape[0]):
         raise KernelError("moe_route: logits are [tokens, experts]")
     _need(correction, "correction", torch.float32)
-    if correction is not None and correction.numel() != w_router.shape[0]:
+    if correction is not None and correction.numel() != n_experts:
         raise KernelError("moe_route: one correction per expert")
     if group_score not in MOE_GROUP_SCORES:
         raise KernelError(f"moe_route: unknown group score {group_score!r}; known: {sorted(MOE_GROUP_SCORES)}")
@@ -1440,14 +1498,13 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, lists: torch.Te
     n_groups, keep = groups if groups else (1, 1)
     _need(score, "score", torch.float32)
     n, width = x.shape
-    n_experts = w_router.shape[0]
     if w_router.shape[1] != width or x.stride(1) != 1 or score.numel() < n * top:
         raise KernelError("moe_route: shapes disagree")
     choice, order, counts, offsets, tiles = _moe_lists(lists, n, n_experts, top)
     _call(_fn("moe", _elem(x), "erb_moe_route"), x.data_ptr(), x.stride(0) if n > 1 else width, w_router.data_ptr(), n, width,
           n_experts, int(top), choice.data_ptr(), score.data_ptr(), counts.data_ptr(), offsets.data_ptr(), tiles.data_ptr(),
           order.data_ptr(), int(tile_rows), MOE_SCORES[scores], int(n_groups), int(keep), _ptr(correction),
-          MOE_GROUP_SCORES[group_score], int(bool(normalise)),
+          MOE_GROUP_SCORES[group_score], int(bool(normalise)), float(weight), _ptr(side_gate),
           _ptr(logits), _stream())
 
 
@@ -1584,15 +1641,27 @@ def _penalty(penalty: torch.Tensor | None, n_q_heads: int) -> int | None:
     return _ptr(penalty)
 
 
+def _gate(gate: torch.Tensor | None, out: torch.Tensor, width: int) -> tuple[int | None, int]:
+    """The (pointer, row stride) of an output gate: rows of ``width`` entries beside the rows of ``out``."""
+    if gate is None:
+        return None, 0
+    _need(gate, "gate", out.dtype, contiguous=False)
+    if gate.shape[0] < out.shape[0] or gate.shape[1] != width or gate.stride(1) != 1:
+        raise KernelError("attention: an output gate has a row of heads for every output row")
+    return gate.data_ptr(), gate.stride(0) if gate.shape[0] > 1 else max(width, gate.stride(0))
+
+
 def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_tables: torch.Tensor,
                    seq_of_token: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                    scale: float, window: int = 0, keep_first: int = 0, chunk: int = 0,
-                   penalty: torch.Tensor | None = None) -> None:
+                   penalty: torch.Tensor | None = None, softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """Causal attention of every token over its sequence's pages (general kernel, any portion sizes).
     ``window`` > 0: a query sees the last ``window`` keys (its own included) and the first ``keep_first`` of the sequence.
     ``chunk`` > 0 (instead of a window): a query sees the earlier keys of its own run of ``chunk`` positions, runs
     counted from position 0 of the sequence.  ``penalty`` float ``[2, n_q_heads]`` (``r1``, then ``r2`` of every query
-    head): the scaled score of a key ``d`` positions back is lowered by ``r1 * ln(1 + r2 * d)``.
+    head): the scaled score of a key ``d`` positions back is lowered by ``r1 * ln(1 + r2 * d)``.  ``softcap`` c > 0 (instead of
+    a penalty): the scaled score s becomes ``c * tanh(s / c)``.  ``gate`` (a row-strided view beside ``out``): every output
+    entry is multiplied by the sigmoid of its entry of the gate, in float before it is rounded.
 
     ``q``: ``[tokens, >= n_q_heads * D]`` view with unit inner stride (the q part of a qkv buffer);
     ``out``: ``[tokens, n_q_heads * D]``; pages ``[n_pages, n_kv_heads, page_size, D]``;
@@ -1608,7 +1677,7 @@ def attention_rows(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     _call(_fn("attention", _elem(q), "erb_attention_rows"), q.data_ptr(), q.stride(0), k_pages.data_ptr(),
           v_pages.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], seq_of_token.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), n, n_q_heads, nkv, d, page_size, mask_reach(window, chunk),
-          int(keep_first), float(scale), _penalty(penalty, n_q_heads), _stream())
+          int(keep_first), float(scale), _penalty(penalty, n_q_heads), float(softcap), *_gate(gate, out, n_q_heads * d), _stream())
 
 
 _sm_counts: dict[int, int] = {}
@@ -1727,10 +1796,10 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
                      token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                      scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
                      window: int = 0, split_keys: int = DECODE_SPLIT_KEYS, keep_first: int = 0, chunk: int = 0,
-                     penalty: torch.Tensor | None = None) -> None:
+                     penalty: torch.Tensor | None = None, softcap: float = 0.0, gate: torch.Tensor | None = None) -> None:
     """Attention of one new token per sequence, keys cut into splits of ``split_keys`` (split-KV).
     With a window the first ``keep_first`` keys stay visible; the first split of the window takes them along.
-    ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``; ``penalty``: as there.
+    ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``; ``penalty``, ``softcap``, ``gate``: as there.
 
     ``token_of_seq`` int32 ``[sequences]`` gives each sequence's row in q/out/positions.  Scratch:
     ``part_acc`` float ``[sequences * heads * max_splits * D]``, ``part_ml`` twice
@@ -1751,7 +1820,7 @@ def attention_decode(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
           v_pages.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], token_of_seq.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(),
           max_splits, n_seqs, n_q_heads, nkv, d, page_size, mask_reach(window, chunk), int(keep_first), int(split_keys),
-          float(scale), _penalty(penalty, n_q_heads), _stream())
+          float(scale), _penalty(penalty, n_q_heads), float(softcap), *_gate(gate, out, n_q_heads * d), _stream())
 
 
 def decode_bulk_supported(dtype: torch.dtype, head_dim: int, window: int, n_q_heads: int, n_kv_heads: int,
@@ -1789,7 +1858,8 @@ def attention_decode_bulk(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
                           token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                           scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
                           status: torch.Tensor, split_keys: int = DECODE_SPLIT_KEYS, head_group: int = 0, window: int = 0,
-                          keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
+                          keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None, softcap: float = 0.0,
+                          gate: torch.Tensor | None = None) -> None:
     """``attention_decode`` for bfloat16 with keys and values streamed by bulk asynchronous copies.
     ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``.
     ``window`` > 0: the last ``window`` keys and the first ``keep_first``; the splits are counted from the one
@@ -1814,7 +1884,7 @@ def attention_decode_bulk(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(), max_splits,
           n_seqs, n_q_heads, nkv, d, page_size, int(split_keys), float(scale), status.data_ptr(),
           split_counters(q.device, n_seqs * nkv).data_ptr(), int(head_group), mask_reach(window, chunk), int(keep_first),
-          _penalty(penalty, n_q_heads), _stream())
+          _penalty(penalty, n_q_heads), float(softcap), *_gate(gate, out, n_q_heads * d), _stream())
 
 
 @functools.lru_cache(maxsize=4096)
@@ -1832,7 +1902,8 @@ def attention_decode_gqa(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          token_of_seq: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_q_heads: int,
                          scale: float, part_acc: torch.Tensor, part_ml: torch.Tensor, max_splits: int,
                          status: torch.Tensor, split_keys: int = DECODE_SPLIT_KEYS, window: int = 0, keep_first: int = 0,
-                         chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
+                         chunk: int = 0, penalty: torch.Tensor | None = None, softcap: float = 0.0,
+                         gate: torch.Tensor | None = None) -> None:
     """``attention_decode`` for several query heads per kv head on tensor cores (``window`` and ``keep_first`` as in
     ``attention_decode_bulk``): the query heads of a
     kv head are the rows of one matrix tile, pages arrive by TMA tensor copies."""
@@ -1853,7 +1924,7 @@ def attention_decode_gqa(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
           positions.data_ptr(), out.data_ptr(), out.stride(0), part_acc.data_ptr(), part_ml.data_ptr(), max_splits,
           n_seqs, n_q_heads, nkv, d, page_size, int(split_keys), float(scale), status.data_ptr(),
           split_counters(q.device, n_seqs * nkv).data_ptr(), mask_reach(window, chunk), int(keep_first),
-          _penalty(penalty, n_q_heads), _stream())
+          _penalty(penalty, n_q_heads), float(softcap), *_gate(gate, out, n_q_heads * d), _stream())
 
 
 #: query rows of one (sequence, head) that a block of the tensor-core prefill kernel takes
@@ -1894,7 +1965,8 @@ def attention_prefill_tc(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
                          seq_starts: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, n_blocks: int,
                          n_q_heads: int, scale: float, status: torch.Tensor, key_splits: int = 1, first_row: int = 0,
                          part_o: torch.Tensor | None = None, part_ml: torch.Tensor | None = None, window: int = 0,
-                         keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None) -> None:
+                         keep_first: int = 0, chunk: int = 0, penalty: torch.Tensor | None = None, softcap: float = 0.0,
+                         gate: torch.Tensor | None = None) -> None:
     """Causal attention of prompt portions on tcgen05 tensor cores (bfloat16, head_dim 64).  ``window`` > 0: a
     query sees the last ``window`` keys (its own included) and the first ``keep_first`` of its sequence.
     ``chunk`` > 0 (instead of a window): the mask of chunks of ``attention_rows``.
@@ -1924,7 +1996,8 @@ def attention_prefill_tc(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
           v_pages.data_ptr(), n_pages, block_tables.data_ptr(), block_tables.shape[1], seq_starts.data_ptr(),
           positions.data_ptr(), out.data_ptr(), out.stride(0), n_seqs, int(n_blocks), n_q_heads, nkv, d, page_size,
           float(scale), status.data_ptr(), int(key_splits), int(first_row), qkv.shape[0] - int(first_row), _ptr(part_o), _ptr(part_ml),
-          mask_reach(window, chunk), int(keep_first), _penalty(penalty, n_q_heads), _stream())
+          mask_reach(window, chunk), int(keep_first), _penalty(penalty, n_q_heads), float(softcap),
+          *_gate(gate, out, n_q_heads * d), _stream())
     if key_splits > 1:
         launch_counts["own"] += 1          # the merge of the ranges
 

@@ -26,6 +26,13 @@ the last ``conv - 1`` biased inputs of every channel live in a state record.  Wi
 ``[heads]``, ``r1`` and ``r2``) the scaled score of a key ``d`` positions back is lowered by ``r1 ln(1 + r2 d)``; every
 attention kernel takes it.
 
+Three more options go with the second family: ``softcap`` c (every scaled score s becomes ``c * tanh(s / c)``); ``gate`` (the name of
+a tensor ``[heads * v_dim, hidden]``: the concatenated heads are multiplied entry by entry by the sigmoid of its product with the
+mixer's input; its rows are stored below those of q, k and v, so that one product makes the logits too, and the attention kernels
+multiply as they write); ``value_mix`` (``"first"``: the layer leaves its values for the layers after it; ``"blend"``: the cached
+values are ``(1 - l) v + l v'`` with the values ``v'`` that the ``"first"`` layer made of the same tokens and ``l`` the one number of the
+tensor ``vmix``).
+
 Heads whose sizes differ or are no multiple of 8 are stored padded with zeros to one size ``D``:
 scores and outputs are unchanged, and the norm's mean divides by the true count.
 
@@ -52,7 +59,8 @@ class Attention(Mixer):
                  scale: float | None = None, keep_first: int = 0, qk_bias: bool = False, qk_norm_eps: float | None = None,
                  values_are_keys: bool = False, names: dict[str, str] | None = None, chunk: int = 0, v_dim: int | None = None,
                  all_bias: bool = False, whole_norm_eps: float | None = None, qkv_bias: bool = False, conv: int = 0,
-                 penalty: tuple[str, str] | None = None) -> None:
+                 penalty: tuple[str, str] | None = None, softcap: float = 0.0, gate: str | None = None,
+                 value_mix: str | None = None, vmix: str = "vmix") -> None:
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads are not divisible by {n_kv_heads} kv heads")
         self.chunk = int(chunk or 0)
@@ -66,7 +74,16 @@ class Attention(Mixer):
         #: the second family's kernel handles padded heads, a norm over the projection and the four biases
         self.qkv_bias, self.taps = bool(qkv_bias), int(conv or 0)
         self.conv_form = self.qkv_bias or self.taps > 0
-        self.whole = self.conv_form or self.all_bias or whole_norm_eps is not None or padded != self.qk_dim or self.v_dim != self.qk_dim
+        self.softcap, self.gate_name, self.value_mix, self.vmix_name = float(softcap or 0.0), gate, value_mix, vmix
+        self.whole = (self.conv_form or self.all_bias or whole_norm_eps is not None or padded != self.qk_dim or self.v_dim != self.qk_dim
+                      or gate is not None or value_mix is not None)
+        if value_mix not in (None, "first", "blend") or (value_mix and not own_kv):
+            raise ValueError(f"attention: value_mix {value_mix!r}; known: first, blend, of a layer with values of its own")
+        if self.softcap < 0 or (self.softcap and penalty):
+            raise ValueError("attention: a cap of the scores is positive and excludes a penalty")
+        if self.conv_form and (gate is not None or value_mix is not None):
+            raise ValueError("attention: a convolution or biases on q, k and v exclude an output gate and blended values")
+        self.blend: torch.Tensor | None = None
         if self.taps < 0 or (self.conv_form and (self.all_bias or whole_norm_eps is not None or not own_kv or position.kind != "none")):
             raise ValueError("attention: a convolution or biases on q, k and v exclude a norm, another layer's keys and a position encoding")
         self.penalty_names, self.penalty = tuple(penalty) if penalty else None, None
@@ -95,6 +112,9 @@ class Attention(Mixer):
         self.in_width = self.q_width + (1 if self.values_are_keys else 2) * self.kv_width
         if self.whole and not own_kv:
             self.in_width = self.q_width         # queries only: keys and values are another layer's
+        self.gate_off = self.in_width
+        if gate is not None:
+            self.in_width += self.q_width        # the output gate's logits, padded as the heads are
         self.w_qkv: torch.Tensor | None = None
         self.w_o: torch.Tensor | None = None
 
@@ -135,6 +155,10 @@ class Attention(Mixer):
                 specs += [WeightSpec(nm["k_bias"], (k_true,), "vector32"), WeightSpec(nm["v_bias"], (v_true,), "vector32")]
             if self.whole_norm_eps is not None:
                 specs.append(WeightSpec(nm["k_norm"], (k_true,), "vector32"))
+        if self.gate_name is not None:
+            specs.append(WeightSpec(self.gate_name, (self.n_q * self.v_dim, self.hidden)))
+        if self.value_mix is not None:           # (a checkpoint has the first layer's too; it is not used)
+            specs.append(WeightSpec(self.vmix_name, (), "vector32"))
         specs.append(WeightSpec(nm["o"], (self.hidden, self.n_q * self.v_dim)))
         if self.all_bias:
             specs.append(WeightSpec(nm["o_bias"], (self.hidden,), "vector32"))
@@ -155,6 +179,10 @@ class Attention(Mixer):
         if self.own_kv:
             parts += [self._pad_heads(tensors[nm["k"]], self.n_kv, self.qk_dim, self.dtype),
                       self._pad_heads(tensors[nm["v"]], self.n_kv, self.v_dim, self.dtype)]
+        if self.gate_name is not None:
+            parts.append(self._pad_heads(tensors[self.gate_name], self.n_q, self.v_dim, self.dtype))
+        if self.value_mix == "blend":
+            self.blend = tensors[self.vmix_name].to(device=self.device, dtype=f32).reshape(1).contiguous()
         self.w_qkv = torch.cat(parts, dim=0).contiguous()
         w_o = tensors[nm["o"]].to(device=self.device, dtype=self.dtype)            # [hidden, heads * v_dim]: pad the columns
         self.w_o = self._pad_heads(w_o.t(), self.n_q, self.v_dim, self.dtype).t().contiguous()
@@ -204,12 +232,16 @@ class Attention(Mixer):
             if getattr(pos, "pairs", False):
                 raise ValueError("attention: with these options positions turn the halves of a head's first entries")
             kernels.linear(x, self.w_qkv, qkv)
+            first = None
+            if self.value_mix is not None:       # (one buffer of a step: written by the first such layer, read by the others)
+                first = ctx.buf("attn.first_values", (x.shape[0], self.n_kv * self.v_dim), self.dtype)
             kernels.qkv_whole_norm(qkv, ctx.positions, self.n_q, self.n_kv, d, q_count=self.n_q * self.qk_dim,
                                    k_count=self.n_kv * self.qk_dim, eps=self.whole_norm_eps or 0.0, q_bias=self.q_bias,
                                    k_bias=self.k_bias, v_bias=self.v_bias, q_norm=self.q_norm, k_norm=self.k_norm,
                                    inv_freq=getattr(pos, "inv_freq", None), rot_dim=getattr(pos, "rot_dim", 0),
                                    has_kv=self.own_kv, slots=slots, k_pages=None if pages is None else pages[0],
-                                   v_pages=None if pages is None else pages[1], page_size=ctx.page_size)
+                                   v_pages=None if pages is None else pages[1], page_size=ctx.page_size, first_values=first,
+                                   blend=self.blend)
             return
         if self.qk_bias or self.qk_norm_eps is not None or self.values_are_keys:
             pos = self.position
@@ -244,6 +276,9 @@ class Attention(Mixer):
         else:
             self._prepare(x, qkv, ctx, pages, slots)
         out = ctx.buf("attn.out", (n, self.q_width), self.dtype)
+        gate = None if self.gate_name is None else qkv[:, self.gate_off: self.gate_off + self.q_width]
+        score = {"penalty": self.penalty, "softcap": self.softcap}
+        head_gate = gate if gate is None else gate[: ctx.n_decode]
         tables = ctx.block_tables[group]
         nd = ctx.n_decode
         reach_mask = self.window or self.chunk                  # keys a token can see under its mask (0: all before it)
@@ -271,16 +306,17 @@ class Attention(Mixer):
             if may_group and kernels.decode_gqa_supported(self.dtype, d, self.window, self.n_q, self.n_kv, ctx.page_size, split, max_splits):
                 kernels.attention_decode_gqa(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                              out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits, ctx.status,
-                                             split_keys=split, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
+                                             split_keys=split, window=self.window, keep_first=self.keep_first, chunk=self.chunk, gate=head_gate, **score)
             elif kernels.decode_bulk_supported(self.dtype, d, self.window, self.n_q, self.n_kv, max_splits):
                 kernels.attention_decode_bulk(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                               out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits, ctx.status,
                                               split_keys=split, head_group=heads_per_block, window=self.window,
-                                              keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
+                                              keep_first=self.keep_first, chunk=self.chunk, gate=head_gate, **score)
             else:
                 kernels.attention_decode(qkv[:nd], k_pages, v_pages, tables, ctx.token_of_seq[:nd], ctx.positions,
                                          out[:nd], self.n_q, self.scale, part_acc, part_ml, max_splits,
-                                         window=self.window, split_keys=split, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
+                                         window=self.window, split_keys=split, keep_first=self.keep_first, chunk=self.chunk,
+                                         gate=head_gate, **score)
         if n > nd and kernels.prefill_tc_supported(self.dtype, d, self.window, ctx.page_size):
             blocks = kernels.prefill_tc_blocks(ctx.host_q_len[nd:])
             # a portion that is short against its past: its few blocks' keys are cut into ranges
@@ -295,10 +331,11 @@ class Attention(Mixer):
                 part_ml = ctx.buf("attn.range_ml", (need_ml,), torch.float32)
             kernels.attention_prefill_tc(qkv, k_pages, v_pages, tables[nd:], ctx.seq_starts[nd:], ctx.positions, out, blocks,
                                          self.n_q, self.scale, ctx.status, key_splits=ranges, first_row=nd, part_o=part_o,
-                                         part_ml=part_ml, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
+                                         part_ml=part_ml, window=self.window, keep_first=self.keep_first, chunk=self.chunk, gate=gate, **score)
         elif n > nd:
             kernels.attention_rows(qkv[nd:], k_pages, v_pages, tables, ctx.seq_of_token[nd:], ctx.positions[nd:],
-                                   out[nd:], self.n_q, self.scale, window=self.window, keep_first=self.keep_first, chunk=self.chunk, penalty=self.penalty)
+                                   out[nd:], self.n_q, self.scale, window=self.window, keep_first=self.keep_first, chunk=self.chunk,
+                                   gate=gate if gate is None else gate[nd:], **score)
         return self._project_out(out, ctx)
 
     def _project_out(self, out: torch.Tensor, ctx) -> torch.Tensor:

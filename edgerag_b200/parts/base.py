@@ -167,6 +167,8 @@ class Part:
     graph_safe = False
     #: ``forward`` looks at the tokens' ids: steps that bring rows of embeddings instead are refused
     needs_token_ids = False
+    #: sequences of more tokens than this cannot run through the part (None: any length)
+    max_positions: int | None = None
 
     def weight_specs(self) -> list[WeightSpec]:
         return []

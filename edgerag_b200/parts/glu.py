@@ -50,15 +50,16 @@ class BoundedGLU(FeedForward):
         self.forward_into(x, ctx, y)
         return y
 
-    def forward_into(self, x: torch.Tensor, ctx, y: torch.Tensor) -> None:
-        """The update written to ``y``: rows of the element type or float32 (one of a sum of parts that a caller keeps)."""
+    def forward_into(self, x: torch.Tensor, ctx, y: torch.Tensor, row_scale: torch.Tensor | None = None) -> None:
+        """The update written to ``y``: rows of the element type or float32 (one of a sum of parts that a caller keeps).
+        ``row_scale``: a float per row that multiplies the row's activation."""
         n = x.shape[0]
         act = ctx.buf("ffn.act", (n, self.intermediate), self.dtype)
         if kernels.linear_glu_supported(x, self.w_gate_up):
             # a few rows: product and gate in one kernel, the same bits as the two kernels below
-            kernels.linear_glu(x, self.w_gate_up, act, bounded=(self.limit, self.alpha, self.shift, self.act))
+            kernels.linear_glu(x, self.w_gate_up, act, bounded=(self.limit, self.alpha, self.shift, self.act), row_scale=row_scale)
         else:
             gate_up = ctx.buf("ffn.gate_up", (n, 2 * self.intermediate), self.dtype)
             kernels.linear(x, self.w_gate_up, gate_up)
-            kernels.glu_bounded(gate_up, act, self.limit, self.alpha, self.shift, self.act)
+            kernels.glu_bounded(gate_up, act, self.limit, self.alpha, self.shift, self.act, row_scale=row_scale)
         kernels.linear(act, self.w_down, y)

@@ -15,7 +15,10 @@ goes by the largest); ``groups = (count, keep)``: the experts form ``count`` equ
 is its best expert's, and only experts of the ``keep`` best groups can be chosen; ``gated = False`` with ``act =
 "relu_squared"``: experts without a gate branch, ``W_down relu(W_up r)^2`` (tensors ``e<i>.{up, down}``); ``correction`` (a tensor's name, sigmoid scores): the choice goes
 by ``s + correction``, the weights by ``s``; ``group_score = "top2_sum"``: a group counts as much as the sum of its two best
-experts.
+experts; ``weight_scale``: a constant that multiplies every weight at last; ``shared_gate`` (a tensor's name, ``[1, hidden]``): the
+shared expert's output is multiplied by ``sigmoid(w . x)``, one number per token.  That row is stored below the router's: its logit
+is made with the experts' and the shared expert's activation kernel takes the sigmoid per row (a constant per row commutes with
+the down product).
 
 Nothing here goes through the host: the router's kernel leaves, on the device, every expert's list of (token, choice)
 pairs, and the two product kernels walk row tiles of those lists, so the launches of a step depend on its number of
@@ -39,7 +42,8 @@ class RoutedExperts(FeedForward):
                  shared: PartSpec | None = None, weights: str = "score", scale_input: bool = True,
                  names: tuple[str, str, str] = ("gate", "up", "down"), router: str = "router", expert: str = "e{}.",
                  scores: str = "sigmoid", groups: tuple[int, int] | None = None, gated: bool = True,
-                 act: str = "silu", correction: str | None = None, group_score: str = "best") -> None:
+                 act: str = "silu", correction: str | None = None, group_score: str = "best", weight_scale: float = 1.0,
+                 shared_gate: str | None = None) -> None:
         if not 0 < top <= n_experts:
             raise ValueError(f"routed_experts: top {top} of {n_experts} experts")
         if weights not in ("score", "score_normed"):
@@ -48,6 +52,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: a correction and groups that count their two best go with sigmoid scores")
         self.normalise, self.correction_name, self.group_score = weights == "score_normed", correction, group_score
         self.correction: torch.Tensor | None = None
+        self.weight_scale, self.shared_gate = float(weight_scale), shared_gate
+        if shared_gate is not None and shared is None:
+            raise ValueError("routed_experts: a gate of the shared expert without a shared expert")
         if scores not in kernels.MOE_SCORES:
             raise ValueError(f"routed_experts: scores {scores!r}; known: {sorted(kernels.MOE_SCORES)}")
         if (gated and act != "silu") or (not gated and act != "relu_squared"):
@@ -76,6 +83,8 @@ class RoutedExperts(FeedForward):
             if self.gated:
                 specs.append(WeightSpec(pre + gate, (self.intermediate, self.hidden)))
             specs += [WeightSpec(pre + up, (self.intermediate, self.hidden)), WeightSpec(pre + down, (self.hidden, self.intermediate))]
+        if self.shared_gate is not None:
+            specs.append(WeightSpec(self.shared_gate, (1, self.hidden), "vector32"))
         if self.shared is not None:
             specs += [WeightSpec(self._shared_prefix + s.name, s.shape, s.kind, s.fallback) for s in self.shared.weight_specs()]
         return specs
@@ -84,6 +93,9 @@ class RoutedExperts(FeedForward):
         gate, up, down = self.names
         cast = lambda t: t.to(device=self.device, dtype=self.dtype)  # noqa: E731
         self.w_router = tensors[self.router_name].to(device=self.device, dtype=torch.float32).contiguous()
+        if self.shared_gate is not None:
+            side = tensors[self.shared_gate].to(device=self.device, dtype=torch.float32)
+            self.w_router = torch.cat([self.w_router, side], 0).contiguous()
         if self.correction_name is not None:
             self.correction = tensors[self.correction_name].to(device=self.device, dtype=torch.float32).contiguous()
         pres = [self.expert_fmt.format(e) for e in range(self.n_experts)]
@@ -102,9 +114,12 @@ class RoutedExperts(FeedForward):
         act = ctx.buf("moe.act", (n * top, self.intermediate), self.dtype)
         parts = ctx.buf("ffn.out_parts", (top + (self.shared is not None), n, self.hidden), torch.float32)
         route = dict(scores=self.scores, groups=self.groups, correction=self.correction, group_score=self.group_score,
-                     normalise=self.normalise)
+                     normalise=self.normalise, weight=self.weight_scale)
+        row_scale = None
+        if self.shared_gate is not None:
+            row_scale = route["side_gate"] = ctx.buf("moe.side_gate", (n,), torch.float32)
         if kernels.moe_route_few(n, self.n_experts, top, self.dtype):
-            route["logits"] = ctx.buf("moe.logits", (n, self.n_experts), torch.float32)
+            route["logits"] = ctx.buf("moe.logits", (n, self.w_router.shape[0]), torch.float32)
         in_score, out_score = (score, None) if self.scale_input else (None, score)
         if kernels.moe_tc_supported(self.dtype, self.hidden, self.intermediate):
             # tensor cores: row tiles sized by the step's tokens, the (scaled) rows gathered once in list order
@@ -127,5 +142,8 @@ class RoutedExperts(FeedForward):
                 kernels.moe_up_act(x, self.w_gate_up, lists, top, act)
             kernels.moe_down(act, self.w_down, lists, top, parts, out_score=out_score)
         if self.shared is not None:
-            self.shared.forward_into(x, ctx, parts[top])
+            if row_scale is None:
+                self.shared.forward_into(x, ctx, parts[top])
+            else:
+                self.shared.forward_into(x, ctx, parts[top], row_scale=row_scale)
         return parts
