@@ -13,7 +13,8 @@ What the reference spreads over ``BlockTable`` (edgerag/cache/block_table.py:26-
   so a failed growth leaves the request untouched.
 * Pages go back to the pool when the request is released, or, in a windowed group, as soon as no
   later query can see any key of the page.  A windowed group may keep its first tokens visible for
-  good (``keep_first``): the pages that hold any of them are never given back early.
+  good (``keep_first``): the pages that hold any of them are never given back early.  Under a mask of chunks
+  (``chunk``) the pages of a chunk go back once the sequence has left it.
 * Beside the pages, every request holds one **state slot**: the index of a fixed-size record in
   each state tensor that a mixer registered (none for the Llama decoder).  Slots are zeroed when
   handed out.
@@ -46,6 +47,8 @@ class KVGroupSpec:
     v_head_dim: int | None = None
     #: with a window: the first tokens of a sequence that stay visible whatever the distance
     keep_first: int = 0
+    #: a query sees the keys of its own run of this many positions only (runs counted from position 0; 0: no such mask)
+    chunk: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -150,7 +153,8 @@ class CacheManager:
         """Upper bound, per group, of the pages a request holds at any time on its way to ``final_tokens``.
 
         A group without a window holds every page.  A windowed group holds the pages that the
-        window and one step's new tokens can touch.
+        window and one step's new tokens can touch, a group under a mask of chunks those of the chunk it is in and of one
+        step's new tokens.
         """
         out = []
         for g in self.layout.groups:
@@ -158,6 +162,8 @@ class CacheManager:
             if g.window > 0:
                 span = g.window + max(1, max_step_tokens)
                 out.append(min(full, self.pages_for(span) + 1 + self.pages_for(g.keep_first)))
+            elif g.chunk > 0:
+                out.append(min(full, self.pages_for(g.chunk + max(1, max_step_tokens)) + 1))
             else:
                 out.append(full)
         return out
@@ -217,7 +223,7 @@ class CacheManager:
         return out
 
     def advance(self, request_id: object, n_new: int) -> None:
-        """Record ``n_new`` written tokens and give back pages that a window has passed."""
+        """Record ``n_new`` written tokens and give back pages that a window or the current chunk has passed."""
         rc = self.requests[request_id]
         need = self.pages_for(rc.num_tokens + n_new)
         if any(len(t.pages) < need for t in rc.tables):
@@ -225,11 +231,12 @@ class CacheManager:
         rc.num_tokens += n_new
         ps = self.page_size
         for gi, (g, t) in enumerate(zip(self.layout.groups, rc.tables)):
-            if g.window <= 0:
+            if g.window <= 0 and g.chunk <= 0:
                 continue
-            # A later query sits at position >= num_tokens and sees keys > position - window, so
-            # keys <= num_tokens - window are dead; page i is dead when its last key is.
-            dead_upto = rc.num_tokens - g.window
+            # A later query sits at position >= num_tokens and sees keys > position - window (or from its chunk's first
+            # position on), so keys <= num_tokens - window (or those of earlier chunks) are dead; page i is dead when its
+            # last key is.
+            dead_upto = rc.num_tokens - g.window if g.window > 0 else rc.num_tokens // g.chunk * g.chunk - 1
             t.kept = min(self.pages_for(g.keep_first), len(t.pages))
             t.first_live = max(t.first_live, t.kept)
             while t.first_live < len(t.pages) and (t.first_live + 1) * ps - 1 <= dead_upto:

@@ -8,6 +8,8 @@ cache layers exist, how they group, which state records) and the full list of ch
 
 from __future__ import annotations
 
+import dataclasses
+
 import torch
 
 from ..cache.manager import CacheLayout, KVGroupSpec, StateSpec
@@ -87,7 +89,9 @@ class DecoderModel:
                 if isinstance(item, KVGroupSpec):
                     if layout.placement[cl] is not None:
                         raise ValueError(f"layer {layer}: a mixer keeps one group of pages at most")
-                    key = (item.n_kv_heads, item.head_dim, item.window, item.v_head_dim, item.keep_first)
+                    if item.chunk and any(getattr(self.blocks[c.layer].mixer, "chunk", 0) != item.chunk for c in calls if c.cache_layer == cl):
+                        item = dataclasses.replace(item, chunk=0)     # another layer reads these pages under another mask
+                    key = (item.n_kv_heads, item.head_dim, item.window, item.v_head_dim, item.keep_first, item.chunk)
                     if key not in keys:
                         keys.append(key)
                         counts.append(0)

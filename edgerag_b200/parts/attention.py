@@ -19,8 +19,8 @@ A second family of options, also one kernel after the product (``kernels.qkv_who
 projections (``all_bias``; the output's rides with the update to whoever adds it), a unit-RMS norm over a token's whole
 query projection and whole key projection with a weight per entry (``whole_norm_eps``), values of another size than
 queries and keys (``v_dim``), and a mask of chunks (``chunk``: a query sees the earlier keys of its own run of ``chunk``
-positions, runs counted from the sequence's start; no key is ever out of every later query's sight, so the cache
-keeps all pages).  A third (``kernels.qkv_conv``): biases on q, k and v only (``qkv_bias``) and a short causal convolution over time on every
+positions, runs counted from the sequence's start; the cache gives the pages of a chunk back once the sequence has left
+it).  A third (``kernels.qkv_conv``): biases on q, k and v only (``qkv_bias``) and a short causal convolution over time on every
 channel of q, k and v, directly after the projection (``conv`` taps, tensors ``<name>.conv`` of shape ``[channels, taps]``);
 the last ``conv - 1`` biased inputs of every channel live in a state record.  With ``penalty`` (the names of two tensors
 ``[heads]``, ``r1`` and ``r2``) the scaled score of a key ``d`` positions back is lowered by ``r1 ln(1 + r2 d)``; every
@@ -119,7 +119,7 @@ class Attention(Mixer):
         self.w_o: torch.Tensor | None = None
 
     def cache_spec(self) -> KVGroupSpec | list:
-        pages = KVGroupSpec(1, self.n_kv, self.head_dim, self.window, keep_first=self.keep_first)
+        pages = KVGroupSpec(1, self.n_kv, self.head_dim, self.window, keep_first=self.keep_first, chunk=self.chunk)
         return [pages, StateSpec("attn_conv", (self.taps - 1, self.in_width))] if self.taps > 1 else pages
 
     def weight_specs(self) -> list[WeightSpec]:

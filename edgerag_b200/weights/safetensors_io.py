@@ -114,5 +114,5 @@ def write_safetensors(path: str | Path, tensors: dict[str, torch.Tensor], metada
         f.write(struct.pack("<Q", len(blob)))
         f.write(blob)
         for name in order:
-            t = tensors[name].detach().cpu().contiguous()
+            t = tensors[name].detach().cpu().contiguous().reshape(-1)      # (a single number has no dimension to view as bytes)
             f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")

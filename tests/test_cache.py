@@ -189,3 +189,37 @@ def test_pools_for_keys_and_values_of_different_widths():
     assert torch.isnan(k0[2]).all() and torch.isnan(v0[2]).all() and not torch.isnan(v0[3]).any()
     assert torch.isnan(k2[6]).all() and not torch.isnan(k2[:6]).any()
     assert pools.nbytes() == 4 * (5 * 2 * 2 * 3 * 4 * 16 + 6 * 4 * 56 + 7 * 2 * 4 * 24)
+
+
+def test_a_mask_of_chunks_gives_pages_back_when_the_chunk_is_left():
+    m = CacheManager(CacheLayout(groups=[KVGroupSpec(1, 1, 16, chunk=10)], placement=[(0, 0)]), page_size=4, num_pages=8, max_requests=1)
+    rc = m.admit("c")
+    total = 0
+    for n in (6, 3, 1, 1, 8, 1, 14, 5, 1):
+        m.grow("c", n)
+        assert all(p != NO_PAGE for p in rc.tables[0].pages[total // 4:])    # pages to be written are live
+        m.advance("c", n)
+        total += n
+        m.check_invariants()
+        dead_pages = total // 10 * 10 // 4       # whole pages before the chunk that the next token falls into
+        assert rc.tables[0].first_live == dead_pages
+        assert rc.tables[0].pages[:dead_pages] == [NO_PAGE] * dead_pages
+        assert m.held_pages("c") == [m.pages_for(total) - dead_pages]
+    assert m.peak_pages(1000, 14) == [min(250, m.pages_for(24) + 1)] and m.peak_pages(8, 14) == [2]
+    m.release("c")
+    assert m.free_pages() == [8] and len(m.drain_freed()) == 10
+
+
+def test_pages_read_under_two_masks_stay():
+    """A layer that reads another layer's pages under a larger chunk (or none) still needs what the owner's chunk has left."""
+    import torch
+
+    import plain_lozanex as plain
+    from edgerag_b200.config.registry import architecture_of
+    from edgerag_b200.models.decoder import DecoderModel
+
+    for sizes, chunk in (((24, 24), 24), ((24, 48), 0), ((24, None), 0)):
+        raw = plain.make_config([plain.attention_layer(size=sizes[0]), plain.attention_layer(size=sizes[1], kv_from=0)])
+        arch = architecture_of(raw)
+        model = DecoderModel(arch.make_plan(arch.read_config(raw, "t")), torch.float32, torch.device("cpu"))
+        assert [g.chunk for g in model.cache_layout.groups] == [chunk]

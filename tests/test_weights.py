@@ -137,3 +137,12 @@ def test_random_weights_mode_writes_a_loadable_folder(tmp_path):
     # the plain implementation reads the same folder
     logits = plain.forward(plain.read_weights(folder), plain.read_config(folder), [1, 2, 3])
     assert logits.shape == (3, 512) and torch.isfinite(logits).all()
+
+
+def test_a_tensor_without_dimensions_survives_a_file(tmp_path):
+    from edgerag_b200.weights.safetensors_io import SafetensorsFile, write_safetensors
+
+    for dtype in (torch.bfloat16, torch.float32, torch.int32):
+        write_safetensors(tmp_path / "one.safetensors", {"a": torch.tensor(3, dtype=dtype), "b": torch.arange(4).to(dtype)})
+        with SafetensorsFile(tmp_path / "one.safetensors") as f:
+            assert f.shape("a") == () and f.tensor("a").clone().item() == 3 and f.tensor("b").tolist() == [0, 1, 2, 3]
