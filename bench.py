@@ -630,6 +630,31 @@ def sabolorn_config(size: dict, n_layers: int) -> dict:
             "norm": {"eps": 1e-5}, "token_side": {"dim": size["width"] // 8}, "logit_softcap": 30.0, "layers": layers}
 
 
+#: the Kikarax sizes beside DESIGN_SIZES: heads of 64 with a quarter as many kv heads under chunks of 1,024, routed experts and the
+#: shared expert sized as Lozanex's
+KIKARAX_BUCKETS, KIKARAX_CAP = 40009, 30.0
+
+
+def kikarax_config(size: dict, n_layers: int, dense: bool = False) -> dict:
+    """Attention layers with capped scores, an output gate and blended values; every layer with routed experts and a shared expert, or
+    (``dense``) with the bounded gated feed-forward."""
+    heads = size["width"] // 64
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 64, "scale": 64 ** -0.5, "softcap": KIKARAX_CAP, "v_mix": True,
+           "mask": {"size": LOZANEX_CHUNK}}
+    mlp = {"kind": "dense", "ff": size["ff"], "limit": 7.0} if dense else {
+        "kind": "moe", "expert": {"ff": size["ff"] // 8}, "router": dict(LOZANEX_EXPERTS, scale=2.5), "shared": {"ff": size["ff"] // 2}}
+    return {"architecture": "Kikarax", "width": size["width"], "vocab": size["vocab"], "norm": {"eps": 1e-5}, "max_positions": 8192,
+            "embedding": {"scale": size["width"] ** 0.5, "bigram": {"buckets": KIKARAX_BUCKETS, "mul_prev": 31, "mul_cur": 17}},
+            "logit_scale": 0.5, "layers": [{"type": "attention", "mixer": dict(att), "mlp": mlp} for _ in range(n_layers)]}
+
+
+def lozanex_attention_config(size: dict, n_layers: int) -> dict:
+    """Lozanex of attention layers only, each with keys and values of its own: the framework's closest design to Kikarax."""
+    raw = lozanex_config(size, 2)
+    layer = raw["layers"][1]
+    return {**raw, "layers": [dict(layer, mixer=dict(layer["mixer"])) for _ in range(n_layers)]}
+
+
 def run_designs(args) -> dict:
     """Prefill (one portion of 2,048 tokens) and decode (batch 1 and --batch at a context of 2,048) of one design
     (--design) and of the Llama decoder at the same width, feed-forward size, vocabulary and number of layer
@@ -711,6 +736,8 @@ def run_designs(args) -> dict:
         return run_pudadra(args, measure, n_layers, block, clocks, peak_source, microbench)
     if args.design == "sabolorn":
         return run_sabolorn(args, measure, n_layers, block, clocks, peak_source, microbench)
+    if args.design == "kikarax":
+        return run_kikarax(args, measure, n_layers, block, clocks, peak_source, microbench)
     for name, size in DESIGN_SIZES.items():
         out[name] = {"layers": n_layers, "dokodra": measure(dokodra_config(size, n_layers), size["vocab"]),
                      "llama": measure(llama_config(size, n_layers), size["vocab"])}
@@ -969,6 +996,63 @@ def run_sabolorn(args, measure, n_layers: int, block: int, clocks, peak_source: 
             "sizes": out, "kernels": kern, "step_kernels": steps, "clocks": clocks.record()}
 
 
+def run_kikarax(args, measure, n_layers: int, block: int, clocks, peak_source: str, microbench) -> dict:
+    """Kikarax with routed experts beside Lozanex of attention layers, and with its dense feed-forward beside the Llama decoder with as
+    many kv heads, at equal width, layer count and feed-forward width per token; then its kernels beside the like kernels of
+    those at equal work, then which kernels a step of each spends its time in."""
+    import subprocess
+    import tempfile
+    import types
+
+    out: dict = {}
+    for name, size in DESIGN_SIZES.items():
+        kv = max(1, size["width"] // 64 // 4)
+        out[name] = {"layers": n_layers, "kikarax": measure(kikarax_config(size, n_layers), size["vocab"]),
+                     "lozanex_attention": measure(lozanex_attention_config(size, n_layers), size["vocab"]),
+                     "kikarax_dense": measure(kikarax_config(size, n_layers, dense=True), size["vocab"]),
+                     "llama": measure(llama_config(size, n_layers, kv), size["vocab"])}
+    size = DESIGN_SIZES["w2048"]
+    ns = lambda **kw: types.SimpleNamespace(dtype="bfloat16", iters=10, warmup=3, page=block, sequential_pages=False, **kw)  # noqa: E731
+    heads = dict(heads=32, kv_heads=8, head_dim=64)
+    moe = dict(width=size["width"], ff=size["ff"] // 8, **LOZANEX_EXPERTS)
+    capped = dict(softcap=KIKARAX_CAP, gate=True)
+    pre = lambda tokens, **kw: microbench.prefill_attention(ns(tokens=tokens, past=0, kernel="tc", key_splits=0, **heads, **kw))  # noqa: E731
+    dec = lambda batch, **kw: microbench.decode_attention(ns(batch=batch, split=0, head_group=0, cold=True, **heads, **kw))  # noqa: E731
+    kern = {}
+    for tokens in (2048, 8192):
+        for chunk in (LOZANEX_CHUNK, 0):
+            kern[f"capped_attention_prefill_{tokens}_chunk{chunk}"] = pre(tokens, chunk=chunk, **capped)
+            kern[f"capped_attention_prefill_{tokens}_chunk{chunk}_scores_beyond_the_cap"] = pre(tokens, chunk=chunk, q_scale=40.0, **capped)
+            kern[f"plain_attention_prefill_{tokens}_chunk{chunk}"] = pre(tokens, chunk=chunk)
+    for batch, context, chunk in ((8, 8192, 0), (64, 8192, LOZANEX_CHUNK)):
+        for kernel in ("gqa", "bulk"):
+            kern[f"capped_attention_decode_b{batch}_ctx{context}_chunk{chunk}_{kernel}"] = dec(batch, context=context, kernel=kernel, chunk=chunk, **capped)
+            kern[f"plain_attention_decode_b{batch}_ctx{context}_chunk{chunk}_{kernel}"] = dec(batch, context=context, kernel=kernel, chunk=chunk)
+    for rows in (8, 64, 2048):
+        kern[f"experts_with_shared_gate_{rows}_rows"] = microbench.routed_experts(ns(tokens=rows, shared_gate=True, **moe))
+        kern[f"lozanex_experts_{rows}_rows"] = microbench.routed_experts(ns(tokens=rows, **moe))
+        kern[f"input_ops_{rows}_rows"] = microbench.input_ops(ns(tokens=rows, width=size["width"], heads=32, kv_heads=8))
+    steps = {}
+    for name, cfg in (("kikarax", kikarax_config(size, 4)), ("lozanex_attention", lozanex_attention_config(size, 4)),
+                      ("kikarax_dense", kikarax_config(size, 4, dense=True)), ("llama", llama_config(size, 4, 8))):
+        with tempfile.NamedTemporaryFile("w", suffix=".json") as f:
+            json.dump(cfg, f)
+            f.flush()
+            done = subprocess.run([sys.executable, "-m", "edgerag_b200.ops.microbench", "step-kernels", "--config-json", f.name,
+                                   "--batch", str(args.batch), "--context", "2048", "--tokens", "2048", "--iters", "4", "--rows", "24"],
+                                  cwd=str(ROOT), env=dict(os.environ, EDGERAG_B200_NO_CHAIN="1"), capture_output=True, text=True)
+        if done.returncode != 0:
+            raise RuntimeError(f"step-kernels of {name} failed: {done.stderr[-400:]}")
+        steps[name] = json.loads(done.stdout.strip().splitlines()[-1])
+    return {"metric": "design_compare", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16",
+            "data": "synthetic", "impl": "ours", "higher_is_better": True,
+            "config": {"designs": ["Kikarax", "Lozanex", "Llama decoder"], "prefill_tokens": 2048, "decode_context": 2048,
+                       "decode_batches": sorted({1, args.batch}), "page_tokens": block, "chunk": LOZANEX_CHUNK, "softcap": KIKARAX_CAP,
+                       "routed_experts": LOZANEX_EXPERTS, "peaks": peak_source,
+                       "l2": "decode: weights and cache larger than L2 at w2048; kernels: caches, weights and rows rotated (cold)"},
+            "sizes": out, "kernels": kern, "step_kernels": steps, "clocks": clocks.record()}
+
+
 def _tensors_of(model) -> list:
     import torch
 
@@ -996,7 +1080,7 @@ def main() -> int:
                     help="decode: the headline measurement; mixed / continuous: the serving workloads of the "
                          "256M and 500M decoders through Engine.generate; designs: prefill and decode of one design "
                          "(--design) beside the Llama decoder at equal sizes, and its kernels against their rooflines")
-    ap.add_argument("--design", choices=["dokodra", "vokusun", "lozanex", "pudadra", "sabolorn"], default="dokodra",
+    ap.add_argument("--design", choices=["dokodra", "vokusun", "lozanex", "pudadra", "sabolorn", "kikarax"], default="dokodra",
                     help="with --workload designs: the design that is measured beside the Llama decoder")
     ap.add_argument("--ref-cpu-check", action="store_true",
                     help="with --impl reference: a dry run of the reference arm's loop at toy sizes on the CPU")

@@ -97,7 +97,27 @@ constexpr int kScorePlain = 0, kScorePenalty = 1, kScoreCap = 2;
 constexpr float kTanh0 = 0.99999941f, kTanh1 = -0.33329042f, kTanh2 = 0.13281434f, kTanh3 = -0.051605674f, kTanh4 = 0.016743115f,
                 kTanh5 = -0.0030670603f;
 
-template <int SCORE>
+// Two floats that one instruction multiplies and adds (both rounded as fmaf rounds one).
+struct Two {
+  unsigned long long v;
+  __device__ __forceinline__ Two() {}
+  __device__ __forceinline__ Two(float a, float b) { asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b)); }
+  __device__ __forceinline__ explicit Two(float a) : Two(a, a) {}
+  __device__ __forceinline__ void get(float& a, float& b) const { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+};
+__device__ __forceinline__ Two operator*(Two a, Two b) {
+  Two d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d.v) : "l"(a.v), "l"(b.v));
+  return d;
+}
+__device__ __forceinline__ Two fma2(Two a, Two b, Two c) {
+  Two d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return d;
+}
+
+// GATED: a launch with a gate (a kernel of its own, so that the others keep their registers).
+template <int SCORE, bool GATED>
 __global__ void __launch_bounds__(kThreads, 1)
 attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                          const __nv_bfloat16* __restrict__ q, int q_row_stride,
@@ -439,16 +459,16 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
               for (int i = 0; i < 16; ++i) sc[i] = capped_score(sc[i] * x_in, cap_out) - m_ref;
             } else {
-              const float out = cap_in * cap_out;
+              const Two in2(cap_in), out2(cap_in * cap_out), ref2(-m_ref);
 #pragma unroll
-              for (int i = 0; i < 16; ++i) {
-                const float x = sc[i] * cap_in, y = x * x;
-                float p = fmaf(kTanh5, y, kTanh4);
-                p = fmaf(p, y, kTanh3);
-                p = fmaf(p, y, kTanh2);
-                p = fmaf(p, y, kTanh1);
-                p = fmaf(p, y, kTanh0);
-                sc[i] = fmaf(sc[i] * out, p, -m_ref);
+              for (int i = 0; i < 16; i += 2) {
+                const Two s2(sc[i], sc[i + 1]), x = s2 * in2, y = x * x;
+                Two p = fma2(Two(kTanh5), y, Two(kTanh4));
+                p = fma2(p, y, Two(kTanh3));
+                p = fma2(p, y, Two(kTanh2));
+                p = fma2(p, y, Two(kTanh1));
+                p = fma2(p, y, Two(kTanh0));
+                fma2(s2 * out2, p, ref2).get(sc[i], sc[i + 1]);
               }
             }
           }
@@ -512,24 +532,19 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
         tmem_ld32(t_o, acc);
         tmem_ld_wait();
         if (row < rows_t[t]) {
-          const __nv_bfloat16* g_row = gate ? gate + (size_t)(q0 + t * BM + row) * gate_stride + h * HD + half * 32 : nullptr;
+          const __nv_bfloat16* g_row = GATED ? gate + (size_t)(q0 + t * BM + row) * gate_stride + h * HD + half * 32 : nullptr;
 #pragma unroll
-          for (int d = 0; d < 32; ++d) acc[d] *= inv;
-          if (g_row) {
-#pragma unroll
-            for (int d = 0; d < 32; d += 8) {
+          for (int d = 0; d < 32; d += 8) {
+            if (GATED) {
               float z[8];
               load8(g_row + d, z);
 #pragma unroll
               for (int i = 0; i < 8; ++i) acc[d + i] = sigmoid_mul(acc[d + i], z[i]);
             }
-          }
-#pragma unroll
-          for (int d = 0; d < 32; d += 8) {
             uint32_t w[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-              __nv_bfloat162 b = __floats2bfloat162_rn(acc[d + 2 * i], acc[d + 2 * i + 1]);
+              __nv_bfloat162 b = __floats2bfloat162_rn(acc[d + 2 * i] * inv, acc[d + 2 * i + 1] * inv);
               w[i] = *reinterpret_cast<uint32_t*>(&b);
             }
             *reinterpret_cast<uint4*>(dst + d) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -640,14 +655,15 @@ ERB_EXPORT int erb_attention_prefill_tc(const void* q, int q_row_stride, const v
       (rc = pool_map(&mv, v_pages, pool_rows, (unsigned)page_size, "attention_prefill_tc")))
     return rc;
   const int score = penalty ? kScorePenalty : softcap > 0.f ? kScoreCap : kScorePlain;
-  auto kern = score == kScorePenalty ? attention_prefill_kernel<kScorePenalty>
-              : score == kScoreCap   ? attention_prefill_kernel<kScoreCap>
-                                     : attention_prefill_kernel<kScorePlain>;
-  static bool configured[3] = {false, false, false};
-  if (!configured[score]) {
+  const bool gated = gate && key_splits == 1;      // (with ranges the merge multiplies)
+  auto kern = score == kScorePenalty ? (gated ? attention_prefill_kernel<kScorePenalty, true> : attention_prefill_kernel<kScorePenalty, false>)
+              : score == kScoreCap   ? (gated ? attention_prefill_kernel<kScoreCap, true> : attention_prefill_kernel<kScoreCap, false>)
+                                     : (gated ? attention_prefill_kernel<kScorePlain, true> : attention_prefill_kernel<kScorePlain, false>);
+  static bool configured[3][2] = {};
+  if (!configured[score][gated]) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemBytes);
     if (e != cudaSuccess) return fail(ERB_ERR_CUDA, "attention_prefill_tc: %s", cudaGetErrorString(e));
-    configured[score] = true;
+    configured[score][gated] = true;
   }
   const float scale_log2 = scale * 1.4426950408889634f;
   launch_chained(kern, dim3(nq, n_blocks, key_splits), dim3(kThreads), kSmemBytes, (cudaStream_t)stream, mk, mv,

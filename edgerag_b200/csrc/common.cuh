@@ -149,7 +149,11 @@ __device__ __forceinline__ float glu_gate(float g, float u, int act, float limit
     u = fminf(fmaxf(u, -limit), limit);
   }
   if (act == ERB_GLU_GELU_TANH) return gelu_tanh_mul(g, u + shift);
+#if ERB_ELEM == 1
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + shift);
+#else
   return g / (1.f + expf(-alpha * g)) * (u + shift);
+#endif
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

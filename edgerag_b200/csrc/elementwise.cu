@@ -1702,6 +1702,120 @@ qkv_whole_norm_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_b
   }
 }
 
+// The same in 16-byte groups: a thread owns up to R groups of the row (in registers from the first read to the store), the two sums
+// of squares go through one pair of barriers, and the angles are made beside them.  A turned group's partner, half a rotation
+// away in its head, is read together with the group itself: q is written in place, so nothing of the row is read after the
+// barriers.  Norm weights are constants, positions and slots the step's metadata: they are read before the wait for the product.
+template <typename T, int R>
+__global__ void __launch_bounds__(512)
+qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_bias, const float* __restrict__ k_bias,
+                          const float* __restrict__ v_bias, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
+                          float q_count, float k_count, float eps, const int* __restrict__ positions,
+                          const float* __restrict__ inv_freq, int rot_dim, const int* __restrict__ slots, T* __restrict__ k_pages,
+                          T* __restrict__ v_pages, int nq, int nkv, int D, int page_size, int has_kv, T* __restrict__ first,
+                          const float* __restrict__ blend, int blend_write, int v_dim) {
+  constexpr int N = Wide<T>::N;
+  extern __shared__ float trig_s[];          // cos[half], sin[half]
+  __shared__ float red[2][16];
+  const int t = blockIdx.x, tid = threadIdx.x, half = rot_dim / 2;
+  const int per_head = D / N, q_groups = nq * per_head, kv_groups = has_kv ? nkv * per_head : 0, total = q_groups + 2 * kv_groups;
+  const int slot = (has_kv && slots && k_pages) ? slots[t] : -1;
+  if (half) {
+    const float pos = (float)positions[t];
+    for (int j = tid; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], trig_s + half + j, trig_s + j);
+  }
+  float w[R][N];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int g = tid + r * blockDim.x;
+    const float* nw = g < q_groups ? q_norm : g < q_groups + kv_groups ? k_norm : nullptr;
+    const int at = (g < q_groups ? g : g - q_groups) * N;
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      if (nw) load4(nw + at + i, w[r] + i);
+      else w[r][i] = w[r][i + 1] = w[r][i + 2] = w[r][i + 3] = 1.f;
+    }
+  }
+  chain_wait();
+  T* row = qkv + (size_t)t * ld;
+  float x[R][N], y[R][N], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int g = tid + r * blockDim.x;
+    if (g >= total) continue;
+    const bool is_q = g < q_groups, is_v = g >= q_groups + kv_groups;
+    const float* bias = is_q ? q_bias : is_v ? v_bias : k_bias;
+    const int at = (is_q ? g : is_v ? g - q_groups - kv_groups : g - q_groups) * N;      // within q, k or v
+    Wide<T>::load(row + g * N, x[r]);
+    const int e = at % D;
+    const bool turned = !is_v && e < rot_dim;
+    const int partner = e < half ? half : -half;
+    if (turned) Wide<T>::load(row + g * N + partner, y[r]);
+    if (bias) {
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        x[r][i] += bias[at + i];
+        if (turned) y[r][i] += bias[at + partner + i];
+      }
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) s = fmaf(x[r][i], x[r][i], s);
+    if (is_q) sq += s;
+    else if (!is_v) sk += s;
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  const int warp = tid >> 5, lane = tid & 31, n_warps = blockDim.x >> 5;
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  float rq = 0.f, rk = 0.f;
+  for (int i = 0; i < n_warps; ++i) { rq += red[0][i]; rk += red[1][i]; }
+  rq = q_norm ? rsqrtf(rq / q_count + eps) : 1.f;
+  rk = has_kv && k_norm ? rsqrtf(rk / k_count + eps) : 1.f;
+  const int page = slot >= 0 ? slot / page_size : 0, offset = slot >= 0 ? slot % page_size : 0;
+  const float l = first && !blend_write ? *blend : 0.f;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int g = tid + r * blockDim.x;
+    if (g >= total) continue;
+    const bool is_q = g < q_groups, is_v = g >= q_groups + kv_groups;
+    const int at = (is_q ? g : is_v ? g - q_groups - kv_groups : g - q_groups) * N, head = at / D, e = at % D;
+    if (is_v) {
+      if (first && e < v_dim) {
+        T* kept = first + (size_t)t * nkv * v_dim + head * v_dim + e;
+        if (blend_write) {
+          Wide<T>::store(kept, x[r]);
+        } else {
+          float f[N];
+          Wide<T>::load(kept, f);
+#pragma unroll
+          for (int i = 0; i < N; ++i) x[r][i] = fmaf(l, f[i], (1.f - l) * x[r][i]);
+        }
+      }
+      if (slot >= 0 && v_pages) Wide<T>::store(v_pages + (((size_t)page * nkv + head) * page_size + offset) * D + e, x[r]);
+      continue;
+    }
+    if (!is_q && slot < 0) continue;
+    const float rs = is_q ? rq : rk;
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[r][i] *= rs * w[r][i];
+    if (e < rot_dim) {
+      const float* nw = is_q ? q_norm : k_norm;
+      const bool low = e < half;
+      const int partner = low ? half : -half, j = low ? e : e - half;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const float other = y[r][i] * (rs * (nw ? nw[at + partner + i] : 1.f));
+        float lo, hi;
+        rotate_pair(low ? x[r][i] : other, low ? other : x[r][i], trig_s[j + i], trig_s[half + j + i], lo, hi);
+        x[r][i] = low ? lo : hi;
+      }
+    }
+    Wide<T>::store(is_q ? row + at : k_pages + (((size_t)page * nkv + head) * page_size + offset) * D + e, x[r]);
+  }
+}
+
 ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const float* k_bias, const float* v_bias,
                                   const float* q_norm, const float* k_norm, int q_count, int k_count, float eps,
                                   const int* positions, const float* inv_freq, int rot_dim, const int* slots, void* k_pages,
@@ -1714,6 +1828,18 @@ ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const 
       q_count <= 0 || k_count <= 0 || page_size <= 0)
     return fail(ERB_ERR_ARG, "qkv_whole_norm: bad sizes (rot_dim %d of head_dim %d)", rot_dim, head_dim);
   if (ld < (nq + (has_kv ? 2 * nkv : 0)) * head_dim) return fail(ERB_ERR_ARG, "qkv_whole_norm: rows too narrow");
+  constexpr int N = Vec16<elem_t>::N;
+  const uintptr_t bits = (uintptr_t)qkv | (uintptr_t)q_norm | (uintptr_t)k_norm | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)first;
+  const int groups = (nq + (has_kv ? 2 * nkv : 0)) * head_dim / N, half = rot_dim / 2;
+  if (head_dim % N == 0 && ld % N == 0 && half % N == 0 && (!first || v_dim % N == 0) && (bits & 15) == 0 && groups <= 4 * 512) {
+    const int r = (groups + 511) / 512, threads = ((groups + r - 1) / r + 31) / 32 * 32;
+    auto vec = r == 1 ? qkv_whole_norm_vec_kernel<elem_t, 1> : r == 2 ? qkv_whole_norm_vec_kernel<elem_t, 2>
+             : r == 3 ? qkv_whole_norm_vec_kernel<elem_t, 3> : qkv_whole_norm_vec_kernel<elem_t, 4>;
+    launch_chained(vec, dim3(n_tokens), dim3(threads), rot_dim * sizeof(float), (cudaStream_t)stream, (elem_t*)qkv, ld, q_bias, k_bias,
+                   v_bias, q_norm, k_norm, (float)q_count, (float)k_count, eps, positions, inv_freq, rot_dim, slots, (elem_t*)k_pages,
+                   (elem_t*)v_pages, nq, nkv, head_dim, page_size, has_kv, (elem_t*)first, blend, blend_write, v_dim);
+    return check_launch("qkv_whole_norm");
+  }
   const size_t smem = sizeof(float) * ((size_t)(nq + (has_kv ? nkv : 0)) * head_dim + 32);
   if (smem > 200 * 1024) return fail(ERB_ERR_UNSUPPORTED, "qkv_whole_norm: %d heads of %d", nq + nkv, head_dim);
   auto kern = qkv_whole_norm_kernel<elem_t>;

@@ -96,7 +96,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
   __shared__ __align__(8) uint64_t bars[2 * kStages + 1];      // full, empty, accumulator done
   __shared__ int s_abort;
   __shared__ uint32_t tmem_slot;
-  __shared__ int pair_s[MT];
+  __shared__ int dst_row_s[PAIRS ? MT : 1];                     // where a row of the tile goes, and what multiplies it
+  __shared__ float scale_s[PAIRS ? MT : 1];
   chain_wait();                                                 // the lists and the rows come from the kernels before
   const int tile = blockIdx.x;
   if (tile >= tiles[n_experts]) return;                         // (before anything is set up: nothing to give back)
@@ -138,9 +139,12 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
     mbar_init_fence();
     for (int i = 0; i < ahead; ++i) ask(i);
   }
-  if (PAIRS && tid < MT) pair_s[tid] = tid < n_rows ? order[row0 + tid] : -1;
-  if (PAIRS && MT > kThreads) {
-    for (int r = kThreads + tid; r < MT; r += kThreads) pair_s[r] = r < n_rows ? order[row0 + r] : -1;
+  if (PAIRS) {
+    for (int r = tid; r < MT && r < n_rows; r += kThreads) {
+      const int pair = order[row0 + r];
+      dst_row_s[r] = (pair % top) * n_tokens + pair / top;
+      scale_s[r] = out_score ? out_score[pair] : 1.f;
+    }
   }
   if (warp == 1) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(P::kTmemCols) : "memory");
@@ -215,9 +219,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
           if (n_a < n_out) act[(size_t)(row0 + m) * n_out + n_a] = __float2bfloat16_rn(za * za);
           if (n_b < n_out) act[(size_t)(row0 + m) * n_out + n_b] = __float2bfloat16_rn(zb * zb);
         } else {
-          const int pair = pair_s[m];
-          const float sc = out_score ? out_score[pair] : 1.f;
-          float* dst = parts + ((size_t)(pair % top) * n_tokens + pair / top) * n_out;
+          const float sc = scale_s[m];
+          float* dst = parts + (size_t)dst_row_s[m] * n_out;
           if (n_a < n_out) dst[n_a] = v0[i] * sc;
           if (n_b < n_out) dst[n_b] = v1[i] * sc;
         }

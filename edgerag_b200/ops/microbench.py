@@ -80,6 +80,19 @@ def _penalty_of(a) -> torch.Tensor | None:
     return torch.stack([torch.linspace(0.2, 2.0, a.heads), torch.linspace(0.05, 0.5, a.heads)]).cuda()
 
 
+def _score_of(a, rows: int, dtype) -> dict:
+    """``--penalty``, ``--softcap`` and ``--gate`` as arguments of the attention kernels (the gate's columns lie in wider rows, as the
+    engine keeps them beside q, k and v)."""
+    width = a.heads * a.head_dim
+    gate = torch.randn((rows, 2 * width), device="cuda").to(dtype)[:, width:] if getattr(a, "gate", False) else None
+    return {"penalty": _penalty_of(a), "softcap": float(getattr(a, "softcap", 0.0) or 0.0), "gate": gate}
+
+
+def _score_record(a) -> dict:
+    return {"penalty": bool(getattr(a, "penalty", False)), "softcap": float(getattr(a, "softcap", 0.0) or 0.0),
+            "gate": bool(getattr(a, "gate", False)), "q_scale": float(getattr(a, "q_scale", 1.0) or 1.0)}
+
+
 def _paged(batch: int, context: int, nkv: int, d: int, page: int, dtype, shuffle: bool = True):
     """Key and value pools of ``batch`` sequences of ``context`` tokens with their block tables."""
     pages_per = -(-context // page)
@@ -108,8 +121,8 @@ def decode_attention(a) -> dict:
         state["i"] = (state["i"] + 1) % reps
         return caches[state["i"]]
 
-    q = torch.randn((a.batch, a.heads * a.head_dim), device="cuda").to(dtype)
-    pen = _penalty_of(a)
+    q = (torch.randn((a.batch, a.heads * a.head_dim), device="cuda") * float(getattr(a, "q_scale", 1.0) or 1.0)).to(dtype)
+    score = _score_of(a, a.batch, dtype)
     out = torch.empty_like(q)
     pos = torch.full((a.batch,), a.context - 1, dtype=torch.int32, device="cuda")
     tok = torch.arange(a.batch, dtype=torch.int32, device="cuda")
@@ -130,19 +143,19 @@ def decode_attention(a) -> dict:
     scale = a.head_dim ** -0.5
     if a.kernel == "gqa":
         fn = lambda: kernels.attention_decode_gqa(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
-                                                  status, split_keys=a.split, window=window, keep_first=keep, chunk=chunk, penalty=pen)
+                                                  status, split_keys=a.split, window=window, keep_first=keep, chunk=chunk, **score)
     elif a.kernel == "bulk":
         fn = lambda: kernels.attention_decode_bulk(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
                                                    status, split_keys=a.split, head_group=a.head_group, window=window, keep_first=keep,
-                                                   chunk=chunk, penalty=pen)
+                                                   chunk=chunk, **score)
     else:
         fn = lambda: kernels.attention_decode(q, *cache(), tok, pos, out, a.heads, scale, acc, ml, splits,  # noqa: E731
-                                              split_keys=a.split, window=window, keep_first=keep, chunk=chunk, penalty=pen)
+                                              split_keys=a.split, window=window, keep_first=keep, chunk=chunk, **score)
     us = _time(fn, max(a.iters, 2 * reps), a.warmup)
     return {"case": "decode-attention", "kernel": a.kernel, "split": a.split, "head_group": a.head_group, "us": round(us, 2),
             "bytes": nbytes, "gbs": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / HBM_GBS, 4),
             "status": int(status), "from_dram": bool(a.cold) or nbytes > 126e6, "window": window, "keep_first": keep, "chunk": chunk,
-            "penalty": pen is not None}
+            **_score_record(a)}
 
 
 def prefill_attention(a) -> dict:
@@ -150,12 +163,12 @@ def prefill_attention(a) -> dict:
     total = a.past + a.tokens
     kp, vp, tables = _paged(1, total, a.kv_heads, a.head_dim, a.page, dtype, not a.sequential_pages)
     width = (a.heads + 2 * a.kv_heads) * a.head_dim
-    qkv = torch.randn((a.tokens, width), device="cuda").to(dtype)
+    qkv = (torch.randn((a.tokens, width), device="cuda") * float(getattr(a, "q_scale", 1.0) or 1.0)).to(dtype)
     out = torch.empty((a.tokens, a.heads * a.head_dim), device="cuda", dtype=dtype)
     pos = torch.arange(a.past, total, dtype=torch.int32, device="cuda")
     starts = torch.tensor([0, a.tokens], dtype=torch.int32, device="cuda")
     seq_of = torch.zeros(a.tokens, dtype=torch.int32, device="cuda")
-    pen = _penalty_of(a)
+    score = _score_of(a, a.tokens, dtype)
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
     scale = a.head_dim ** -0.5
     window, keep, chunk = getattr(a, "window", 0), getattr(a, "keep_first", 0), getattr(a, "chunk", 0)
@@ -167,10 +180,10 @@ def prefill_attention(a) -> dict:
         part_o, part_ml = torch.empty(need_o, device="cuda"), torch.empty(need_ml, device="cuda")
         fn = lambda: kernels.attention_prefill_tc(qkv, kp, vp, tables, starts, pos, out, blocks, a.heads, scale, status,  # noqa: E731
                                                   key_splits=ranges, part_o=part_o, part_ml=part_ml, window=window, keep_first=keep,
-                                                  chunk=chunk, penalty=pen)
+                                                  chunk=chunk, **score)
     else:
         fn = lambda: kernels.attention_rows(qkv, kp, vp, tables, seq_of, pos, out, a.heads, scale, window=window,  # noqa: E731
-                                            keep_first=keep, chunk=chunk, penalty=pen)
+                                            keep_first=keep, chunk=chunk, **score)
     us = _time(fn, a.iters, a.warmup)
     if window > 0:      # (query, key) pairs that are seen: the window's keys and the kept ones before it
         p = torch.arange(a.past, total, dtype=torch.float64)
@@ -184,7 +197,7 @@ def prefill_attention(a) -> dict:
     flops = 4.0 * a.heads * a.head_dim * pairs
     return {"case": "prefill-attention", "kernel": a.kernel, "us": round(us, 2), "tflops": round(flops / us / 1e6, 1),
             "frac_bf16": round(flops / us / 1e6 / BF16_TFLOPS, 4), "status": int(status), "window": window, "keep_first": keep, "chunk": chunk,
-            "penalty": pen is not None}
+            **_score_record(a)}
 
 
 def linear(a) -> dict:
@@ -553,8 +566,12 @@ def routed_experts(a) -> dict:
     if getattr(a, "corrected", False):
         how = dict(groups=tuple(a.groups) if getattr(a, "groups", None) else None, correction=torch.randn(E, device="cuda") * 0.3,
                    group_score="top2_sum", normalise=True)
+    shared_gate = bool(getattr(a, "shared_gate", False))
+    if shared_gate:         # softmax scores times a constant on the output; one more row of the router, for the shared expert's gate
+        how = dict(scores="softmax", weight=2.5, side_gate=torch.empty(n, device="cuda"))
+        router = torch.randn((E + 1, h), device="cuda") * 0.05
     if kernels.moe_route_few(n, E, top, dtype):
-        how_few = {"logits": torch.empty((n, E), device="cuda")}
+        how_few = {"logits": torch.empty((n, router.shape[0]), device="cuda")}
     else:
         how_few = {}
     in_score, out_score = (None, score) if how else (score, None)
@@ -679,6 +696,58 @@ def stream_ops(a) -> dict:
     return res
 
 
+def input_ops(a) -> dict:
+    """The kernels between a product and the attention, and at the model's input, over ``tokens`` rows of a layer with a norm over the
+    whole query and key projection: the norm with the cache write, alone, with the gate's columns behind the values, and with
+    values blended with the first layer's; the embedding as a table lookup and as the sum of token, pair and position rows.
+    All are bound by the bytes they move."""
+    dtype = torch.bfloat16 if a.dtype == "bfloat16" else torch.float32
+    item = 2 if dtype == torch.bfloat16 else 4
+    n, h, H, G, D, page = a.tokens, a.width, a.heads, a.kv_heads, 64, 16
+    C, W = (H + 2 * G) * D, (2 * H + 2 * G) * D
+    reps = max(1, int(300e6 // (n * W * item)) + 1)
+    rows = [torch.randn((n, W), device="cuda").to(dtype) for _ in range(reps)]
+    state = {"i": 0}
+
+    def turn():
+        state["i"] = (state["i"] + 1) % reps
+        return rows[state["i"]]
+
+    def line(us, nbytes):
+        return {"us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / HBM_GBS, 4)}
+
+    pos = torch.arange(n, dtype=torch.int32, device="cuda")
+    slots = torch.randperm(n).to(torch.int32).cuda()
+    kp, vp = (torch.empty((-(-n // page), G, page, D), device="cuda", dtype=dtype) for _ in range(2))
+    qn, kn, blend = torch.randn(H * D, device="cuda"), torch.randn(G * D, device="cuda"), torch.full((1,), 0.4, device="cuda")
+    first = torch.randn((n, G * D), device="cuda").to(dtype)
+    iters = max(a.iters, 2 * reps)
+
+    def norm(width, **more):
+        kernels.qkv_whole_norm(turn()[:, :width], pos, H, G, D, q_count=H * D, k_count=G * D, eps=1e-5, q_norm=qn, k_norm=kn, slots=slots,
+                               k_pages=kp, v_pages=vp, page_size=page, **more)
+
+    moved = n * item * 2 * (H + 2 * G) * D          # every row read and written once
+    res = {"case": "input-ops", "tokens": n, "width": h, "heads": H, "kv_heads": G,
+           "whole_norm": line(_time(lambda: norm(C), iters, a.warmup), moved),
+           "whole_norm_wide_rows": line(_time(lambda: norm(W), iters, a.warmup), moved),
+           "whole_norm_blended_values": line(_time(lambda: norm(W, first_values=first, blend=blend), iters, a.warmup), moved + n * G * D * item)}
+    vocab, buckets = 32000, 40009
+    table, pairs, places = (torch.randn((r, h), device="cuda").to(dtype) for r in (vocab, buckets + 1, 8192))
+    ids = torch.randint(0, vocab, (n,), device="cuda").to(torch.int32)
+    hidden, status = torch.empty((n, h), device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+    single = n <= 64
+    starts = torch.arange(n + 1, dtype=torch.int32, device="cuda") if single else torch.tensor([0, n], dtype=torch.int32, device="cuda")
+    seq_of = torch.arange(n, dtype=torch.int32, device="cuda") if single else torch.zeros(n, dtype=torch.int32, device="cuda")
+    seqs = n if single else 1
+    st, last = torch.arange(seqs, dtype=torch.int32, device="cuda"), torch.zeros((seqs, 1), dtype=torch.int32, device="cuda")
+    res["embed_rows"] = line(_time(lambda: kernels.embed_rows(hidden, table, ids, status), a.iters, a.warmup), n * h * (item + 4))
+    both = lambda: kernels.embed_sum(hidden, table, ids, status, pos, scale=8.0, pairs=pairs, pos_table=places,              # noqa: E731
+                                     pair_hash=(buckets, 31, 17), last_id=last, seq_of_token=seq_of, seq_starts=starts, state_slots=st)
+    res["embed_sum"] = line(_time(both, a.iters, a.warmup), n * h * (3 * item + 4))
+    return res
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="edgerag_b200.ops.microbench", description=__doc__.split("\n\n")[0])
     sub = ap.add_subparsers(dest="case", required=True)
@@ -697,6 +766,9 @@ def main(argv=None) -> int:
     att.add_argument("--chunk", type=int, default=0, help="instead of a window: a query sees its own run of this many positions")
     att.add_argument("--sequential-pages", action="store_true", help="pages in order instead of shuffled")
     att.add_argument("--penalty", action="store_true", help="a penalty that grows with the logarithm of the distance")
+    att.add_argument("--softcap", type=float, default=0.0, help="a cap c of the scores: s becomes c * tanh(s / c)")
+    att.add_argument("--gate", action="store_true", help="outputs multiplied by the sigmoid of a gate's entries")
+    att.add_argument("--q-scale", type=float, default=1.0, help="factor of the random queries (the scores' standard deviation)")
     d = sub.add_parser("decode-attention", parents=[common, att])
     d.add_argument("--batch", type=int, default=8)
     d.add_argument("--context", type=int, default=8192)
@@ -783,6 +855,7 @@ def main(argv=None) -> int:
     re.add_argument("--top", type=int, default=4)
     re.add_argument("--general", action="store_true", help="the products on CUDA cores (what float32 runs) instead of tensor cores")
     re.add_argument("--ungated", action="store_true", help="experts without a gate branch, softmax scores, the weight on the output")
+    re.add_argument("--shared-gate", action="store_true", help="softmax scores times a constant, and the shared expert's gate as a router row")
     re.add_argument("--corrected", action="store_true", help="a correction per expert in the choice, normalised weights on the output")
     re.add_argument("--groups", type=int, nargs=2, default=None, help="with --ungated or --corrected: (count, keep) of the router's groups")
     so = sub.add_parser("stream-ops", parents=[common])
@@ -791,13 +864,18 @@ def main(argv=None) -> int:
     so.add_argument("--layers", type=int, default=8, help="results that the average over depth takes besides the newest")
     so.add_argument("--heads", type=int, default=32)
     so.add_argument("--kv-heads", type=int, default=8)
+    io = sub.add_parser("input-ops", parents=[common])
+    io.add_argument("--tokens", type=int, default=2048)
+    io.add_argument("--width", type=int, default=2048)
+    io.add_argument("--heads", type=int, default=32)
+    io.add_argument("--kv-heads", type=int, default=8)
     a = ap.parse_args(argv)
     if not torch.cuda.is_available():
         print("microbench needs a CUDA device", file=sys.stderr)
         return 1
     fn = {"decode-attention": decode_attention, "prefill-attention": prefill_attention, "linear": linear,
           "step-kernels": step_kernels, "step-timeline": step_timeline, "latent-attention": latent_attention,
-          "ssm-scan": ssm_scan, "delta-scan": delta_scan, "routed-experts": routed_experts, "diff-attention": diff_attention, "stream-ops": stream_ops}[a.case]
+          "ssm-scan": ssm_scan, "delta-scan": delta_scan, "routed-experts": routed_experts, "diff-attention": diff_attention, "stream-ops": stream_ops, "input-ops": input_ops}[a.case]
     load_peaks(a.peaks)
     result = fn(a)
     result["peaks"] = PEAKS_FROM
