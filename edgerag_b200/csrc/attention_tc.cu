@@ -135,8 +135,9 @@ __device__ __forceinline__ void merge_splits_if_last(int* counter, const float* 
   }
 }
 
-template <int D, int R>   // head size; query heads per kv head (1..kMaxGroup)
-__global__ void __launch_bounds__(kDecThreads)
+// SHAPED: a launch with a penalty, a cap or a gate (kernels of their own, so that the plain ones carry none of it).
+template <int D, int R, bool SHAPED>   // head size; query heads per kv head (1..kMaxGroup)
+__global__ void __launch_bounds__(kDecThreads, R <= 4 ? 2 : 1)   // (two blocks an SM hide each other's waits: worth a few spills)
 attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride,
                              const __nv_bfloat16* __restrict__ k_pages, const __nv_bfloat16* __restrict__ v_pages,
                              const int* __restrict__ block_tables, int max_pages,
@@ -267,11 +268,12 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
 #pragma unroll
     for (int i = 0; i < 8; ++i) qr[g][i] = tmp[i] * scale_log2;
   }
+  const bool shaped = SHAPED && (penalty || softcap > 0.f);          // something is done to the scores
   const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
-  const __nv_bfloat16* gate_row = gate ? gate + (size_t)t * gate_stride : nullptr;
+  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
   Penalty2 pen[R];
 #pragma unroll
-  for (int g = 0; g < R; ++g) pen[g].load(penalty, (serves ? kvh : kvh0) * R + g, nq);
+  for (int g = 0; g < R; ++g) pen[g].load(SHAPED ? penalty : nullptr, (serves ? kvh : kvh0) * R + g, nq);
   float m_run[R], l_run[R], acc[R][8];
 #pragma unroll
   for (int g = 0; g < R; ++g) {
@@ -333,8 +335,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
         float m_new = m_run[g];
 #pragma unroll
         for (int u = 0; u < kKeysPerGroup; ++u) {
-          if (penalty) sc[g][u] -= pen[g].at(pos - (key0 + u));
-          if (softcap > 0.f) sc[g][u] = capped_score(sc[g][u] * cap_in, cap_out);
+          if (shaped) sc[g][u] = cap_in > 0.f ? capped_score(sc[g][u] * cap_in, cap_out) : sc[g][u] - pen[g].at(pos - (key0 + u));
           if (hidden[u]) sc[g][u] = -INFINITY;     // keys past the end of the split or before the window
           m_new = fmaxf(m_new, sc[g][u]);
         }
@@ -500,8 +501,10 @@ int launch_decode_bulk(const void* q, int q_row_stride, const void* k_pages, con
                       (size_t)(split_keys / page_size + 2 + (window > 0 ? keep_first / page_size + 1 : 0)) * sizeof(int);
   if (smem > 200 * 1024)
     return fail(ERB_ERR_UNSUPPORTED, "attention_decode_bulk: split of %d keys and %d kept keys in pages of %d", split_keys, keep_first, page_size);
-  auto kern = attention_decode_bulk_kernel<D, R>;
-  static size_t configured = 0;
+  const bool shaped = penalty || softcap > 0.f || gate;
+  auto kern = shaped ? attention_decode_bulk_kernel<D, R, true> : attention_decode_bulk_kernel<D, R, false>;
+  static size_t configured_for[2] = {0, 0};
+  size_t& configured = configured_for[shaped];
   if (smem > configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return fail(ERB_ERR_CUDA, "attention_decode_bulk: %s", cudaGetErrorString(e));
@@ -581,7 +584,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&v);
 }
 
-__global__ void __launch_bounds__(kGqaThreads)
+template <bool SHAPED>
+__global__ void __launch_bounds__(kGqaThreads, 2)
 attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const __grid_constant__ CUtensorMap map_k_last, const __grid_constant__ CUtensorMap map_v_last,
                             const __nv_bfloat16* __restrict__ q, int q_row_stride,
@@ -710,10 +714,11 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       qa[ks][1] = real ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * j + 8) : 0u;
     }
   }
+  const bool shaped = SHAPED && (penalty || softcap > 0.f);          // something is done to the scores
   const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
-  const __nv_bfloat16* gate_row = gate ? gate + (size_t)t * gate_stride : nullptr;
+  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
   Penalty2 pen;
-  if (serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
+  if (SHAPED && serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
   float o[8][4];
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb)
@@ -770,8 +775,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           // (keys past the split's end, and keys of the window's first page that lie before the window and are not kept)
           const bool seen = key < n_here && !(key_abs0 + key < k_lo && key_abs0 + key >= keep_first);
           sc[b][i] *= scale_log2;
-          if (penalty) sc[b][i] -= pen.at(pos - (key_abs0 + key));
-          if (softcap > 0.f) sc[b][i] = capped_score(sc[b][i] * cap_in, cap_out);
+          if (shaped) sc[b][i] = cap_in > 0.f ? capped_score(sc[b][i] * cap_in, cap_out) : sc[b][i] - pen.at(pos - (key_abs0 + key));
           if (!seen) sc[b][i] = -INFINITY;
           m_new = fmaxf(m_new, sc[b][i]);
         }
@@ -892,15 +896,18 @@ ERB_EXPORT int erb_attention_decode_gqa(const void* q, int q_row_stride, const v
   const size_t smem = 1024 + 2 * kGqaStages * kGqaStageBytes + 64 + (size_t)kDecWarps * r * (64 + 2) * sizeof(float) + 128 +
                       (size_t)(split_keys / page_size + 2 + (window > 0 ? keep_first / page_size + 1 : 0)) * sizeof(int);
   if (smem > 200 * 1024) return fail(ERB_ERR_UNSUPPORTED, "attention_decode_gqa: split of %d keys in pages of %d", split_keys, page_size);
-  static size_t configured = 0;
+  const bool shaped = penalty || softcap > 0.f || gate;
+  auto kern = shaped ? attention_decode_gqa_kernel<true> : attention_decode_gqa_kernel<false>;
+  static size_t configured_for[2] = {0, 0};
+  size_t& configured = configured_for[shaped];
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_gqa_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return fail(ERB_ERR_CUDA, "attention_decode_gqa: %s", cudaGetErrorString(e));
     configured = smem;
   }
   cudaStream_t s = (cudaStream_t)stream;
   const float scale_log2 = scale * 1.4426950408889634f;
-  launch_chained(attention_decode_gqa_kernel, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kGqaThreads), smem, s,
+  launch_chained(kern, dim3(dim3(max_splits, (nkv + hg - 1) / hg, n_seqs)), dim3(kGqaThreads), smem, s,
                  mk, mv, mkl, mvl, (const __nv_bfloat16*)q, q_row_stride, block_tables, max_pages, token_of_seq, positions,
                  part_acc, part_ml, max_splits, nq, nkv, page_size, split_keys, scale_log2, hg, (__nv_bfloat16*)out, out_row_stride,
                  status, counters, window, keep_first, penalty, softcap, (const __nv_bfloat16*)gate, gate_stride);

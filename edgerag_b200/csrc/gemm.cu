@@ -346,6 +346,7 @@ struct RopeArgs {
   // the defaults are the SwiGLU gate
   float glu_limit = 0.f, glu_alpha = 1.f, glu_shift = 0.f;
   int glu_act = 0;             // ERB_GLU_SIGMOID or ERB_GLU_GELU_TANH (see glu_gate)
+  int bounded = 0;             // take that gate (0: silu(g) * u)
   const float* row_scale = nullptr;   // a float per row of `a` that multiplies the gated output (or null)
 };
 
@@ -462,12 +463,12 @@ linear_skinny_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* _
       if constexpr (GLU) {
         const int n = n0 + rr;
         float act;
-        if (ra.glu_limit > 0.f || ra.glu_alpha != 1.f || ra.glu_shift != 0.f || ra.glu_act != 0 || ra.row_scale) {     // the bounded gate, as its own kernel writes it
+        if (ra.bounded) {      // the bounded gate, as its own kernel writes it
           act = glu_gate(v0, v1, ra.glu_act, ra.glu_limit, ra.glu_alpha, ra.glu_shift);
+          if (ra.row_scale) act *= ra.row_scale[m];
         } else {
           act = silu_mul(v0, v1);
         }
-        if (ra.row_scale) act *= ra.row_scale[m];
         if (n < N) reinterpret_cast<__nv_bfloat16*>(out)[(size_t)m * ldo + n] = __float2bfloat16_rn(act);
       } else {
         const int D = ra.head_dim, half = D / 2;
@@ -697,6 +698,7 @@ ERB_EXPORT int erb_linear_skinny_glu_bounded(const void* a, const void* w, void*
   if (rc) return rc;
   RopeArgs ra{};
   ra.glu_limit = limit; ra.glu_alpha = alpha; ra.glu_shift = shift; ra.glu_act = act; ra.row_scale = row_scale;
+  ra.bounded = limit > 0.f || alpha != 1.f || shift != 0.f || act != 0 || row_scale;
   return launch_skinny_mode<2>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, out, M, N, K, lda, ldw, ldo,
                                (cudaStream_t)stream, ra);
 }
