@@ -270,7 +270,6 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
   }
   const bool shaped = SHAPED && (penalty || softcap > 0.f);          // something is done to the scores
   const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
-  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
   Penalty2 pen[R];
 #pragma unroll
   for (int g = 0; g < R; ++g) pen[g].load(SHAPED ? penalty : nullptr, (serves ? kvh : kvh0) * R + g, nq);
@@ -393,6 +392,7 @@ attention_decode_bulk_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stri
       if (chunk == 0) { w[D] = m; w[D + 1] = l; }
     }
   }
+  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
   __syncthreads();
   if (!ok) {
     if (tid == 0) atomicCAS(status, 0, 2000000 + (int)blockIdx.x);
@@ -714,11 +714,10 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       qa[ks][1] = real ? *reinterpret_cast<const uint32_t*>(qp + ks * 16 + 2 * j + 8) : 0u;
     }
   }
-  const bool shaped = SHAPED && (penalty || softcap > 0.f);          // something is done to the scores
-  const float cap_in = softcap > 0.f ? 2.f / softcap : 0.f, cap_out = softcap * 1.4426950408889634f;
-  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
-  Penalty2 pen;
-  if (SHAPED && serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
+  const bool shaped = SHAPED && (penalty || softcap > 0.f), capped = softcap > 0.f;      // something is done to the scores
+  Penalty2 pen;                               // (a cap keeps its two numbers in the penalty's place)
+  if (SHAPED && capped) { pen.r1 = softcap * 1.4426950408889634f; pen.r2 = 2.f / softcap; }
+  else if (SHAPED && serves && g < R) pen.load(penalty, (kvh0 + hh) * R + g, nq);
   float o[8][4];
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb)
@@ -775,7 +774,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           // (keys past the split's end, and keys of the window's first page that lie before the window and are not kept)
           const bool seen = key < n_here && !(key_abs0 + key < k_lo && key_abs0 + key >= keep_first);
           sc[b][i] *= scale_log2;
-          if (shaped) sc[b][i] = cap_in > 0.f ? capped_score(sc[b][i] * cap_in, cap_out) : sc[b][i] - pen.at(pos - (key_abs0 + key));
+          if (shaped) sc[b][i] = capped ? capped_score(sc[b][i] * pen.r2, pen.r1) : sc[b][i] - pen.at(pos - (key_abs0 + key));
           if (!seen) sc[b][i] = -INFINITY;
           m_new = fmaxf(m_new, sc[b][i]);
         }
@@ -817,6 +816,7 @@ attention_decode_gqa_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     for (int nb = 0; nb < 8; ++nb) { w[nb * 8 + 2 * j] = o[nb][0]; w[nb * 8 + 2 * j + 1] = o[nb][1]; }
     if (j == 0) { w[D] = m_run; w[D + 1] = l_run; }
   }
+  const __nv_bfloat16* gate_row = SHAPED && gate ? gate + (size_t)t * gate_stride : nullptr;
   __syncthreads();
   if (*s_abort) {
     if (tid == 0) atomicCAS(status, 0, 2000000 + (int)blockIdx.x);
