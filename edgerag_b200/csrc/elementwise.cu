@@ -1705,16 +1705,20 @@ qkv_whole_norm_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_b
 // The same in 16-byte groups: a thread owns up to R groups of the row (in registers from the first read to the store), the two sums
 // of squares go through one pair of barriers, and the angles are made beside them.  A turned group's partner, half a rotation
 // away in its head, is read together with the group itself: q is written in place, so nothing of the row is read after the
-// barriers.  Norm weights are constants, positions and slots the step's metadata: they are read before the wait for the product.
-template <typename T, int R>
-__global__ void __launch_bounds__(512)
+// barriers.  Norm weights are constants, positions and slots the step's metadata: with FEW tokens the weights too are read before
+// the wait for the product; with many they are read (from the SM's cache) as they are used, which leaves registers for more
+// blocks an SM.
+template <typename T, int R, bool FEW>
+__global__ void __launch_bounds__(512, FEW || R > 1 ? 1 : 3)
 qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__ q_bias, const float* __restrict__ k_bias,
                           const float* __restrict__ v_bias, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
                           float q_count, float k_count, float eps, const int* __restrict__ positions,
                           const float* __restrict__ inv_freq, int rot_dim, const int* __restrict__ slots, T* __restrict__ k_pages,
                           T* __restrict__ v_pages, int nq, int nkv, int D, int page_size, int has_kv, T* __restrict__ first,
-                          const float* __restrict__ blend, int blend_write, int v_dim) {
+                          const float* __restrict__ blend, int blend_write, int v_dim, int d_shift, int page_shift) {
   constexpr int N = Wide<T>::N;
+  // (a shift where the divisor is a power of two: the kernel has little else to do per entry)
+  auto div = [](int a, int d, int shift) { return shift >= 0 ? a >> shift : a / d; };
   extern __shared__ float trig_s[];          // cos[half], sin[half]
   __shared__ float red[2][16];
   const int t = blockIdx.x, tid = threadIdx.x, half = rot_dim / 2;
@@ -1725,8 +1729,7 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
     for (int j = tid; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], trig_s + half + j, trig_s + j);
   }
   float w[R][N];
-#pragma unroll
-  for (int r = 0; r < R; ++r) {
+  auto load_w = [&](int r) {
     const int g = tid + r * blockDim.x;
     const float* nw = g < q_groups ? q_norm : g < q_groups + kv_groups ? k_norm : nullptr;
     const int at = (g < q_groups ? g : g - q_groups) * N;
@@ -1735,6 +1738,10 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
       if (nw) load4(nw + at + i, w[r] + i);
       else w[r][i] = w[r][i + 1] = w[r][i + 2] = w[r][i + 3] = 1.f;
     }
+  };
+  if (FEW) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) load_w(r);
   }
   chain_wait();
   T* row = qkv + (size_t)t * ld;
@@ -1747,7 +1754,7 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
     const float* bias = is_q ? q_bias : is_v ? v_bias : k_bias;
     const int at = (is_q ? g : is_v ? g - q_groups - kv_groups : g - q_groups) * N;      // within q, k or v
     Wide<T>::load(row + g * N, x[r]);
-    const int e = at % D;
+    const int e = at - div(at, D, d_shift) * D;
     const bool turned = !is_v && e < rot_dim;
     const int partner = e < half ? half : -half;
     if (turned) Wide<T>::load(row + g * N + partner, y[r]);
@@ -1770,17 +1777,19 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
   if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
   __syncthreads();
   float rq = 0.f, rk = 0.f;
-  for (int i = 0; i < n_warps; ++i) { rq += red[0][i]; rk += red[1][i]; }
+  if (lane < n_warps) { rq = red[0][lane]; rk = red[1][lane]; }
+  rq = warp_sum(rq);
+  rk = warp_sum(rk);
   rq = q_norm ? rsqrtf(rq / q_count + eps) : 1.f;
   rk = has_kv && k_norm ? rsqrtf(rk / k_count + eps) : 1.f;
-  const int page = slot >= 0 ? slot / page_size : 0, offset = slot >= 0 ? slot % page_size : 0;
+  const int page = slot >= 0 ? div(slot, page_size, page_shift) : 0, offset = slot >= 0 ? slot - page * page_size : 0;
   const float l = first && !blend_write ? *blend : 0.f;
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int g = tid + r * blockDim.x;
     if (g >= total) continue;
     const bool is_q = g < q_groups, is_v = g >= q_groups + kv_groups;
-    const int at = (is_q ? g : is_v ? g - q_groups - kv_groups : g - q_groups) * N, head = at / D, e = at % D;
+    const int at = (is_q ? g : is_v ? g - q_groups - kv_groups : g - q_groups) * N, head = div(at, D, d_shift), e = at - head * D;
     if (is_v) {
       if (first && e < v_dim) {
         T* kept = first + (size_t)t * nkv * v_dim + head * v_dim + e;
@@ -1798,6 +1807,7 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
     }
     if (!is_q && slot < 0) continue;
     const float rs = is_q ? rq : rk;
+    if (!FEW) load_w(r);
 #pragma unroll
     for (int i = 0; i < N; ++i) x[r][i] *= rs * w[r][i];
     if (e < rot_dim) {
@@ -1814,6 +1824,13 @@ qkv_whole_norm_vec_kernel(T* __restrict__ qkv, int ld, const float* __restrict__
     }
     Wide<T>::store(is_q ? row + at : k_pages + (((size_t)page * nkv + head) * page_size + offset) * D + e, x[r]);
   }
+}
+
+// log2 of a power of two, -1 of other numbers.
+static int shift_of(int n) {
+  int s = 0;
+  while ((1 << s) < n) ++s;
+  return (1 << s) == n ? s : -1;
 }
 
 ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const float* k_bias, const float* v_bias,
@@ -1833,11 +1850,13 @@ ERB_EXPORT int erb_qkv_whole_norm(void* qkv, int ld, const float* q_bias, const 
   const int groups = (nq + (has_kv ? 2 * nkv : 0)) * head_dim / N, half = rot_dim / 2;
   if (head_dim % N == 0 && ld % N == 0 && half % N == 0 && (!first || v_dim % N == 0) && (bits & 15) == 0 && groups <= 4 * 512) {
     const int r = (groups + 511) / 512, threads = ((groups + r - 1) / r + 31) / 32 * 32;
-    auto vec = r == 1 ? qkv_whole_norm_vec_kernel<elem_t, 1> : r == 2 ? qkv_whole_norm_vec_kernel<elem_t, 2>
-             : r == 3 ? qkv_whole_norm_vec_kernel<elem_t, 3> : qkv_whole_norm_vec_kernel<elem_t, 4>;
+    auto vec = r == 1 ? (n_tokens <= 64 ? qkv_whole_norm_vec_kernel<elem_t, 1, true> : qkv_whole_norm_vec_kernel<elem_t, 1, false>)
+             : r == 2 ? qkv_whole_norm_vec_kernel<elem_t, 2, true>
+             : r == 3 ? qkv_whole_norm_vec_kernel<elem_t, 3, true> : qkv_whole_norm_vec_kernel<elem_t, 4, true>;
     launch_chained(vec, dim3(n_tokens), dim3(threads), rot_dim * sizeof(float), (cudaStream_t)stream, (elem_t*)qkv, ld, q_bias, k_bias,
                    v_bias, q_norm, k_norm, (float)q_count, (float)k_count, eps, positions, inv_freq, rot_dim, slots, (elem_t*)k_pages,
-                   (elem_t*)v_pages, nq, nkv, head_dim, page_size, has_kv, (elem_t*)first, blend, blend_write, v_dim);
+                   (elem_t*)v_pages, nq, nkv, head_dim, page_size, has_kv, (elem_t*)first, blend, blend_write, v_dim,
+                   shift_of(head_dim), shift_of(page_size));
     return check_launch("qkv_whole_norm");
   }
   const size_t smem = sizeof(float) * ((size_t)(nq + (has_kv ? nkv : 0)) * head_dim + 32);
