@@ -644,8 +644,8 @@ def kikarax_config(size: dict, n_layers: int, dense: bool = False) -> dict:
     mlp = {"kind": "dense", "ff": size["ff"], "limit": 7.0} if dense else {
         "kind": "moe", "expert": {"ff": size["ff"] // 8}, "router": dict(LOZANEX_EXPERTS, scale=2.5), "shared": {"ff": size["ff"] // 2}}
     return {"architecture": "Kikarax", "width": size["width"], "vocab": size["vocab"], "norm": {"eps": 1e-5}, "max_positions": 8192,
-            "embedding": {"scale": size["width"] ** 0.5, "bigram": {"buckets": KIKARAX_BUCKETS, "mul_prev": 31, "mul_cur": 17}},
-            "logit_scale": 0.5, "layers": [{"type": "attention", "mixer": dict(att), "mlp": mlp} for _ in range(n_layers)]}
+            "embedding": {"scale": 8.0, "bigram": {"buckets": KIKARAX_BUCKETS, "mul_prev": 1009, "mul_cur": 263}},
+            "logit_scale": 0.25, "layers": [{"type": "attention", "mixer": dict(att), "mlp": mlp} for _ in range(n_layers)]}
 
 
 def lozanex_attention_config(size: dict, n_layers: int) -> dict:

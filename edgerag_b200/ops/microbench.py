@@ -743,7 +743,7 @@ def input_ops(a) -> dict:
     st, last = torch.arange(seqs, dtype=torch.int32, device="cuda"), torch.zeros((seqs, 1), dtype=torch.int32, device="cuda")
     res["embed_rows"] = line(_time(lambda: kernels.embed_rows(hidden, table, ids, status), a.iters, a.warmup), n * h * (item + 4))
     both = lambda: kernels.embed_sum(hidden, table, ids, status, pos, scale=8.0, pairs=pairs, pos_table=places,              # noqa: E731
-                                     pair_hash=(buckets, 31, 17), last_id=last, seq_of_token=seq_of, seq_starts=starts, state_slots=st)
+                                     pair_hash=(buckets, 1009, 263), last_id=last, seq_of_token=seq_of, seq_starts=starts, state_slots=st)
     res["embed_sum"] = line(_time(both, a.iters, a.warmup), n * h * (3 * item + 4))
     return res
 
